@@ -3,8 +3,8 @@
 The reference keeps one pool whose page ids are valid in every layer
 (tinyinfer/engine/block_manager.py:53-67) and gives pages back only when a request ends
 (:174-177). Here the cache entries of a model are put into *groups* by what they need (number of
-kv heads, head size, window); each group has a pool and each request one block table per group,
-so that a group whose mixers read only a window of keys can give pages back as soon as the window
+kv heads, head size, window or chunk); each group has a pool and each request one block table per group,
+so that a group whose mixers read only a window (or a chunk) of keys can give pages back as soon as it
 has passed them, while a group that reads all keys keeps them to the end. Beside the pages, a
 request holds one *state slot* for per-request state of fixed size.
 
@@ -145,7 +145,7 @@ def prefix_caching_possible(needs) -> bool:
     of cache entries, every one keeping all keys, and no per-request state."""
     needs = list(needs)
     groups = group_cache_needs(needs)
-    return (len(groups) == 1 and groups[0][0].window is None
+    return (len(groups) == 1 and groups[0][0].keeps_all
             and all(state is None for _need, state in needs))
 
 
@@ -270,9 +270,7 @@ class CacheManager:
     # ------------------------------------------------------------------ pages
     def _first_needed_page(self, group: CacheGroup, start: int) -> int:
         """Lowest logical page a query at position >= start can read in this group."""
-        if group.need.window is None:
-            return 0
-        return max(0, start - group.need.window + 1) // self.page_size
+        return group.need.first_read(start) // self.page_size
 
     def _missing(self, rc: RequestCache, new_length: int) -> List[int]:
         """Per group, how many pages must be taken to hold positions < new_length."""
@@ -317,14 +315,14 @@ class CacheManager:
 
     def commit(self, request_id, new_length: int) -> None:
         """Records that keys of positions < new_length are stored, and gives back every page a
-        window has passed: no later query of this request can read it."""
+        window or a chunk has passed: no later query of this request can read it."""
         rc = self._requests[request_id]
         if new_length < rc.length:
             raise ValueError("a request's cache cannot shrink")
         for g, table in zip(self.groups, rc.tables):
             if len(table) * self.page_size < new_length:
                 raise RuntimeError("commit beyond the pages held")
-            if g.need.window is None:
+            if g.need.keeps_all:
                 continue
             for logical in range(min(self._first_needed_page(g, new_length), len(table))):
                 if table[logical] >= 0:
@@ -354,7 +352,7 @@ class CacheManager:
             "prefix_queries": self.prefix_queries,
             "prefix_hit_tokens": self.prefix_hit_tokens,
             "kept_pages": len(self._page_key),
-            "groups": [{"window": g.need.window, "entries": len(g.entries),
+            "groups": [{"window": g.need.window, "chunk": g.need.chunk, "entries": len(g.entries),
                         "pages": g.pool.num_pages, "free_pages": g.pool.num_free,
                         "pages_taken": g.pool.pages_taken, "pages_returned": g.pool.pages_returned}
                        for g in self.groups],

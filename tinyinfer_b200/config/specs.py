@@ -14,12 +14,14 @@ from typing import Optional, Tuple
 
 @dataclass(frozen=True)
 class NormSpec:
-    """A normalisation over the last axis. ``kind='rmsnorm'``: w * x * rsqrt(mean(x^2) + eps)."""
+    """A normalisation over the last axis. ``kind='rmsnorm'``: w * x * rsqrt(mean(x^2) + eps). ``single_gain``: the
+    checkpoint has ONE number for w (a tensor without dimensions), the same for every coordinate."""
     size: int
     eps: float
     kind: str = "rmsnorm"
     tensor: str = "weight"                  # local name of the weight behind the norm's prefix ('' : the prefix itself)
     offset: float = 0.0                     # the stored weight is added to this (1.0: a weight stored around zero)
+    single_gain: bool = False
 
 
 @dataclass(frozen=True)
@@ -70,6 +72,12 @@ class AttentionSpec:
     softcap: Optional[float] = None         # a score s becomes softcap * tanh(s / softcap) before the softmax
     qk_unit_norm: Optional[float] = None    # eps: q and k are divided by their root mean square per head (no weight)
                                             # AFTER the rotation
+    chunk: Optional[int] = None             # n: a query sees the keys of its own chunk of n positions, chunks counted
+                                            # from position 0 of the request (not together with ``window``)
+    conv_taps: int = 0                      # a causal convolution per channel of q, k and v right after the projection
+                                            # (0: none; 1: a weight per channel; 'q.conv', 'k.conv', 'v.conv')
+    qk_row_norm: Optional[NormSpec] = None  # norm of ALL rows of q, and of k, at once before the rotation (weights 'q.norm'
+                                            # and 'k.norm' as long as the projections); its ``size`` is not used
 
     @property
     def q_size(self) -> int:
@@ -86,7 +94,7 @@ class AttentionSpec:
 
 @dataclass(frozen=True)
 class GatedMLPSpec:
-    """Dense gated feed-forward: down(act(gate(x)) * up(x)), no bias."""
+    """Dense gated feed-forward: down(act(gate(x)) * up(x)), no bias; act 'silu' or 'gelu_tanh' (the tanh form)."""
     hidden_size: int
     intermediate_size: int
     activation: str = "silu"
@@ -156,6 +164,10 @@ class ExpertsSpec:
     # activation 'silu_glu': an expert is down(silu(gate h) * (up h))
     scoring: str = "softmax"                # 'sigmoid': an expert's score is the sigmoid of its own router logit
     weight_input: bool = False              # the weight multiplies what the expert READS (expert(w h)), not its output
+    groups: int = 1                         # the experts form this many equal groups of neighbours; a group's score is its
+    keep_groups: int = 1                    # best expert's, and only experts of the best ``keep_groups`` groups can be chosen
+    weight_scale: float = 1.0               # a factor on the weights
+    shared_gate: bool = False               # the shared expert's output is multiplied by sigmoid(w_sg . h), one number a token
 
 
 @dataclass(frozen=True)
@@ -234,6 +246,25 @@ class ChannelDeltaSpec:
 
 
 @dataclass(frozen=True)
+class GeneralDeltaSpec:
+    """The generalized delta rule with a decay AND a removal rate per head and key channel. r, k (``num_heads`` heads of
+    ``key_dim``) and v (of ``value_dim``) are projections; with u = k / sqrt(k.k + ``unit_eps``),
+    w = exp(``decay_scale`` * sigmoid(W_w2 tanh(W_w1 h) + w0)) and a = sigmoid(W_a h + b):
+    S <- diag(w) S - (a * u)(u^T S) + k v^T (both terms from the old S), o = S^T r. Each head's o is divided by its root
+    mean square; the heads side by side are multiplied by one weight of their length and by sigmoid(W_g h), and projected.
+    ``gate_rank``: the inner size of the decay's two projections; 0: whatever the checkpoint's tensors have."""
+    hidden_size: int
+    num_heads: int
+    key_dim: int
+    value_dim: int
+    decay_scale: float
+    norm_eps: float
+    unit_eps: float = 1e-6
+    gate_rank: int = 0
+    kind: str = "general_delta"
+
+
+@dataclass(frozen=True)
 class StateSpaceSpec:
     """Selective state-space mixer with a scalar decay per head (state-space duality): the input projection
     gives [z | x | B | C | dt]; x, B and C pass a causal convolution with bias and silu; dt = softplus(dt + dt_bias);
@@ -288,6 +319,10 @@ class LayerSpec:
     through its norm and writes back into all of them (``learned_mixing``: the block owns the coefficients
     ``hc1.*`` for the mixer and ``hc2.*`` for the feed-forward; otherwise all are 1, which with one stream is the
     pre-norm residual kept in float32).
+    ``arrangement='scaled_residual'``: x += m * (s1 * mixer(shift(norm1(x)))); x += m * (s2 * feed_forward(norm2(x))) around
+    one float32 stream: m is ``residual_mult``, s1 and s2 are vectors named by ``mixer_scale`` and ``feed_forward_scale``
+    behind the layer's prefix (None: no such factor), and shift, named by ``token_shift``, replaces h_t by
+    h_t + (h_(t-1) - h_t) * v per feature, the h before a request's first token being zero (None: no shift).
     ``feed_forward`` None (with ``feed_forward_norm`` None): the block has a mixer only.
     ``mixer_out_norm`` / ``feed_forward_out_norm`` ('multi_stream' only): a second norm on the sublayer's OUTPUT
     before it is added, x += norm_b(sublayer(norm(x))); its ``tensor`` is the name behind the LAYER's prefix.
@@ -303,16 +338,23 @@ class LayerSpec:
     mixer_out_norm: Optional[NormSpec] = None
     feed_forward_out_norm: Optional[NormSpec] = None
     index: Optional[int] = None
+    residual_mult: float = 1.0                  # 'scaled_residual' only, like the three names below
+    mixer_scale: Optional[str] = None
+    feed_forward_scale: Optional[str] = None
+    token_shift: Optional[str] = None
 
 
 @dataclass(frozen=True)
 class ExecStep:
     """One entry of the run order. ``layer`` indexes ``ModelSpec.layers`` (a layer may be named
     more than once). ``cache`` names the cache entry the mixer works on; ``writes_cache`` is
-    False for an entry that only reads what an earlier entry wrote there."""
+    False for an entry that only reads what an earlier entry wrote there. Right before the layer, ``adds_embedding``
+    adds the embedding's output to the residual, and ``adds_vector`` a row of ``ModelSpec.step_vectors``."""
     layer: int
     cache: int
     writes_cache: bool = True
+    adds_embedding: bool = False
+    adds_vector: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -340,9 +382,13 @@ class ModelSpec:
     tie_embeddings: bool
     max_positions: int
     names: TensorNames = field(default_factory=TensorNames)
+    step_vectors: Optional[Tuple[str, int]] = None      # (tensor name, rows): vectors that entries of the run order add
 
     def __post_init__(self):
         seen = set()
+        rows = self.step_vectors[1] if self.step_vectors else 0
+        if any(s.adds_vector is not None and not 0 <= s.adds_vector < rows for s in self.execution):
+            raise ValueError(f"the run order adds a vector that is not among the model's {rows}")
         for step in self.execution:
             if not 0 <= step.layer < len(self.layers):
                 raise ValueError(f"execution names layer {step.layer}, the model has {len(self.layers)}")

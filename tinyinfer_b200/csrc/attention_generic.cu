@@ -25,7 +25,7 @@ __global__ void __launch_bounds__(AG_THREADS) attention_generic_kernel(
     const int tid = threadIdx.x;
     const int h = blockIdx.x, t = blockIdx.y;
     const int pos = positions[t];
-    const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+    const int lo = ti_first_key(pos, window);
     const int kvh = h / (hq / hkv);
     const int* table = block_table + (size_t)token_seq[t] * max_blocks;
     const T* qrow = q + ((size_t)t * hq + h) * d;
@@ -85,7 +85,7 @@ TI_API int ti_attention_generic(
     int num_pages, float scale, int window, int* status, int dtype, cudaStream_t stream) {
     TI_REQUIRE(d > 0 && d <= AG_MAX_D, "attention: head_dim %d not in 1..%d", d, AG_MAX_D);
     TI_REQUIRE(hq > 0 && hkv > 0 && hq % hkv == 0, "attention: %d query heads do not group over %d kv heads", hq, hkv);
-    TI_REQUIRE(page_size > 0 && num_tokens >= 0 && window >= 0, "attention: bad sizes");
+    TI_REQUIRE(page_size > 0 && num_tokens >= 0, "attention: bad sizes");
     TI_REQUIRE(num_tokens <= 65535, "attention: more than 65535 tokens in one step");
     if (num_tokens == 0) return 0;
     const size_t v_off = (size_t)num_pages * hkv * page_size * d;

@@ -141,7 +141,7 @@ __device__ __forceinline__ RowTiles row_tiles(const AttnParams& p, int r) {
     RowTiles t;
     t.row = p.rows[r];
     t.ctx = p.positions[t.row] + 1;
-    t.lo = p.window > 0 ? max(0, t.ctx - p.window) : 0;
+    t.lo = ti_first_key(t.ctx - 1, p.window);
     t.lo_tile = t.lo / TK;
     t.n = (t.ctx + TK - 1) / TK - t.lo_tile;
     return t;
@@ -642,7 +642,8 @@ int decode_slots(int d, int group) {
 // alone, so a captured launch and the scratch sized for it agree.
 TI_API int ti_attention_decode_ctas(int num_rows, int hq, int hkv, int d, int max_context, int window) {
     if (num_rows <= 0 || hkv <= 0 || hq % hkv != 0 || (d != 64 && d != 128) || max_context <= 0) return 1;
-    const long long visible = window > 0 && window + TK < max_context ? window + TK : max_context;
+    const int span = window < 0 ? -window : window;         // a window's or a chunk's keys, and one tile for its edges
+    const long long visible = span > 0 && span < max_context - TK ? span + TK : max_context;
     const long long runs = ((long long)num_rows * hkv * ((visible + TK - 1) / TK) + MIN_RUN_TILES - 1) / MIN_RUN_TILES;
     // Seven eighths of the CTAs that would run side by side, where two and more share an SM: every SM still streams,
     // and the free places let the CTAs of the kernel behind (the output projection) move in and ask for their

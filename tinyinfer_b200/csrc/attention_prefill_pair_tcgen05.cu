@@ -175,13 +175,13 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap q_map, const _
         const int rows_x = min(QM, nrows - x * QM);
         if (rows_x <= 0) { t0x[x] = 0; t1x[x] = 0; continue; }
         const int first = pos0 + x * QM, hi_x = first + rows_x;
-        const int lo_x = p.window > 0 ? max(0, first - p.window + 1) : 0;
+        const int lo_x = ti_first_key(first, p.window);
         t0x[x] = lo_x / KT;
         t1x[x] = (hi_x + KT - 1) / KT;
     }
     const bool has_b = t1x[1] > t0x[1];
     const int tmin = has_b ? min(t0x[0], t0x[1]) : t0x[0], tmax = has_b ? max(t1x[0], t1x[1]) : t1x[0];
-    const int lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;   // first key any query of the CTA sees
+    const int lo = ti_first_key(pos0, p.window);                     // first key any query of the CTA sees
     const int hi = pos0 + nrows;                                     // one past the last
 
     if (warp == 0) {
@@ -308,6 +308,7 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap q_map, const _
         const uint32_t lane_addr = tmem_base + ((uint32_t)(lane_group * 32) << 16);
         const uint32_t s_tmem = lane_addr + x * KT, o_tmem = lane_addr + 2 * KT + x * D;
         const int gtid = threadIdx.x - 64 - x * 128;                    // 0..127 among this tile's softmax threads
+        const int before_row = ti_first_key(qpos, p.window) - 1;          // one before the first key the row may see
         float m_ref = -INFINITY, l_run = 0.f;
         bool ok = true;
         for (int i = 0; i < num_x && ok; ++i) {
@@ -317,7 +318,7 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap q_map, const _
             tmem_fence_after();
             // columns of this tile the row may see: kmin < column <= kmax (tile-local)
             const int kmax = qpos - tk0;
-            const int kmin = p.window > 0 ? qpos - p.window - tk0 : -1;
+            const int kmin = before_row - tk0;
             const bool all_seen = KT - 1 <= kmax && kmin < 0;
             uint32_t sr[KT];
 #pragma unroll

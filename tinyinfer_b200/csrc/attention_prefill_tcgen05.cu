@@ -122,7 +122,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
     const int head = blockIdx.x;
     const int kvh = head / (p.hq / p.hkv);
     const int hi = pos0 + nrows;                                   // one past the last key any query sees
-    const int lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0; // first key the first query sees
+    const int lo = ti_first_key(pos0, p.window);                     // first key the first query sees
     // With a split of the keys (few query tiles behind long prefixes: too few CTAs otherwise) this CTA takes the
     // key tiles of its share only and leaves an unnormalised partial result for the merge kernel.
     int tile0 = lo / KT, tile1 = (hi + KT - 1) / KT;
@@ -234,6 +234,10 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
         const int qpos = pos0 + r;
         const int etid = threadIdx.x - 64;                             // 0..255 among the softmax threads
         constexpr int KH = KT / 2, DH = D / 2;                         // this thread's share of keys and features
+        // one before the first key that this thread's row, and the warp's first and last row, may see
+        const int before_row = ti_first_key(qpos, p.window) - 1;
+        const int before_first = ti_first_key(pos0 + lane_group * 32, p.window) - 1;
+        const int before_last = ti_first_key(pos0 + lane_group * 32 + 31, p.window) - 1;
         float o[DH];
 #pragma unroll
         for (int i = 0; i < DH; ++i) o[i] = 0.f;
@@ -247,11 +251,11 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
             // Columns of this tile the row may see: kmin < column <= kmax (tile-local). A chunk of 32
             // columns inside that range needs no per-element test, one outside it no arithmetic at all.
             const int kmax = qpos - tk0;
-            const int kmin = p.window > 0 ? qpos - p.window - tk0 : -1;
+            const int kmin = before_row - tk0;
             // the same bounds for the warp's first and last row: the choice per chunk must be the
             // same for the whole warp, because tcgen05.ld is a warp-wide instruction
             const int wmax0 = pos0 + lane_group * 32 - tk0, wmax1 = wmax0 + 31;
-            const int wmin0 = p.window > 0 ? wmax0 - p.window : -1, wmin1 = p.window > 0 ? wmax1 - p.window : -1;
+            const int wmin0 = before_first - tk0, wmin1 = before_last - tk0;
             float v[32];
             // pass 1: the row maximum of the visible scores (raw; the scale is positive)
             float mx = -INFINITY;
@@ -404,7 +408,7 @@ __global__ void prefill_merge_kernel(const PrefillParams p) {
     const int nrows = min(td.z - half_off, QM);
     if (r >= nrows) return;
     const int hi = pos0 + nrows;
-    const int lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
+    const int lo = ti_first_key(pos0, p.window);
     const int tile0 = lo / KT, tile1 = (hi + KT - 1) / KT, per = p.split_keys / KT;
     float m_run = -INFINITY, acc = 0.f, l_all = 0.f;
     for (int z = tile0 / per; z < p.splits && z * per < tile1; ++z) {

@@ -124,6 +124,14 @@ __device__ __forceinline__ float block_max(float v, float* red) {
     return r;
 }
 
+// The first key position that a query at position `pos` may see (the last is pos itself). window > 0: the last `window`
+// keys; window < 0: its own chunk of -window positions, chunks counted from position 0 of the request; 0: every key.
+// It never falls as pos grows, which is what the kernels' ranges of key tiles rest on.
+__device__ __forceinline__ int ti_first_key(int pos, int window) {
+    if (window > 0) return max(0, pos - window + 1);
+    return window < 0 ? pos - pos % -window : 0;
+}
+
 // Scores that level off smoothly: s -> cap * tanh(s / cap). P is an attention kernel's parameter block with scale_log2
 // (the softmax scale times log2 e), cap_log2 (cap * log2 e; 0: no cap) and cap_arg (scale / cap). The result is in log2
 // units, like raw * scale_log2; a masked score (-inf) stays -inf. These are the bfloat16 tensor-core kernels, whose

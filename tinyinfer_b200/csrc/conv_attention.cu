@@ -16,84 +16,10 @@
 //                       softmax denominator holds one more term exp(sink) that has no value ("sink")
 // Everything is computed in float32 from the stored operands; each result is rounded once.
 #include "common.cuh"
+#include "short_conv.cuh"
 
-constexpr int SC_MAX_TAPS = 16;
-
-template <typename T>
-__device__ __forceinline__ float conv_at(const T* __restrict__ in, int ld_in, int col, int t, int local,
-                                         const float* __restrict__ hist, int width, int c,
-                                         const float* __restrict__ w, int taps) {
-    float acc = 0.f;
-    for (int j = 0; j < taps; ++j) {                       // column taps - 1 meets the current token
-        const int back = taps - 1 - j;
-        const float v = local - back >= 0 ? to_f32(in[(size_t)(t - back) * ld_in + col])
-                                          : hist[(size_t)(taps - 1 + local - back) * width + c];
-        acc = fmaf(w[(size_t)j * width + c], v, acc);
-    }
-    return acc;
-}
-
-// A step in which every request brings ONE token: the thread that made the token's output is the only one that
-// read this channel's history, so it may also move the history on by one (oldest out, the token's input in).
-__device__ __forceinline__ void conv_shift_history(float* __restrict__ hist, int width, int c, int taps, float newest) {
-    float kept[SC_MAX_TAPS];
-    for (int j = 1; j < taps - 1; ++j) kept[j] = hist[(size_t)j * width + c];
-    for (int j = 1; j < taps - 1; ++j) hist[(size_t)(j - 1) * width + c] = kept[j];
-    hist[(size_t)(taps - 2) * width + c] = newest;
-}
-
-// ------------------------------------------------------------------ sixteen bytes of channels a thread
 // The *_vec kernels do the same as short_conv_kernel and conv_qkv_append_kernel for rows whose pieces (q, k, v, a
 // head) all start on 16-byte boundaries: a thread takes V = 16 / sizeof(T) neighbouring channels, one load per tap, one store.
-template <typename T, int V>
-__device__ __forceinline__ void load_row(const T* __restrict__ p, float* v) {
-    const uint4 raw = *reinterpret_cast<const uint4*>(p);
-    const T* e = reinterpret_cast<const T*>(&raw);
-#pragma unroll
-    for (int i = 0; i < V; ++i) v[i] = to_f32(e[i]);
-}
-template <typename T, int V>
-__device__ __forceinline__ void store_row(T* __restrict__ p, const float* v) {
-    uint4 raw;
-    T* e = reinterpret_cast<T*>(&raw);
-#pragma unroll
-    for (int i = 0; i < V; ++i) e[i] = from_f32<T>(v[i]);
-    *reinterpret_cast<uint4*>(p) = raw;
-}
-
-// acc[i] = sum_j w[j][c0 + i] * in(t - (taps - 1 - j))[c0 + i]; newest[i]: the current token's own input.
-template <typename T, int V>
-__device__ __forceinline__ void conv_at_vec(const T* __restrict__ in, int ld_in, int col0, int t, int local,
-                                            const float* __restrict__ hist, int width, int c0,
-                                            const float* __restrict__ w, int taps, float* acc, float* newest) {
-#pragma unroll
-    for (int i = 0; i < V; ++i) acc[i] = 0.f;
-    for (int j = 0; j < taps; ++j) {
-        const int back = taps - 1 - j;
-        float v[V];
-        if (local - back >= 0) {
-            load_row<T, V>(in + (size_t)(t - back) * ld_in + col0, v);
-        } else {
-#pragma unroll
-            for (int i = 0; i < V; ++i) v[i] = hist[(size_t)(taps - 1 + local - back) * width + c0 + i];
-        }
-        float wj[V];
-        if (w) {
-#pragma unroll
-            for (int i = 0; i < V; i += 4) {
-                const float4 f = *reinterpret_cast<const float4*>(w + (size_t)j * width + c0 + i);
-                wj[i] = f.x; wj[i + 1] = f.y; wj[i + 2] = f.z; wj[i + 3] = f.w;
-            }
-        }
-#pragma unroll
-        for (int i = 0; i < V; ++i) acc[i] = fmaf(w ? wj[i] : 1.f, v[i], acc[i]);
-        if (back == 0) {
-#pragma unroll
-            for (int i = 0; i < V; ++i) newest[i] = v[i];
-        }
-    }
-}
-
 template <typename T>
 __global__ void short_conv_vec_kernel(T* __restrict__ out, const T* __restrict__ in, int ld_in, int in_off,
                                       const float* __restrict__ state, long long slot_stride, const float* __restrict__ w,
@@ -386,7 +312,7 @@ __global__ void __launch_bounds__(AR_THREADS) attention_rows_kernel(
     const int tid = threadIdx.x;
     const int h = blockIdx.x, t = blockIdx.y;
     const int pos = positions[t];
-    const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+    const int lo = ti_first_key(pos, window);
     const int kvh = h / (hq / hkv);
     const int* table = block_table + (size_t)token_seq[t] * max_blocks;
     const T* qrow = q + ((size_t)t * hq + h) * d;
@@ -462,7 +388,7 @@ TI_API int ti_attention_rows(void* out, const void* q, const void* cache, const 
     const long long v_off = planes == 2 ? (long long)num_pages * hkv * page_size * d : d;
     TI_REQUIRE(d > 0 && d <= AR_MAX_D && dv > 0 && dv <= AR_MAX_D, "attention_rows: head sizes %d / %d not in 1..%d", d, dv, AR_MAX_D);
     TI_REQUIRE(hq > 0 && hkv > 0 && hq % hkv == 0, "attention_rows: %d query heads do not group over %d kv heads", hq, hkv);
-    TI_REQUIRE(page_size > 0 && num_tokens >= 0 && window >= 0 && softcap >= 0.f, "attention_rows: bad sizes");
+    TI_REQUIRE(page_size > 0 && num_tokens >= 0 && softcap >= 0.f, "attention_rows: bad sizes");
     TI_REQUIRE(num_tokens <= 65535, "attention_rows: more than 65535 tokens in one step");
     if (num_tokens == 0) return 0;
     dim3 grid(hq, num_tokens);

@@ -15,6 +15,14 @@
 //   read-out is o = D^T q + u (k.q): both sums over the rows, D^T k and D^T q, are taken in one pass and meet in
 //   one round of shuffles, and only S <- D + k u^T is carried to the next token. Chunks of tokens come into shared
 //   memory by cp.async, the next chunk while the current one is walked.
+//
+// The general form (ti_general_delta_scan) removes along a unit key with a rate per head and key channel, and adds the
+// key as it is. With u = k / sqrt(k.k + unit_eps), for every token
+//     S <- diag(w) S - (a * u) (u^T S) + k v^T          (both terms read the old S)          o = S^T r
+// Its own prepare kernel, a warp a token and head, makes per channel u, r, the decay w = exp(decay_scale *
+// sigmoid(logit + bias)) and the rate a = sigmoid(logit + bias), per value column p = sqrt(k.k + unit_eps) * v (so that
+// k v^T = u p^T), and the two products r.u and r.(a * u). The walk is the same kernel: with e = u^T S of the old state
+// a row becomes w s + u (p - a e), and o = r^T diag(w) S - e (r.(a * u)) + p (r.u), again one round of shuffles.
 #include "common.cuh"
 
 constexpr int DS_MAX_WARPS = 4;
@@ -26,7 +34,8 @@ struct DeltaWork {                // float32, one row per token of the step
     float *q, *k;                 // [T][groups * dk]
     float* g;                     // [T][heads * dk]
     float* v;                     // [T][heads * dv]
-    float *kq, *beta;             // [T][groups], [T][heads]
+    float *kq, *beta;             // [T][groups], [T][heads]; general form: r.u and r.(a * u)
+    float* a;                     // general form: the removal rate, [T][heads * dk] (q: r, k: u, g: w, v: p, groups = heads)
 };
 
 struct DeltaPrepArgs {
@@ -80,6 +89,59 @@ __global__ void __launch_bounds__(DP_THREADS) delta_prepare_kernel(DeltaPrepArgs
     if (tid == 0) a.w.beta[(size_t)t * a.heads + h] = 1.f / (1.f + expf(-a.b[(size_t)t * a.ld_b + a.b_off + h]));
 }
 
+struct GeneralPrepArgs {
+    DeltaWork w;
+    const void *r, *k, *v;        // rows of ld_* elements, first column *_off: [H][dk], [H][dk], [H][dv]
+    int ld_r, r_off, ld_k, k_off, ld_v, v_off;
+    const float* decay;           // float32 rows of ld_decay, first column decay_off: [H][dk] logits; bias decay_b or null
+    int ld_decay, decay_off;
+    const float* rate;            // the same for the removal rate
+    int ld_rate, rate_off;
+    const float *decay_b, *rate_b;
+    float decay_scale, unit_eps;
+    int tokens, heads, dk, dv;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(DP_THREADS) general_delta_prepare_kernel(GeneralPrepArgs a) {
+    ti_grid_launch_dependents();
+    ti_grid_wait();
+    const int lane = threadIdx.x & 31;
+    const size_t item = (size_t)blockIdx.x * (DP_THREADS / 32) + (threadIdx.x >> 5);     // (token, head)
+    if (item >= (size_t)a.tokens * a.heads) return;
+    const size_t t = item / a.heads;
+    const int h = (int)(item % a.heads);
+    const T* r = (const T*)a.r + t * a.ld_r + a.r_off + (size_t)h * a.dk;
+    const T* k = (const T*)a.k + t * a.ld_k + a.k_off + (size_t)h * a.dk;
+    const float* dl = a.decay + t * a.ld_decay + a.decay_off + (size_t)h * a.dk;
+    const float* rl = a.rate + t * a.ld_rate + a.rate_off + (size_t)h * a.dk;
+    const size_t row = item * a.dk;                      // [T][heads * dk]
+    float ss = 0.f, rk = 0.f, rak = 0.f;
+    for (int c = lane; c < a.dk; c += 32) {
+        const float rv = to_f32(r[c]), kv = to_f32(k[c]);
+        const float zd = dl[c] + (a.decay_b ? a.decay_b[h * a.dk + c] : 0.f);
+        const float zr = rl[c] + (a.rate_b ? a.rate_b[h * a.dk + c] : 0.f);
+        const float rate = 1.f / (1.f + expf(-zr));
+        a.w.q[row + c] = rv;
+        a.w.g[row + c] = expf(a.decay_scale / (1.f + expf(-zd)));
+        a.w.a[row + c] = rate;
+        ss = fmaf(kv, kv, ss);
+        rk = fmaf(rv, kv, rk);
+        rak = fmaf(rv * rate, kv, rak);
+    }
+    ss = warp_sum(ss);
+    rk = warp_sum(rk);
+    rak = warp_sum(rak);
+    const float len = sqrtf(ss + a.unit_eps), inv = 1.f / len;
+    for (int c = lane; c < a.dk; c += 32) a.w.k[row + c] = to_f32(k[c]) * inv;
+    const T* v = (const T*)a.v + t * a.ld_v + a.v_off + (size_t)h * a.dv;
+    for (int c = lane; c < a.dv; c += 32) a.w.v[item * a.dv + c] = to_f32(v[c]) * len;
+    if (lane == 0) {
+        a.w.kq[item] = rk * inv;
+        a.w.beta[item] = rak * inv;
+    }
+}
+
 __device__ __forceinline__ void ds_copy16(float* dst, const float* src) {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
@@ -99,11 +161,12 @@ struct DeltaScanArgs {
     int vec_k, vec_v;             // rows of dk floats, and a block's columns of v, move in 16-byte pieces
 };
 
-template <int KPT, int KP>
+template <int KPT, int KP, bool GENERAL>
 __global__ void __launch_bounds__(DS_MAX_WARPS * 32) delta_scan_kernel(DeltaScanArgs a) {
     extern __shared__ __align__(16) float smem[];
     constexpr int PITCH = KPT + 4;                       // floats from one lane part's rows to the next: no two lanes in a bank
     constexpr int trow = KP * PITCH;
+    constexpr int ROWS = GENERAL ? 4 : 3;                // rows of channels a token brings: q, k, g and, in the general form, a
     constexpr int cols_per_warp = 32 / KP;
     const int threads = blockDim.x, warps = threads >> 5;
     const int cpb = warps * cols_per_warp;
@@ -116,7 +179,7 @@ __global__ void __launch_bounds__(DS_MAX_WARPS * 32) delta_scan_kernel(DeltaScan
     const int col = cb * cpb + lcol;
     const bool col_ok = col < a.dv;
     const int g = h / (a.heads / a.groups);
-    const int buf_floats = (a.chunk * (3 * trow + cpb + 2) + 3) & ~3;
+    const int buf_floats = (a.chunk * (ROWS * trow + cpb + 2) + 3) & ~3;
     for (int e = tid; e < 2 * buf_floats; e += threads) smem[e] = 0.f;   // the rows past dk stay zero
     // which pieces of a token's rows this thread fetches: piece p_first (and every `threads`-th after it) of the
     // tokens tt_first, tt_first + tt_step, ...; with more threads than pieces, several tokens side by side
@@ -139,7 +202,8 @@ __global__ void __launch_bounds__(DS_MAX_WARPS * 32) delta_scan_kernel(DeltaScan
         float* sq = buf;
         float* sk = sq + (size_t)a.chunk * trow;
         float* sg = sk + (size_t)a.chunk * trow;
-        float* sv = sg + (size_t)a.chunk * trow;         // [chunk][cpb]
+        float* sa = sg + (size_t)a.chunk * trow;         // general form only
+        float* sv = sq + (size_t)ROWS * a.chunk * trow;  // [chunk][cpb]
         float* sb = sv + (size_t)a.chunk * cpb;          // [chunk]
         float* sx = sb + a.chunk;                        // [chunk]: k.q
         if (tt_first < tt_step) {
@@ -150,13 +214,16 @@ __global__ void __launch_bounds__(DS_MAX_WARPS * 32) delta_scan_kernel(DeltaScan
                 const float* gq = a.w.q + ((size_t)(t0 + tt_first) * a.groups + g) * a.dk + idx;
                 const float* gk = a.w.k + ((size_t)(t0 + tt_first) * a.groups + g) * a.dk + idx;
                 const float* gg = a.w.g + ((size_t)(t0 + tt_first) * a.heads + h) * a.dk + idx;
+                const float* ga = GENERAL ? a.w.a + ((size_t)(t0 + tt_first) * a.heads + h) * a.dk + idx : nullptr;
                 for (int tt = tt_first; tt < n; tt += tt_step) {
                     if (a.vec_k) { ds_copy16(sq + at, gq); ds_copy16(sk + at, gk); ds_copy16(sg + at, gg); }
                     else { ds_copy4(sq + at, gq); ds_copy4(sk + at, gk); ds_copy4(sg + at, gg); }
+                    if constexpr (GENERAL) { if (a.vec_k) ds_copy16(sa + at, ga); else ds_copy4(sa + at, ga); }
                     at += tt_step * trow;
                     gq += tt_step * ld_qk;
                     gk += tt_step * ld_qk;
                     gg += tt_step * ld_g;
+                    if constexpr (GENERAL) ga += tt_step * ld_g;
                 }
             }
         }
@@ -185,7 +252,8 @@ __global__ void __launch_bounds__(DS_MAX_WARPS * 32) delta_scan_kernel(DeltaScan
         const float* sq = smem + which * buf_floats;
         const float* sk = sq + (size_t)a.chunk * trow;
         const float* sg = sk + (size_t)a.chunk * trow;
-        const float* sv = sg + (size_t)a.chunk * trow;
+        const float* sa = sg + (size_t)a.chunk * trow;   // general form only
+        const float* sv = sq + (size_t)ROWS * a.chunk * trow;
         const float* sb = sv + (size_t)a.chunk * cpb;
         const float* sx = sb + a.chunk;
         for (int tt = 0; tt < n; ++tt) {
@@ -203,8 +271,12 @@ __global__ void __launch_bounds__(DS_MAX_WARPS * 32) delta_scan_kernel(DeltaScan
 #pragma unroll
                 for (int j = 0; j < 4; ++j) {
                     const int r = r4 * 4 + j;
+                    const float old = S[r];
                     S[r] *= gr[j];
-                    if (j & 1) { dk1 = fmaf(S[r], kr[r], dk1); dq1 = fmaf(S[r], qr[j], dq1); }
+                    if constexpr (GENERAL) {             // the removal reads the old state, the read-out the decayed one
+                        if (j & 1) { dk1 = fmaf(old, kr[r], dk1); dq1 = fmaf(S[r], qr[j], dq1); }
+                        else { dk0 = fmaf(old, kr[r], dk0); dq0 = fmaf(S[r], qr[j], dq0); }
+                    } else if (j & 1) { dk1 = fmaf(S[r], kr[r], dk1); dq1 = fmaf(S[r], qr[j], dq1); }
                     else { dk0 = fmaf(S[r], kr[r], dk0); dq0 = fmaf(S[r], qr[j], dq0); }
                 }
             }
@@ -214,10 +286,27 @@ __global__ void __launch_bounds__(DS_MAX_WARPS * 32) delta_scan_kernel(DeltaScan
                 dot += __shfl_xor_sync(0xffffffffu, dot, off);
                 oq += __shfl_xor_sync(0xffffffffu, oq, off);
             }
-            const float u = beta * (vv - dot);
+            float o;
+            if constexpr (GENERAL) {
+                const float4* pa = reinterpret_cast<const float4*>(sa + (size_t)tt * trow + kpart * PITCH);
 #pragma unroll
-            for (int r = 0; r < KPT; ++r) S[r] = fmaf(kr[r], u, S[r]);
-            if (kpart == 0 && col_ok) a.y[(size_t)(t0 + tt) * a.heads * a.dv + h * a.dv + col] = fmaf(u, kq, oq);
+                for (int r4 = 0; r4 < KPT / 4; ++r4) {
+                    const float4 av = pa[r4];
+                    const float ar[4] = {av.x, av.y, av.z, av.w};
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) {
+                        const int r = r4 * 4 + j;
+                        S[r] = fmaf(kr[r], fmaf(-ar[j], dot, vv), S[r]);
+                    }
+                }
+                o = fmaf(vv, kq, fmaf(-dot, beta, oq));
+            } else {
+                const float u = beta * (vv - dot);
+#pragma unroll
+                for (int r = 0; r < KPT; ++r) S[r] = fmaf(kr[r], u, S[r]);
+                o = fmaf(u, kq, oq);
+            }
+            if (kpart == 0 && col_ok) a.y[(size_t)(t0 + tt) * a.heads * a.dv + h * a.dv + col] = o;
         }
         __syncthreads();                                 // the chunk has been read: its buffer may be filled again
     }
@@ -231,6 +320,48 @@ __global__ void __launch_bounds__(DS_MAX_WARPS * 32) delta_scan_kernel(DeltaScan
 }
 
 static inline size_t ds_round4(size_t n) { return (n + 3) & ~(size_t)3; }
+
+// The walk over the prepared rows `w`.
+template <bool GENERAL>
+static int ds_launch_scan(const DeltaWork& w, float* y, float* state, long long slot_stride, const int* cu_seqlens,
+                          const int* state_slots, int num_seqs, int num_tokens, int heads, int groups, int dk, int dv,
+                          cudaStream_t stream) {
+    constexpr int rows_in = GENERAL ? 4 : 3;
+    int kp = 1;
+    const int rows = 8;                                  // most rows of a column that a lane holds
+    while (kp < 32 && (dk + kp - 1) / kp > rows) kp <<= 1;
+    const int per_lane = (dk + kp - 1) / kp;
+    const int kpt = per_lane <= 4 ? 4 : per_lane <= 8 ? 8 : per_lane <= 16 ? 16 : 32;
+    // few columns a block when the step has few (request, head) pairs, so that every SM has a block; many columns a
+    // block otherwise, as every block fetches the head's q, k and g for itself
+    int warps = DS_MAX_WARPS;
+    while (warps > 1 && (long long)num_seqs * heads * ((dv + warps * (32 / kp) - 1) / (warps * (32 / kp))) < 148) warps >>= 1;
+    const int trow = kp * (kpt + 4), cpb = warps * (32 / kp);
+    // two buffers of `chunk` tokens within the 48 KB that need no opt-in; a step of single tokens stages no more than one
+    int chunk = 16;
+    while (chunk > 1 && 2 * ds_round4((size_t)chunk * (rows_in * trow + cpb + 2)) * sizeof(float) > 44 * 1024) chunk >>= 1;
+    if (num_tokens == num_seqs) chunk = 1;
+    const size_t smem = 2 * ds_round4((size_t)chunk * (rows_in * trow + cpb + 2)) * sizeof(float);
+    DeltaScanArgs args = {w, y, state, slot_stride, cu_seqlens, state_slots, heads, groups, dk, dv, chunk,
+                          dk % 4 == 0, dv % 4 == 0 && cpb % 4 == 0};
+    dim3 grid(heads * ((dv + cpb - 1) / cpb), num_seqs);
+    // a walk of many tokens starts alone (see ti_launch_alone); a step of single tokens is short and starts early
+    const bool alone = num_tokens != num_seqs;
+    bool launched = false;
+#define TI_DSCAN(KPT, KP)                                                                         \
+    if (!launched && kpt == KPT && kp == KP) {                                                    \
+        if (alone) ti_launch_alone(delta_scan_kernel<KPT, KP, GENERAL>, grid, warps * 32, smem, stream, args); \
+        else ti_launch(delta_scan_kernel<KPT, KP, GENERAL>, grid, warps * 32, smem, stream, args);         \
+        launched = true;                                                                          \
+    }
+#define TI_DSCAN_ROWS(KPT) TI_DSCAN(KPT, 1) TI_DSCAN(KPT, 2) TI_DSCAN(KPT, 4) TI_DSCAN(KPT, 8) TI_DSCAN(KPT, 16) TI_DSCAN(KPT, 32)
+    TI_DSCAN_ROWS(4) TI_DSCAN_ROWS(8) TI_DSCAN_ROWS(16) TI_DSCAN(32, 32)
+#undef TI_DSCAN_ROWS
+#undef TI_DSCAN
+    TI_REQUIRE(launched, "delta_scan: no kernel for %d rows a lane over %d lanes", kpt, kp);
+    TI_CHECK_LAUNCH("delta_scan");
+    return 0;
+}
 
 // floats of workspace for a step of t tokens: every part starts on a 16-byte boundary
 static inline size_t ds_workspace(size_t t, int heads, int groups, int dk, int dv) {
@@ -263,6 +394,7 @@ TI_API int ti_delta_scan(float* y, float* state, long long slot_stride, const vo
     w.v = w.g + ds_round4(t * heads * dk);
     w.kq = w.v + ds_round4(t * heads * dv);
     w.beta = w.kq + ds_round4(t * groups);
+    w.a = nullptr;
     DeltaPrepArgs prep = {w, q, k, v, ld_q, q_off, ld_k, k_off, ld_v, v_off, a, ld_a, a_off, b, ld_b, b_off,
                           a_log, dt_bias, q_scale, unit_eps, heads, groups, dk, dv};
     TI_REQUIRE(heads <= 65535, "delta_scan: too many heads");
@@ -270,38 +402,43 @@ TI_API int ti_delta_scan(float* y, float* state, long long slot_stride, const vo
     else ti_launch(delta_prepare_kernel<__nv_bfloat16>, dim3(num_tokens, heads), DP_THREADS, 0, stream, prep);
     TI_CHECK_LAUNCH("delta_prepare");
 
-    int kp = 1;
-    const int rows = 8;                                  // most rows of a column that a lane holds
-    while (kp < 32 && (dk + kp - 1) / kp > rows) kp <<= 1;
-    const int per_lane = (dk + kp - 1) / kp;
-    const int kpt = per_lane <= 4 ? 4 : per_lane <= 8 ? 8 : per_lane <= 16 ? 16 : 32;
-    // few columns a block when the step has few (request, head) pairs, so that every SM has a block; many columns a
-    // block otherwise, as every block fetches the head's q, k and g for itself
-    int warps = DS_MAX_WARPS;
-    while (warps > 1 && (long long)num_seqs * heads * ((dv + warps * (32 / kp) - 1) / (warps * (32 / kp))) < 148) warps >>= 1;
-    const int trow = kp * (kpt + 4), cpb = warps * (32 / kp);
-    // two buffers of `chunk` tokens within the 48 KB that need no opt-in; a step of single tokens stages no more than one
-    int chunk = 16;
-    while (chunk > 1 && 2 * ds_round4((size_t)chunk * (3 * trow + cpb + 2)) * sizeof(float) > 44 * 1024) chunk >>= 1;
-    if (num_tokens == num_seqs) chunk = 1;
-    const size_t smem = 2 * ds_round4((size_t)chunk * (3 * trow + cpb + 2)) * sizeof(float);
-    DeltaScanArgs args = {w, y, state, slot_stride, cu_seqlens, state_slots, heads, groups, dk, dv, chunk,
-                          dk % 4 == 0, dv % 4 == 0 && cpb % 4 == 0};
-    dim3 grid(heads * ((dv + cpb - 1) / cpb), num_seqs);
-    // a walk of many tokens starts alone (see ti_launch_alone); a step of single tokens is short and starts early
-    const bool alone = num_tokens != num_seqs;
-    bool launched = false;
-#define TI_DSCAN(KPT, KP)                                                                         \
-    if (!launched && kpt == KPT && kp == KP) {                                                    \
-        if (alone) ti_launch_alone(delta_scan_kernel<KPT, KP>, grid, warps * 32, smem, stream, args); \
-        else ti_launch(delta_scan_kernel<KPT, KP>, grid, warps * 32, smem, stream, args);         \
-        launched = true;                                                                          \
-    }
-#define TI_DSCAN_ROWS(KPT) TI_DSCAN(KPT, 1) TI_DSCAN(KPT, 2) TI_DSCAN(KPT, 4) TI_DSCAN(KPT, 8) TI_DSCAN(KPT, 16) TI_DSCAN(KPT, 32)
-    TI_DSCAN_ROWS(4) TI_DSCAN_ROWS(8) TI_DSCAN_ROWS(16) TI_DSCAN(32, 32)
-#undef TI_DSCAN_ROWS
-#undef TI_DSCAN
-    TI_REQUIRE(launched, "delta_scan: no kernel for %d rows a lane over %d lanes", kpt, kp);
-    TI_CHECK_LAUNCH("delta_scan");
-    return 0;
+    return ds_launch_scan<false>(w, y, state, slot_stride, cu_seqlens, state_slots, num_seqs, num_tokens, heads, groups, dk, dv,
+                                 stream);
+}
+
+// The general form. r, k, v in the compute dtype (heads heads of dk, dk and dv features); decay, rate: float32 logits per
+// head and key channel with biases (float32 [heads * dk], or null); w = exp(decay_scale * sigmoid(.)), so decay_scale <= 0.
+// work: at least T * heads * (4 dk + dv + 2) + 28 floats, 16-byte aligned. The rest as in ti_delta_scan.
+TI_API int ti_general_delta_scan(float* y, float* state, long long slot_stride, const void* r, int ld_r, int r_off,
+                                 const void* k, int ld_k, int k_off, const void* v, int ld_v, int v_off, const float* decay,
+                                 int ld_decay, int decay_off, const float* rate, int ld_rate, int rate_off,
+                                 const float* decay_b, const float* rate_b, float decay_scale, float unit_eps,
+                                 const int* cu_seqlens, const int* state_slots, int num_seqs, int num_tokens, int heads, int dk,
+                                 int dv, float* work, long long work_floats, int dtype, cudaStream_t stream) {
+    TI_REQUIRE(num_seqs >= 0 && heads > 0 && dk > 0 && dv > 0, "general_delta_scan: bad sizes");
+    TI_REQUIRE(dk <= 1024, "general_delta_scan: %d key channels a head (at most 1024)", dk);
+    TI_REQUIRE(decay && rate && decay_scale <= 0.f, "general_delta_scan: the decay's and the rate's logits are needed");
+    TI_REQUIRE(num_seqs <= 65535, "general_delta_scan: too many requests");
+    TI_REQUIRE(dtype == TI_F32 || dtype == TI_BF16, "general_delta_scan: unknown dtype %d", dtype);
+    if (num_seqs == 0 || num_tokens == 0) return 0;
+    const size_t t = (size_t)num_tokens, nk = ds_round4(t * heads * dk), nv = ds_round4(t * heads * dv), ns = ds_round4(t * heads);
+    TI_REQUIRE(work && ((uintptr_t)work & 15) == 0, "general_delta_scan: the workspace must be 16-byte aligned");
+    TI_REQUIRE(work_floats >= (long long)(4 * nk + nv + 2 * ns), "general_delta_scan: the workspace is too small");
+    DeltaWork w;
+    w.q = work;
+    w.k = w.q + nk;
+    w.g = w.k + nk;
+    w.a = w.g + nk;
+    w.v = w.a + nk;
+    w.kq = w.v + nv;
+    w.beta = w.kq + ns;
+    GeneralPrepArgs prep = {w, r, k, v, ld_r, r_off, ld_k, k_off, ld_v, v_off, decay, ld_decay, decay_off, rate, ld_rate,
+                            rate_off, decay_b, rate_b, decay_scale, unit_eps, num_tokens, heads, dk, dv};
+    const size_t items = t * heads;
+    const unsigned blocks = (unsigned)((items + DP_THREADS / 32 - 1) / (DP_THREADS / 32));
+    if (dtype == TI_F32) ti_launch(general_delta_prepare_kernel<float>, blocks, DP_THREADS, 0, stream, prep);
+    else ti_launch(general_delta_prepare_kernel<__nv_bfloat16>, blocks, DP_THREADS, 0, stream, prep);
+    TI_CHECK_LAUNCH("general_delta_prepare");
+    return ds_launch_scan<true>(w, y, state, slot_stride, cu_seqlens, state_slots, num_seqs, num_tokens, heads, heads, dk, dv,
+                                stream);
 }

@@ -3,7 +3,8 @@
 //              compute dtype), s = softmax(z) over all experts (or, scoring 1, sigmoid(z) of each expert by itself),
 //              the `top` largest s + correction (a learned number per
 //              expert that only steers the choice; first index on ties), weights s_k / (sum of the chosen + weight_eps)
-//              or, without renormalisation, s_k itself; also counts the tokens of every expert and gives each
+//              or, without renormalisation, s_k itself, times weight_scale; with groups (equal runs of neighbouring
+//              experts) only experts of the `keep` groups whose best score is largest may be chosen; also counts the tokens of every expert and gives each
 //              (token, choice) its rank among them. The last experts of the router may be identity experts, whose
 //              output is the token's row itself: they have no weights, the plan gives them no tiles, and `combine`
 //              adds weight * row for them
@@ -14,7 +15,8 @@
 //              form gathers its rows from the tokens and applies max(v, 0)^2, the down form reads the sorted rows
 //   combine_norm_add : y = sum_k weight_k * down[slot_k] (+ the shared expert's output), in choice order, then the
 //              residual x32 += w * y * rsqrt(mean(y^2) + eps) and its copy in the compute dtype
-//   combine  : the same weighted sum alone, identity experts included, in the compute dtype
+//   combine  : the same weighted sum alone, identity experts included, in the compute dtype; optionally + the shared
+//              expert's output, times the sigmoid of one logit a token (w_sg . row), which the kernel makes itself
 //   clamped_glu : an expert's gated activation on the stored product [gate | up]: g = min(gate, limit),
 //              u = clamp(up, -limit, limit), g * sigmoid(alpha * g) * (u + 1)
 //   silu_glu : silu(gate) * up on the stored product [gate | up]; optionally both halves of a row times the weight of its
@@ -37,8 +39,9 @@ template <typename T, typename XT>
 __global__ void __launch_bounds__(EX_ROUTE_THREADS) moe_route_kernel(
     int* __restrict__ chosen, float* __restrict__ weight, int* __restrict__ rank, int* __restrict__ counts,
     const XT* __restrict__ x32, const T* __restrict__ w_router, int num_tokens, int hidden, int experts, int top,
-    float weight_eps, const float* __restrict__ correction, int renorm, int scoring) {
+    float weight_eps, const float* __restrict__ correction, int renorm, int scoring, int groups, int keep, float weight_scale) {
     __shared__ float logits[32 * EX_PER_LANE];
+    __shared__ int group_kept[32 * EX_PER_LANE];
     ti_grid_launch_dependents();
     ti_grid_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -97,6 +100,47 @@ __global__ void __launch_bounds__(EX_ROUTE_THREADS) moe_route_kernel(
 #pragma unroll
     for (int k = 0; k < EX_PER_LANE; ++k)
         c[k] = s[k] < 0.f ? -INFINITY : (correction ? s[k] + correction[k * 32 + lane] : s[k]);
+    if (groups > 1 && keep < groups) {                 // the experts of the other groups are out of the choice
+        const int per_group = experts / groups;
+#pragma unroll
+        for (int k = 0; k < EX_PER_LANE; ++k)
+            if (k * 32 + lane < experts) logits[k * 32 + lane] = c[k];
+        __syncwarp();
+        float gv[EX_PER_LANE];                         // lane holds groups lane, lane + 32, ...: their best expert
+#pragma unroll
+        for (int k = 0; k < EX_PER_LANE; ++k) {
+            const int g = k * 32 + lane;
+            gv[k] = -INFINITY;
+            if (g < groups) {
+                for (int e = 0; e < per_group; ++e) gv[k] = fmaxf(gv[k], logits[g * per_group + e]);
+                group_kept[g] = 0;
+            }
+        }
+        __syncwarp();
+        for (int n = 0; n < keep; ++n) {
+            float v = -INFINITY;
+            int idx = 0x7fffffff;
+#pragma unroll
+            for (int k = 0; k < EX_PER_LANE; ++k)
+                if (gv[k] > v) { v = gv[k]; idx = k * 32 + lane; }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float ov = __shfl_xor_sync(0xffffffffu, v, o);
+                const int oi = __shfl_xor_sync(0xffffffffu, idx, o);
+                if (ov > v || (ov == v && oi < idx)) { v = ov; idx = oi; }
+            }
+            if (lane == 0 && idx < groups) group_kept[idx] = 1;
+#pragma unroll
+            for (int k = 0; k < EX_PER_LANE; ++k)
+                if (idx == k * 32 + lane) gv[k] = -INFINITY;
+        }
+        __syncwarp();
+#pragma unroll
+        for (int k = 0; k < EX_PER_LANE; ++k) {
+            const int e = k * 32 + lane;
+            if (e < experts && !group_kept[e / per_group]) c[k] = -INFINITY;
+        }
+    }
     float best[EX_MAX_TOP];
     int who[EX_MAX_TOP];
     float total = 0.f;
@@ -121,7 +165,7 @@ __global__ void __launch_bounds__(EX_ROUTE_THREADS) moe_route_kernel(
             if (idx == k * 32 + lane) c[k] = -INFINITY;
     }
     if (lane == 0) {
-        const float norm = renorm ? 1.f / (total + weight_eps) : 1.f;
+        const float norm = (renorm ? 1.f / (total + weight_eps) : 1.f) * weight_scale;
         for (int ch = 0; ch < top; ++ch) {
             chosen[(size_t)t * top + ch] = who[ch];
             weight[(size_t)t * top + ch] = best[ch] * norm;
@@ -170,14 +214,18 @@ __global__ void moe_place_kernel(int* __restrict__ slot_of, int* __restrict__ to
 
 // scoring 0: softmax over the experts; 1: the sigmoid of each logit.
 // slot_weight (float32 [tokens * top], or null): also receives every (token, choice)'s weight at its row in expert order.
+// groups > 1: only experts of the keep_groups best groups can be chosen; weight_scale: a factor on every weight.
 // counts (experts ints) must be zero on entry; the launcher clears them. x_dtype: of the tokens' rows (float32, or
 // the compute dtype of a sublayer's input); correction: float32 [experts] or null; renorm: the weights are divided by
 // their sum; real_experts: how many of the router's outputs are experts with weights (the rest: identity experts).
 TI_API int ti_moe_route(int* chosen, float* weight, int* rank, int* counts, int* starts, int* tiles, int* num_tiles,
                         int* slot_of, int* token_of, const void* x, const void* w_router, int num_tokens, int hidden,
                         int experts, int top, float weight_eps, const float* correction, int renorm, int real_experts,
-                        int tile_rows, int max_tiles, int scoring, float* slot_weight, int x_dtype, int dtype,
-                        cudaStream_t stream) {
+                        int tile_rows, int max_tiles, int scoring, float* slot_weight, int groups, int keep_groups,
+                        float weight_scale, int x_dtype, int dtype, cudaStream_t stream) {
+    TI_REQUIRE(groups >= 1 && experts % groups == 0 && keep_groups >= 1 && keep_groups <= groups &&
+               keep_groups * (experts / groups) >= top, "moe_route: %d of %d groups of %d experts do not hold the %d chosen",
+               keep_groups, groups, groups > 0 ? experts / groups : 0, top);
     TI_REQUIRE(scoring == 0 || scoring == 1, "moe_route: scoring %d is neither the softmax (0) nor the sigmoid (1)", scoring);
     TI_REQUIRE(num_tokens >= 0 && hidden > 0 && experts > 0 && top > 0, "moe_route: bad sizes");
     TI_REQUIRE(top <= EX_MAX_TOP && top <= experts, "moe_route: top %d of %d experts (at most %d)", top, experts, EX_MAX_TOP);
@@ -190,7 +238,7 @@ TI_API int ti_moe_route(int* chosen, float* weight, int* rank, int* counts, int*
     const int blocks = num_tokens;
     typedef __nv_bfloat16 B;
 #define EX_ROUTE(T, XT) ti_launch(moe_route_kernel<T, XT>, blocks, EX_ROUTE_THREADS, 0, stream, chosen, weight, rank, counts, \
-                                  (const XT*)x, (const T*)w_router, num_tokens, hidden, experts, top, weight_eps, correction, renorm, scoring)
+                                  (const XT*)x, (const T*)w_router, num_tokens, hidden, experts, top, weight_eps, correction, renorm, scoring, groups, keep_groups, weight_scale)
     if (dtype == TI_F32) EX_ROUTE(float, float);
     else if (dtype == TI_BF16 && x_dtype == TI_F32) EX_ROUTE(B, float);
     else if (dtype == TI_BF16) EX_ROUTE(B, B);
@@ -487,12 +535,15 @@ TI_API int ti_moe_silu_glu(void* out, const void* in, long long rows, int ff, co
 
 // out[t] = sum_c weight[t][c] * (chosen[t][c] < real_experts ? down[slot_of[t][c]] : x[t]), in choice order, float32
 // sums, one rounding. A block a token. weight may be null: every weight is one (experts weighted at their input).
+// shared_out (compute dtype [T][size], or null) is added, times sigmoid(w_sg . x[t]) where w_sg ([size]) is given.
 template <typename T>
 __global__ void moe_combine_kernel(T* __restrict__ out, const float* __restrict__ down, const T* __restrict__ x,
                                    const int* __restrict__ chosen, const int* __restrict__ slot_of,
-                                   const float* __restrict__ weight, int size, int top, int real_experts) {
+                                   const float* __restrict__ weight, int size, int top, int real_experts,
+                                   const T* __restrict__ shared_out, const T* __restrict__ w_sg) {
     __shared__ int slots[EX_MAX_TOP];
     __shared__ float wts[EX_MAX_TOP];
+    __shared__ float red[33];
     ti_grid_launch_dependents();
     ti_grid_wait();
     const int t = blockIdx.x;
@@ -503,25 +554,33 @@ __global__ void moe_combine_kernel(T* __restrict__ out, const float* __restrict_
     }
     __syncthreads();
     const size_t base = (size_t)t * size;
+    float gate = 1.f;                                  // the shared expert's factor
+    if (shared_out && w_sg) {
+        float dot = 0.f;
+        for (int i = threadIdx.x; i < size; i += blockDim.x) dot = fmaf(to_f32(x[base + i]), to_f32(w_sg[i]), dot);
+        gate = 1.f / (1.f + expf(-block_sum(dot, red)));
+    }
     for (int i = threadIdx.x; i < size; i += blockDim.x) {
         float v = 0.f;
         for (int c = 0; c < top; ++c)
             v = fmaf(wts[c], slots[c] >= 0 ? down[(size_t)slots[c] * size + i] : to_f32(x[base + i]), v);
+        if (shared_out) v = fmaf(gate, to_f32(shared_out[base + i]), v);
         out[base + i] = from_f32<T>(v);
     }
 }
 
 TI_API int ti_moe_combine(void* out, const float* down, const void* x, const int* chosen, const int* slot_of,
-                          const float* weight, int num_tokens, int size, int top, int real_experts, int dtype,
-                          cudaStream_t stream) {
+                          const float* weight, int num_tokens, int size, int top, int real_experts, const void* shared_out,
+                          const void* w_sg, int dtype, cudaStream_t stream) {
     TI_REQUIRE(num_tokens >= 0 && size > 0 && top > 0 && top <= EX_MAX_TOP, "moe_combine: bad sizes");
     if (num_tokens == 0) return 0;
     int threads = 32;
     while (threads < 512 && threads * 4 < size) threads <<= 1;
     if (dtype == TI_F32)
-        ti_launch(moe_combine_kernel<float>, num_tokens, threads, 0, stream, (float*)out, down, (const float*)x, chosen, slot_of, weight, size, top, real_experts);
+        ti_launch(moe_combine_kernel<float>, num_tokens, threads, 0, stream, (float*)out, down, (const float*)x, chosen, slot_of, weight, size, top, real_experts, (const float*)shared_out, (const float*)w_sg);
     else if (dtype == TI_BF16)
-        ti_launch(moe_combine_kernel<__nv_bfloat16>, num_tokens, threads, 0, stream, (__nv_bfloat16*)out, down, (const __nv_bfloat16*)x, chosen, slot_of, weight, size, top, real_experts);
+        ti_launch(moe_combine_kernel<__nv_bfloat16>, num_tokens, threads, 0, stream, (__nv_bfloat16*)out, down, (const __nv_bfloat16*)x, chosen, slot_of, weight, size, top, real_experts,
+                  (const __nv_bfloat16*)shared_out, (const __nv_bfloat16*)w_sg);
     else TI_REQUIRE(false, "moe_combine: unknown dtype %d", dtype);
     TI_CHECK_LAUNCH("moe_combine");
     return 0;

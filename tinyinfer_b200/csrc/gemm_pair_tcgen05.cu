@@ -15,7 +15,7 @@
 //                        (tcgen05.commit with multicast): stage free, accumulator full.
 //   warps 2..5 (both)    epilogue of tile i from one half of tensor memory while the MMAs of tile i+1 fill
 //                        the other: + bias[n], + residual[m,n], float32 output, or the gated form
-//                        out[m,j] = silu(x.w[j]) * (x.w[J+j]) (the even CTA's half of B holds 128 gate rows, the
+//                        out[m,j] = act(x.w[j]) * (x.w[J+j]) (the even CTA's half of B holds 128 gate rows, the
 //                        odd one's the 128 up rows of the same outputs). All on the float32 accumulators,
 //                        one rounding. They tell the even CTA's MMA thread when their half is read.
 //
@@ -40,11 +40,16 @@ struct PairGemmParams {
     const float* bias;
     const __nv_bfloat16* residual;
     int M, N, K;                     // out is [M, N] (gated: N = J, w has 2J rows)
-    int gated, out_f32;
+    int gated, out_f32;              // gated: 0 no, 1 silu, 2 the tanh form of gelu
     int* status;
 };
 
-__device__ __forceinline__ float silu_mul(float g, float u) { return (g / (1.f + __expf(-g))) * u; }
+// act(g) * u. silu(g) = g / (1 + exp(-g)); the tanh form of gelu is the same with another exponent, since
+// (1 + tanh(y)) / 2 = 1 / (1 + exp(-2 y)): y = sqrt(2 / pi) (g + 0.044715 g^3).
+__device__ __forceinline__ float glu_mul(float g, float u, bool gelu) {
+    const float e = gelu ? g * fmaf(0.0713548162726f, g * g, 1.5957691216057308f) : g;
+    return (g / (1.f + __expf(-e))) * u;
+}
 __device__ __forceinline__ uint32_t cluster_rank() {
     uint32_t r;
     asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(r));
@@ -120,6 +125,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constan
     ti_grid_launch_dependents();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const uint32_t rank = cluster_rank();
+    const bool gelu = p.gated == 2;
     const int cols_per_tile = p.gated ? BN / 2 : BN;
     const int row_tiles = (p.M + 2 * BM - 1) / (2 * BM);
     const int col_tiles = (p.N + cols_per_tile - 1) / cols_per_tile;
@@ -336,7 +342,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constan
                     const float* u = reinterpret_cast<const float*>(ru);
                     __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)m * p.N + j0;
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) v[i] = silu_mul(v[i], u[i]);
+                    for (int i = 0; i < 32; ++i) v[i] = glu_mul(v[i], u[i], gelu);
                     if (j0 + 32 <= p.N && (((size_t)m * p.N + j0) & 7) == 0) {
 #pragma unroll
                         for (int h = 0; h < 4; ++h) {
@@ -376,7 +382,7 @@ TI_API int ti_gemm_pair_supported(int M, int N, int K, int gated) {
 }
 
 // y = x . w^T in bfloat16 with float32 accumulation, in the pair form; for steps of many tokens. gated: w is
-// [2N, K] (gate rows, then up rows), out [M, N] = silu(x.gate) * (x.up). out_f32: out is float32.
+// [2N, K] (gate rows, then up rows), out [M, N] = act(x.gate) * (x.up) (gated 1: silu, 2: the tanh form of gelu). out_f32: out is float32.
 // status: device word set if a wait ran out.
 TI_API int ti_gemm_pair_bf16(void* out, const void* x, const void* w, const float* bias, const void* residual,
                              int M, int N, int K, int gated, int out_f32, int* status, cudaStream_t stream) {

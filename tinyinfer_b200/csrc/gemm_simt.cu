@@ -1,14 +1,15 @@
 // y[M,N] = x[M,K] . w[N,K]^T with float32 FMA accumulation in a fixed k order: the true 32-bit
 // matrix product of the engine (no tensor cores, no reduced-precision mode), also the fallback
 // for bfloat16 shapes the tcgen05 kernels refuse. Epilogues: + bias[n], + residual[m,n], or the
-// gated form out[m,j] = silu(x.w[j]) * (x.w[J+j]) on the float32 accumulators
+// gated form out[m,j] = act(x.w[j]) * (x.w[J+j]), act silu or the tanh form of gelu, on the float32 accumulators
 // (tinyinfer/csrc/mlp.cu:116-141; silu(g) = g / (1 + exp(-g)), tinyinfer/csrc/utils.h:76-78).
 // A row's result does not depend on which other rows share its tile.
 #include "common.cuh"
 
 constexpr int GS_BM = 64, GS_BN = 64, GS_BK = 16, GS_THREADS = 256;
 
-template <typename T, typename OutT, bool GATED>
+// GATED: 0 no, 1 silu, 2 the tanh form of gelu.
+template <typename T, typename OutT, int GATED>
 __global__ void __launch_bounds__(GS_THREADS) gemm_simt_kernel(
     OutT* __restrict__ out, const T* __restrict__ x, const T* __restrict__ w,
     const float* __restrict__ bias, const T* __restrict__ residual, int M, int N, int K, int gate_rows) {
@@ -64,8 +65,10 @@ __global__ void __launch_bounds__(GS_THREADS) gemm_simt_kernel(
             const int n = n0 + tx * 4 + j;
             if (n >= N) continue;
             float v = acc[i][j];
-            if constexpr (GATED) {
-                v = (v / (1.f + expf(-v))) * acc2[i][j];
+            if constexpr (GATED != 0) {
+                if constexpr (GATED == 1) v = v / (1.f + expf(-v));
+                else v = 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
+                v *= acc2[i][j];
             } else {
                 if (bias) v += bias[n];
                 if (residual) v += to_f32(residual[(size_t)m * N + n]);
@@ -76,7 +79,7 @@ __global__ void __launch_bounds__(GS_THREADS) gemm_simt_kernel(
 }
 
 // out_f32 != 0: the result is stored as float32 whatever the input dtype (logits).
-// gated != 0: w is [2N, K], rows 0..N-1 the gate and N..2N-1 the up projection; out is [M, N].
+// gated != 0 (1: silu, 2: the tanh form of gelu): w is [2N, K], rows 0..N-1 the gate and N..2N-1 the up projection; out is [M, N].
 TI_API int ti_gemm_simt(void* out, const void* x, const void* w, const float* bias, const void* residual,
                         int M, int N, int K, int gated, int out_f32, int dtype, cudaStream_t stream) {
     TI_REQUIRE(M >= 0 && N > 0 && K > 0, "gemm: bad sizes M=%d N=%d K=%d", M, N, K);
@@ -85,18 +88,22 @@ TI_API int ti_gemm_simt(void* out, const void* x, const void* w, const float* bi
     dim3 grid((N + GS_BN - 1) / GS_BN, (M + GS_BM - 1) / GS_BM);
     TI_REQUIRE(grid.y <= 65535, "gemm: too many rows");
     if (dtype == TI_F32) {
-        if (gated)
-            ti_launch(gemm_simt_kernel<float, float, true>, grid, GS_THREADS, 0, stream, (float*)out, (const float*)x, (const float*)w, nullptr, nullptr, M, N, K, N);
+        if (gated == 2)
+            ti_launch(gemm_simt_kernel<float, float, 2>, grid, GS_THREADS, 0, stream, (float*)out, (const float*)x, (const float*)w, nullptr, nullptr, M, N, K, N);
+        else if (gated)
+            ti_launch(gemm_simt_kernel<float, float, 1>, grid, GS_THREADS, 0, stream, (float*)out, (const float*)x, (const float*)w, nullptr, nullptr, M, N, K, N);
         else
-            ti_launch(gemm_simt_kernel<float, float, false>, grid, GS_THREADS, 0, stream, (float*)out, (const float*)x, (const float*)w, bias, (const float*)residual, M, N, K, 0);
+            ti_launch(gemm_simt_kernel<float, float, 0>, grid, GS_THREADS, 0, stream, (float*)out, (const float*)x, (const float*)w, bias, (const float*)residual, M, N, K, 0);
     } else if (dtype == TI_BF16) {
         typedef __nv_bfloat16 B;
-        if (gated)
-            ti_launch(gemm_simt_kernel<B, B, true>, grid, GS_THREADS, 0, stream, (B*)out, (const B*)x, (const B*)w, nullptr, nullptr, M, N, K, N);
+        if (gated == 2)
+            ti_launch(gemm_simt_kernel<B, B, 2>, grid, GS_THREADS, 0, stream, (B*)out, (const B*)x, (const B*)w, nullptr, nullptr, M, N, K, N);
+        else if (gated)
+            ti_launch(gemm_simt_kernel<B, B, 1>, grid, GS_THREADS, 0, stream, (B*)out, (const B*)x, (const B*)w, nullptr, nullptr, M, N, K, N);
         else if (out_f32)
-            ti_launch(gemm_simt_kernel<B, float, false>, grid, GS_THREADS, 0, stream, (float*)out, (const B*)x, (const B*)w, bias, (const B*)residual, M, N, K, 0);
+            ti_launch(gemm_simt_kernel<B, float, 0>, grid, GS_THREADS, 0, stream, (float*)out, (const B*)x, (const B*)w, bias, (const B*)residual, M, N, K, 0);
         else
-            ti_launch(gemm_simt_kernel<B, B, false>, grid, GS_THREADS, 0, stream, (B*)out, (const B*)x, (const B*)w, bias, (const B*)residual, M, N, K, 0);
+            ti_launch(gemm_simt_kernel<B, B, 0>, grid, GS_THREADS, 0, stream, (B*)out, (const B*)x, (const B*)w, bias, (const B*)residual, M, N, K, 0);
     } else TI_REQUIRE(false, "gemm: unknown dtype %d", dtype);
     TI_CHECK_LAUNCH("gemm_simt");
     return 0;

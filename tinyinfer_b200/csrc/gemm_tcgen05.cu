@@ -15,7 +15,7 @@
 //       loops are cut to fill the SMs; up to 15 tokens the last unit of a tile adds the partial sums
 //       up, from 16 tokens on the units of a tile do so together, each its share of the tokens.
 // Epilogues, all on the float32 accumulators with one rounding: + bias[n], + residual[m,n],
-// float32 output (logits), the gated form out[m,j] = silu(x.w[j]) * (x.w[J+j]) of the
+// float32 output (logits), the gated form out[m,j] = act(x.w[j]) * (x.w[J+j]) (act: silu or tanh-gelu) of the
 // reference's MLP kernel (tinyinfer/csrc/mlp.cu:116-141), and the two halves of an RMSNorm that is
 // spread over the products around it (see GemmParams). A row's result does not depend on
 // which other rows share its tile: every output element is one k loop in a fixed order, or a
@@ -43,7 +43,7 @@ struct GemmParams {
     int M, N, K;            // problem: out is [M, N] (gated: N = J, w has 2J rows)
     int rows_total;         // extent of the rows operand that tiles walk over
     int cols_total;         // extent of the cols operand
-    int gated, out_f32, swap;
+    int gated, out_f32, swap;   // gated: 0 no, 1 silu, 2 the tanh form of gelu
     int splits;             // the k range of a tile is cut into this many work units
     int share_sum;          // weights on the lanes, splits > 1: every unit of a tile adds up its share of the
                             // tokens once all units have arrived (all units run at once), not the last alone
@@ -63,7 +63,12 @@ struct GemmParams {
     int* status;
 };
 
-__device__ __forceinline__ float silu_mul(float g, float u) { return (g / (1.f + __expf(-g))) * u; }
+// act(g) * u. silu(g) = g / (1 + exp(-g)); the tanh form of gelu is the same with another exponent, since
+// (1 + tanh(y)) / 2 = 1 / (1 + exp(-2 y)): y = sqrt(2 / pi) (g + 0.044715 g^3).
+__device__ __forceinline__ float glu_mul(float g, float u, bool gelu) {
+    const float e = gelu ? g * fmaf(0.0713548162726f, g * g, 1.5957691216057308f) : g;
+    return (g / (1.f + __expf(-e))) * u;
+}
 
 // TM: accumulators of 128 rows a tile holds. 1: tiles of 128 x BN with two accumulators in tensor memory,
 // so that the epilogue of a tile overlaps the MMAs of the next. 2 (only with BN = 256, many tokens): tiles of
@@ -111,6 +116,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_c
     ti_grid_launch_dependents();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     // tiles: gated normal tiles hold BN/2 gate and BN/2 up columns; gated swapped tiles 64 + 64 rows
+    const bool gelu = p.gated == 2;
     const int rows_per_tile = (p.gated && SWAP) ? BM / 2 : TM * BM;
     const int cols_per_tile = (p.gated && !SWAP) ? BN / 2 : BN;
     const int row_tiles = (p.rows_total + rows_per_tile - 1) / rows_per_tile;
@@ -393,8 +399,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_c
                                     up.z = __shfl_xor_sync(0xffffffffu, acc[i].z, 16); up.w = __shfl_xor_sync(0xffffffffu, acc[i].w, 16);
                                     if (lane >= 16 || !n_ok || col >= cols_real) continue;
                                     const float sc = row_scale_sh[col];                 // gate and up alike
-                                    __nv_bfloat162 lo2 = __floats2bfloat162_rn(silu_mul(acc[i].x * sc, up.x * sc), silu_mul(acc[i].y * sc, up.y * sc));
-                                    __nv_bfloat162 hi2 = __floats2bfloat162_rn(silu_mul(acc[i].z * sc, up.z * sc), silu_mul(acc[i].w * sc, up.w * sc));
+                                    __nv_bfloat162 lo2 = __floats2bfloat162_rn(glu_mul(acc[i].x * sc, up.x * sc, gelu), glu_mul(acc[i].y * sc, up.y * sc, gelu));
+                                    __nv_bfloat162 hi2 = __floats2bfloat162_rn(glu_mul(acc[i].z * sc, up.z * sc, gelu), glu_mul(acc[i].w * sc, up.w * sc, gelu));
                                     uint2 o2;
                                     o2.x = *reinterpret_cast<uint32_t*>(&lo2);
                                     o2.y = *reinterpret_cast<uint32_t*>(&hi2);
@@ -649,7 +655,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_c
                         if (!row_ok || j0 >= p.N) continue;
                         __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)m * p.N + j0;
 #pragma unroll
-                        for (int i = 0; i < 16; ++i) v[i] = silu_mul(v[i], u[i]);
+                        for (int i = 0; i < 16; ++i) v[i] = glu_mul(v[i], u[i], gelu);
                         if (j0 + 16 <= p.N && (((size_t)m * p.N + j0) & 7) == 0) {
 #pragma unroll
                             for (int h = 0; h < 2; ++h) {
@@ -715,7 +721,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_c
                                     const int m = c0 + c + i;
                                     if (m >= p.M) break;
                                     reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)m * p.N + j] =
-                                        __float2bfloat16_rn(silu_mul(v[i], exch[jj * 17 + i]));
+                                        __float2bfloat16_rn(glu_mul(v[i], exch[jj * 17 + i], gelu));
                                 }
                             }
                         }
@@ -795,7 +801,7 @@ int launch(const CUtensorMap& rows_map, const CUtensorMap& cols_map, const GemmP
 TI_API int ti_gemm_bf16_supported(int M, int N, int K) { return (M > 0 && N > 0 && K > 0 && K % 8 == 0) ? 1 : 0; }
 
 // y = x . w^T in bfloat16 with float32 accumulation. gated: w is [2N, K] (gate rows, then up rows),
-// out [M, N] = silu(x.gate) * (x.up). out_f32: out is float32. status: device word set if a wait ran out.
+// out [M, N] = act(x.gate) * (x.up), act being silu (gated 1) or the tanh form of gelu (gated 2). out_f32: out is float32. status: device word set if a wait ran out.
 // workspace / counters: float32 scratch and zeroed int32 words for the split-k path of small M (may be
 // null: then no tile is split). Calls that share them must be ordered on one stream.
 struct NormLink {                  // an RMSNorm spread over two products (see GemmParams)

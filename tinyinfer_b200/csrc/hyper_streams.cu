@@ -11,6 +11,7 @@
 //   streams_step  : as above; `rows` picks the tokens to work on (the rows whose logits are wanted)
 //   gelu, scale   : the feed-forward's activation on a stored tensor, and a constant factor on float32 logits
 //   soft_cap      : x <- cap * tanh(x / cap) on float32 logits
+//   tanh_rows     : the tanh of some columns of float32 rows, rounded once to the compute dtype
 #include "common.cuh"
 
 constexpr int HS_MAX_STREAMS = 8;
@@ -285,5 +286,28 @@ TI_API int ti_soft_cap(float* x, long long n, float cap, cudaStream_t stream) {
     const long long want = (n + 255) / 256;
     ti_launch(soft_cap_kernel, (int)(want < 148 * 16 ? want : 148 * 16), 256, 0, stream, x, (size_t)n, cap, 1.f / cap);
     TI_CHECK_LAUNCH("soft_cap");
+    return 0;
+}
+
+template <typename T>
+__global__ void tanh_rows_kernel(T* __restrict__ out, const float* __restrict__ in, int ld_in, int in_off, int cols, size_t n) {
+    ti_grid_launch_dependents();
+    ti_grid_wait();
+    const size_t stride = (size_t)gridDim.x * blockDim.x;
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += stride)
+        out[i] = from_f32<T>(tanhf(in[(i / cols) * ld_in + in_off + i % cols]));
+}
+
+// out [rows][cols] = tanh of columns [in_off, in_off + cols) of the float32 rows `in` (ld_in floats apart).
+TI_API int ti_tanh_rows(void* out, const float* in, int ld_in, int in_off, int rows, int cols, int dtype, cudaStream_t stream) {
+    TI_REQUIRE(rows >= 0 && cols > 0 && in_off >= 0 && ld_in >= in_off + cols, "tanh_rows: bad sizes");
+    if (rows == 0) return 0;
+    const size_t n = (size_t)rows * cols;
+    const size_t want = (n + 127) / 128;
+    const int blocks = (int)(want < 148 * 16 ? want : 148 * 16);
+    if (dtype == TI_F32) ti_launch(tanh_rows_kernel<float>, blocks, 128, 0, stream, (float*)out, in, ld_in, in_off, cols, n);
+    else if (dtype == TI_BF16) ti_launch(tanh_rows_kernel<__nv_bfloat16>, blocks, 128, 0, stream, (__nv_bfloat16*)out, in, ld_in, in_off, cols, n);
+    else TI_REQUIRE(false, "tanh_rows: unknown dtype %d", dtype);
+    TI_CHECK_LAUNCH("tanh_rows");
     return 0;
 }

@@ -42,7 +42,7 @@ class ModelRunner:
         self.cuda_graphs = (cuda_graphs and self.device.type == "cuda"
                             and all(b.mixer.graph_safe and (b.feed_forward is None or b.feed_forward.graph_safe)
                                     for b in model.blocks))
-        self._tables_only_grow = all(g.need.window is None for g in self.manager.groups)
+        self._tables_only_grow = all(g.need.keeps_all for g in self.manager.groups)
         self._graphs = {}          # requests in the step -> (graph, static logits, kernels)
         self._graph_pool = None
         self.graph_replays = 0

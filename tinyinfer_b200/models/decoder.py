@@ -29,6 +29,7 @@ class DecoderModel:
         self.final_norm = build_norm(spec.final_norm, dtype, self.device)
         self.embedding: Optional[torch.Tensor] = None
         self.head: Optional[torch.Tensor] = None
+        self.step_vectors: Optional[torch.Tensor] = None      # float32 [rows, hidden]: what entries of the run order add
 
     # ------------------------------------------------------------------ tensors
     def _part_prefixes(self, i: int):
@@ -51,6 +52,8 @@ class DecoderModel:
             for prefix, part in self._part_prefixes(i):
                 for local, ts in part.tensors().items():
                     out[prefix + local] = ts
+        if spec.step_vectors:
+            out[spec.step_vectors[0]] = TensorSpec((spec.step_vectors[1], spec.hidden_size), role="vector32")
         for local, ts in self.final_norm.tensors().items():
             out[spec.names.final_norm + local] = ts
         if not spec.tie_embeddings:
@@ -73,6 +76,8 @@ class DecoderModel:
         for i in range(len(self.blocks)):
             for prefix, part in self._part_prefixes(i):
                 part.load({local: tensors[prefix + local] for local in part.tensors()})
+        if spec.step_vectors:
+            self.step_vectors = tensors[spec.step_vectors[0]].contiguous()
         self.final_norm.load({local: tensors[spec.names.final_norm + local]
                               for local in self.final_norm.tensors()})
         self.head = self.embedding if spec.tie_embeddings else tensors[spec.names.head].contiguous()
@@ -94,7 +99,7 @@ class DecoderModel:
         for step in self.spec.execution:
             if step.writes_cache:
                 mixer = self.blocks[step.layer].mixer
-                needs[step.cache] = (mixer.cache_need(), mixer.state_need())
+                needs[step.cache] = (mixer.cache_need(), self.blocks[step.layer].state_need())
         return needs
 
     # ------------------------------------------------------------------ forward
@@ -118,9 +123,15 @@ class DecoderModel:
         link = None        # what a block's last product leaves for the next block's first norm (see parts.base)
         order = self.spec.execution
         for i, entry in enumerate(order):
+            if entry.adds_embedding or entry.adds_vector is not None:
+                x, link = self.enter(x, entry), None
             after = self.blocks[order[i + 1].layer].mixer_norm if i + 1 < len(order) else None
             x, link = self.blocks[entry.layer].forward_linked(x, link, after, step, step.cache_view(entry))
         return x
+
+    def enter(self, x, entry):
+        """What an entry of the run order adds to the residual right before its layer."""
+        raise NotImplementedError(f"{type(self).__name__} has no residual that an entry of the run order could add to")
 
     def logits(self, x: torch.Tensor, step) -> torch.Tensor:
         """Float32 logits [N, V] of the rows ``step.logit_rows`` (there is at least one) of the last
@@ -154,3 +165,41 @@ class StreamDecoderModel(DecoderModel):
         h = ops.streams_step(stream, pending, self._one, rms[0], rms[1], self.dtype, rows=step.logit_rows)
         z = ops.linear(h, self.head, out_float32=True)
         return ops.soft_cap_(z, self.logit_softcap) if self.logit_softcap else z
+
+
+class ScaledResidualDecoderModel(DecoderModel):
+    """The frame of the decoders whose blocks are 'scaled_residual' blocks: the embedding times a constant starts one
+    float32 stream [T, width]; what travels between the blocks is the pair (stream, update still to be applied). Entries of
+    the run order may add the embedding's output and a row of the step vectors before their layer; both ride in the update.
+    At the end the last update, the final norm and the choice of the wanted rows are one kernel, then the head."""
+
+    def __init__(self, spec: ModelSpec, dtype, device, *, embedding_scale: float = 1.0):
+        super().__init__(spec, dtype, device)
+        self.embedding_scale = float(embedding_scale)
+        self._needs_start = any(e.adds_embedding for e in spec.execution)
+        self._start = None
+
+    def embed(self, step):
+        # the stream is updated in place: where later entries add what it started from, the kernel makes a second copy
+        copies = ops.streams_embed(step.token_ids, self.embedding, 2 if self._needs_start else 1, self.embedding_scale)
+        self._start = copies[1] if self._needs_start else None
+        return copies[0], None
+
+    def run_blocks(self, x, step):
+        try:
+            return super().run_blocks(x, step)
+        finally:
+            self._start = None
+
+    def enter(self, x, entry):
+        stream, pending = x
+        pending = pending if pending is not None else ops.ResidualUpdate()
+        pending.add_rows = self._start if entry.adds_embedding else None
+        pending.add_vec = self.step_vectors[entry.adds_vector] if entry.adds_vector is not None else None
+        return stream, pending
+
+    def logits(self, x, step):
+        stream, pending = x
+        rms = self.final_norm.as_rms()
+        _, h = ops.residual_step(stream, pending, rms[0], rms[1], self.dtype, rows=step.logit_rows)
+        return ops.linear(h, self.head, out_float32=True)

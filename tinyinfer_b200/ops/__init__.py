@@ -75,7 +75,7 @@ _SIGNATURES = {
     "experts": {
         "ti_moe_route": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                          c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
-                         c_int, c_void_p],
+                         c_int, c_float, c_int, c_int, c_void_p],
         "ti_moe_tile_rows": [],
         "ti_moe_gemm": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                         c_void_p],
@@ -85,8 +85,8 @@ _SIGNATURES = {
         "ti_moe_combine_norm_add": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                     c_int, c_float, c_int, c_void_p],
         "ti_moe_clamped_glu": [c_void_p, c_void_p, c_ll, c_int, c_float, c_float, c_int, c_void_p],
-        "ti_moe_combine": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                           c_void_p],
+        "ti_moe_combine": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p,
+                           c_void_p, c_int, c_void_p],
     },
     # parts of designs with several residual streams, short convolutions, attention over [key | value] rows and
     # linear attention with a matrix state
@@ -101,6 +101,17 @@ _SIGNATURES = {
                           c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_ll, c_int, c_void_p],
         "ti_streams_step": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int,
                             c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p],
+        "ti_stream_step": [c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_float, c_void_p,
+                           c_void_p, c_int, c_void_p, c_void_p, c_ll, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                           c_void_p],
+        "ti_qkv_prepare": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_ll, c_int, c_int, c_int,
+                           c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p,
+                           c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
+                           c_void_p],
+        "ti_tanh_rows": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
+        "ti_general_delta_scan": [c_void_p, c_void_p, c_ll, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_int,
+                                  c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_float, c_float,
+                                  c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_ll, c_int, c_void_p],
         "ti_gelu": [c_void_p, c_void_p, c_ll, c_int, c_int, c_void_p],
         "ti_scale": [c_void_p, c_ll, c_float, c_void_p],
         "ti_short_conv": [c_void_p, c_void_p, c_int, c_int, c_void_p, c_ll, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
@@ -438,11 +449,17 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
     return (out, None) if wants_link else out
 
 
+GATED_ACTIVATIONS = {"silu": 1, "gelu_tanh": 2}
+
+
 def gated_linear(x: torch.Tensor, w_gate_up: torch.Tensor, *, link: Optional[NormLink] = None,
-                 link_eps: float = 0.0) -> torch.Tensor:
-    """silu(x.Wg^T) * (x.Wu^T) with ``w_gate_up`` = [Wg; Wu] of shape [2I, K] -> [M, I]; the
-    activation and the product act on the float32 accumulators, one rounding. ``link``: as in
+                 link_eps: float = 0.0, activation: str = "silu") -> torch.Tensor:
+    """act(x.Wg^T) * (x.Wu^T) with ``w_gate_up`` = [Wg; Wu] of shape [2I, K] -> [M, I]; the
+    activation ('silu' or 'gelu_tanh') and the product act on the float32 accumulators, one rounding. ``link``: as in
     ``linear`` (both halves are scaled before the activation)."""
+    if activation not in GATED_ACTIVATIONS:
+        raise KernelError(f"gated_linear: unknown activation {activation!r}; known: {sorted(GATED_ACTIVATIONS)}")
+    act = GATED_ACTIVATIONS[activation]
     _check(x, "x", None, 2)
     _check(w_gate_up, "w_gate_up", x.dtype, 2)
     m, k = x.shape
@@ -453,20 +470,20 @@ def gated_linear(x: torch.Tensor, w_gate_up: torch.Tensor, *, link: Optional[Nor
     if link is not None:
         if not (_tensor_core_ok(x, w_gate_up) and norm_link_ok(x)):
             raise KernelError("gated_linear: a norm link needs the tensor-core product of at most 64 rows")
-        _gemm_linked(out, x, w_gate_up, None, None, m, inter, k, 1, (link, link_eps), None)
+        _gemm_linked(out, x, w_gate_up, None, None, m, inter, k, act, (link, link_eps), None)
         return out
     if _tensor_core_ok(x, w_gate_up) and m >= PAIR_MIN_TOKENS and inter >= 128:
         _run("sm100", "ti_gemm_pair_bf16", out.data_ptr(), x.data_ptr(), w_gate_up.data_ptr(), None, None,
-             m, inter, k, 1, 0, kernel_status(x.device).data_ptr(), _stream())
+             m, inter, k, act, 0, kernel_status(x.device).data_ptr(), _stream())
         return out
     if _tensor_core_ok(x, w_gate_up):
         ws, counters = _gemm_scratch(x.device)
         _run("sm100", "ti_gemm_bf16", out.data_ptr(), x.data_ptr(), w_gate_up.data_ptr(), None, None,
-             m, inter, k, 1, 0, ws.data_ptr(), ws.numel(), counters.data_ptr(), counters.numel(),
+             m, inter, k, act, 0, ws.data_ptr(), ws.numel(), counters.data_ptr(), counters.numel(),
              kernel_status(x.device).data_ptr(), _stream())
         return out
     _run("core", "ti_gemm_simt", out.data_ptr(), x.data_ptr(), w_gate_up.data_ptr(), None, None,
-         m, inter, k, 1, 0, _dtype_code(x), _stream())
+         m, inter, k, act, 0, _dtype_code(x), _stream())
     return out
 
 
@@ -637,14 +654,25 @@ def release_scratch(device) -> None:
     _sample_scratch.pop(key, None)
 
 
+def _mask_code(window: Optional[int], chunk: Optional[int]) -> int:
+    """How the kernels take what a query may see: n > 0: the last n keys; -n: the keys of its own chunk of n positions
+    (chunks counted from position 0 of the request); 0: all."""
+    if window and chunk:
+        raise KernelError("attention: a window or chunks, not both")
+    if (window is not None and window < 0) or (chunk is not None and chunk < 0):
+        raise KernelError("attention: a window and a chunk have at least one position")
+    return int(window or 0) or -int(chunk or 0)
+
+
 def paged_attention(q: torch.Tensor, kv_cache: torch.Tensor, *, positions: torch.Tensor,
                     token_seq: torch.Tensor, block_table: torch.Tensor, scale: float,
-                    window: Optional[int] = None, step=None,
+                    window: Optional[int] = None, chunk: Optional[int] = None, step=None,
                     status: Optional[torch.Tensor] = None, sink: Optional[float] = None,
                     out_scale: float = 1.0, head_sinks: Optional[torch.Tensor] = None,
                     gate: Optional[torch.Tensor] = None, gate_offset: int = 0, softcap: float = 0.0) -> torch.Tensor:
     """Causal attention of q [T, Hq, D] over the pages of each token's own request.
-    Token t sees keys max(0, pos - window + 1) .. pos of request ``token_seq[t]``.
+    Token t sees keys max(0, pos - window + 1) .. pos of request ``token_seq[t]``, or, with ``chunk``, those from
+    floor(pos / chunk) * chunk on.
     ``sink``: a logit whose exponential joins every softmax denominator without a value (0.0 adds one to the sum
     of exp(score)); ``head_sinks`` float32 [Hq]: such a logit per query head instead; ``gate`` [T, cols] of q's dtype:
     the output of (token, head) is multiplied by sigmoid(gate[token, gate_offset + head]); ``out_scale``: a factor on
@@ -663,6 +691,7 @@ def paged_attention(q: torch.Tensor, kv_cache: torch.Tensor, *, positions: torch
     out = torch.empty((t, hq * d), dtype=q.dtype, device=q.device)
     if t == 0:
         return out
+    mask = _mask_code(window, chunk)
     has_sink, sink_v = int(sink is not None), float(sink or 0.0)
     _check_head_extras(q, head_sinks, gate, gate_offset)
     extras = (_ptr(head_sinks), _ptr(gate), gate.shape[1] if gate is not None else 0, int(gate_offset), float(softcap or 0.0))
@@ -671,11 +700,11 @@ def paged_attention(q: torch.Tensor, kv_cache: torch.Tensor, *, positions: torch
             _warn_generic_attention(hq, hkv, d, page_size)
         if softcap or has_sink or out_scale != 1.0 or head_sinks is not None or gate is not None:
             return attention_rows(q, kv_cache, v_dim=d, positions=positions, token_seq=token_seq, block_table=block_table,
-                                  scale=scale, sink=sink, window=window, out_scale=out_scale, status=status,
+                                  scale=scale, sink=sink, window=window, chunk=chunk, out_scale=out_scale, status=status,
                                   head_sinks=head_sinks, gate=gate, gate_offset=gate_offset, softcap=softcap)
         _run("core", "ti_attention_generic", out.data_ptr(), q.data_ptr(), kv_cache.data_ptr(),
              positions.data_ptr(), token_seq.data_ptr(), block_table.data_ptr(), block_table.shape[1],
-             t, hq, hkv, d, page_size, num_pages, float(scale), int(window or 0), _ptr(status),
+             t, hq, hkv, d, page_size, num_pages, float(scale), mask, _ptr(status),
              _dtype_code(q), _stream())
         return out
     if step is not None:
@@ -704,11 +733,11 @@ def paged_attention(q: torch.Tensor, kv_cache: torch.Tensor, *, positions: torch
         num_decode, num_tiles, max_context = len(rows_l), len(tiles_l) // 4, max(pos_h) + 1
     kstatus = kernel_status(q.device).data_ptr()
     if num_decode:
-        scratch = _decode_scratch(q.device, decode_scratch_floats(num_decode, hq, hkv, d, max_context, int(window or 0)))
+        scratch = _decode_scratch(q.device, decode_scratch_floats(num_decode, hq, hkv, d, max_context, mask))
         _run("sm100", "ti_attention_decode_sink_bf16", out.data_ptr(), q.data_ptr(), kv_cache.data_ptr(),
              scratch.data_ptr(), scratch.numel(), decode_rows.data_ptr(), num_decode, positions.data_ptr(),
              token_seq.data_ptr(), block_table.data_ptr(), block_table.shape[1], hq, hkv, d, page_size,
-             num_pages, float(scale), int(window or 0), int(max_context), has_sink, sink_v, float(out_scale), *extras,
+             num_pages, float(scale), mask, int(max_context), has_sink, sink_v, float(out_scale), *extras,
              kstatus, _stream())
     def one_tile_kernel(first: int, count: int, halves: int) -> None:
         # Few query tiles behind a long prefix: the keys are shared out over CTAs too (at least 1,024 to a CTA),
@@ -724,13 +753,13 @@ def paged_attention(q: torch.Tensor, kv_cache: torch.Tensor, *, positions: torch
             scratch_ptr, scratch_floats = scratch.data_ptr(), scratch.numel()
         _run("sm100", "ti_attention_prefill_tc_sink_bf16", out.data_ptr(), q.data_ptr(), kv_cache.data_ptr(),
              tiles.data_ptr() + 16 * first, count, t, block_table.data_ptr(), block_table.shape[1], hq, hkv, d, page_size,
-             num_pages, float(scale), int(window or 0), halves, splits, split_keys, scratch_ptr, scratch_floats, has_sink,
+             num_pages, float(scale), mask, halves, splits, split_keys, scratch_ptr, scratch_floats, has_sink,
              sink_v, float(out_scale), *extras, kstatus, _stream())
 
     if num_pairs * hq >= PAIR_MIN_CTAS:             # two query tiles a CTA
         _run("sm100", "ti_attention_prefill_pair_sink_bf16", out.data_ptr(), q.data_ptr(), kv_cache.data_ptr(),
              tiles.data_ptr(), num_pairs, t, block_table.data_ptr(), block_table.shape[1], hq, hkv, d, page_size,
-             num_pages, float(scale), int(window or 0), has_sink, sink_v, float(out_scale), *extras, kstatus, _stream())
+             num_pages, float(scale), mask, has_sink, sink_v, float(out_scale), *extras, kstatus, _stream())
     elif num_pairs:                                 # too few of them to fill the machine: one query tile a CTA
         one_tile_kernel(0, num_pairs, 1)
     if num_tiles > num_pairs:                       # ends of portions of at most 128 rows
@@ -1019,14 +1048,17 @@ class ExpertRouting:
 
 def route_experts(x32: torch.Tensor, w_router: torch.Tensor, top: int, weight_eps: float,
                   wide_tiles: bool = False, tile_rows: int = 0, *, correction: Optional[torch.Tensor] = None,
-                  renormalize: bool = True, real_experts: Optional[int] = None, scoring: str = "softmax") -> ExpertRouting:
+                  renormalize: bool = True, real_experts: Optional[int] = None, scoring: str = "softmax",
+                  groups: int = 1, keep_groups: int = 1, weight_scale: float = 1.0) -> ExpertRouting:
     """Router of a mixture of experts: float32 logits from the rows ``x32`` [T, H] (float32, or the router's dtype)
     and ``w_router`` [E, H], softmax over all experts, the ``top`` largest (first index on ties), weights = their
     scores over their sum (+ ``weight_eps``). ``correction`` float32 [E]: the choice goes by score + correction, the
     weights stay the plain scores; ``renormalize`` False: the weights are the scores themselves; ``real_experts``:
     only the first so many router outputs are experts with weights, the rest stand for identity experts (rows, but
     no tiles in the plan). ``scoring`` 'sigmoid': an expert's score is the sigmoid of its own logit instead of the
-    softmax over all. ``wide_tiles``: the row tiles of the plan hold 64 rows instead of 32 (for steps that bring
+    softmax over all. ``groups`` > 1: the experts form that many equal groups of neighbours, and only experts of the
+    ``keep_groups`` groups whose best expert ranks highest can be chosen; ``weight_scale``: a factor on every weight.
+    ``wide_tiles``: the row tiles of the plan hold 64 rows instead of 32 (for steps that bring
     an expert many rows; only the tensor-core grouped product takes them, see ``expert_tiles_may_be_wide``);
     ``tile_rows``: any other height the caller has settled with the grouped product (``expert_tile_rows``)."""
     _check(x32, "x32", None, 2)
@@ -1059,7 +1091,8 @@ def route_experts(x32: torch.Tensor, w_router: torch.Tensor, top: int, weight_ep
     _run("experts", "ti_moe_route", chosen.data_ptr(), weight.data_ptr(), rank.data_ptr(), counts.data_ptr(),
          starts.data_ptr(), tiles.data_ptr(), num_tiles.data_ptr(), slot_of.data_ptr(), token_of.data_ptr(),
          x32.data_ptr(), w_router.data_ptr(), t, hidden, experts, top, float(weight_eps), _ptr(correction),
-         int(renormalize), real, tile_rows, max_tiles, int(scoring == "sigmoid"), slot_weight.data_ptr(), _dtype_code(x32),
+         int(renormalize), real, tile_rows, max_tiles, int(scoring == "sigmoid"), slot_weight.data_ptr(), int(groups),
+         int(keep_groups), float(weight_scale), _dtype_code(x32),
          _dtype_code(w_router), _stream())
     return ExpertRouting(chosen.view(t, top), weight, slot_of.view(t, top), token_of, tiles.view(max_tiles, 3),
                          num_tiles, max_tiles, counts, tile_rows, slot_weight)
@@ -1167,12 +1200,22 @@ def silu_glu(gate_up: torch.Tensor, row_scale: Optional[torch.Tensor] = None) ->
 
 
 def experts_combine(down: torch.Tensor, x: torch.Tensor, routing: ExpertRouting, real_experts: int,
-                    weighted: bool = True) -> torch.Tensor:
+                    weighted: bool = True, shared: Optional[torch.Tensor] = None,
+                    shared_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """out[t] = sum_c weight[t, c] * (down[slot_of[t, c]] if chosen[t, c] < real_experts else x[t]) in choice order:
     the weighted sum of the chosen experts' outputs (float32 sorted rows ``down``), an identity expert's output being
     the token's own row of ``x`` [T, H]. Float32 sums, one rounding to x's dtype. ``weighted`` False: every weight is
-    one (the experts were weighted at their input)."""
+    one (the experts were weighted at their input). ``shared`` [T, H]: a shared expert's output, added to the sum, times
+    sigmoid(shared_gate . x[t]) where ``shared_gate`` [H] is given."""
     _check(down, "down", torch.float32, 2)
+    if shared is not None:
+        _check(shared, "shared", x.dtype, 2)
+        if shared.shape != x.shape:
+            raise KernelError("experts_combine: the shared expert's rows do not fit the tokens'")
+    if shared_gate is not None:
+        _check(shared_gate, "shared_gate", x.dtype, 1)
+        if shared is None or shared_gate.shape[0] != x.shape[1]:
+            raise KernelError("experts_combine: the gate belongs to a shared expert and has a number per feature")
     _check(x, "x", None, 2)
     t, size = x.shape
     if down.shape[1] != size or routing.chosen.shape[0] != t:
@@ -1180,7 +1223,7 @@ def experts_combine(down: torch.Tensor, x: torch.Tensor, routing: ExpertRouting,
     out = torch.empty_like(x)
     _run("experts", "ti_moe_combine", out.data_ptr(), down.data_ptr(), x.data_ptr(), routing.chosen.data_ptr(),
          routing.slot_of.data_ptr(), routing.weight.data_ptr() if weighted else None, t, size, routing.chosen.shape[1],
-         int(real_experts), _dtype_code(x), _stream())
+         int(real_experts), _ptr(shared), _ptr(shared_gate), _dtype_code(x), _stream())
     return out
 
 
@@ -1239,6 +1282,64 @@ def streams_step(x: torch.Tensor, pending: Optional[StreamUpdate], read_in: Opti
          width, s, _dtype_code(y) if y is not None else 0, _dtype_code(h) if h is not None else 0,
          _ptr(pending.norm_weight) if pending else None, pending.norm_eps if pending else 0.0, _stream())
     return h
+
+
+class ResidualUpdate:
+    """What lies between two sublayers of a decoder with one float32 residual stream x [T, W], applied by the next
+    ``residual_step``: x <- x + factor * (scale * y), ``scale`` float32 [W] or None; then x <- x + add_rows + add_vec
+    (float32 [T, W] and [W], or None)."""
+
+    def __init__(self, y: Optional[torch.Tensor] = None, scale: Optional[torch.Tensor] = None, factor: float = 1.0,
+                 add_rows: Optional[torch.Tensor] = None, add_vec: Optional[torch.Tensor] = None):
+        self.y, self.scale, self.factor, self.add_rows, self.add_vec = y, scale, float(factor), add_rows, add_vec
+
+
+def residual_step(x: torch.Tensor, pending: Optional[ResidualUpdate], norm_weight: torch.Tensor, eps: float,
+                  out_dtype: torch.dtype, *, shift: Optional[torch.Tensor] = None, previous: Optional[torch.Tensor] = None,
+                  step=None, rows: Optional[torch.Tensor] = None, keep: bool = True):
+    """One kernel between two sublayers: the pending update, then h = norm_weight * x * rsqrt(mean(x^2) + eps) in
+    ``out_dtype``, then, with ``shift`` float32 [W], the token shift h_t + (h_(t-1) - h_t) * shift, where the h before a
+    request's first token of the step comes from ``previous`` (float32 [slots, W], its state slot), which then takes the h
+    of its last; ``step`` is the StepContext. Returns (x updated, h). Without a shift x is updated in place; with one (the
+    token before may be worked on by another block) into a new tensor, ``x`` itself staying as it was. ``rows`` int32
+    [N]: h of these tokens only, x is not updated. ``keep`` False: the updated x is not needed any more."""
+    _check(x, "x", torch.float32, 2)
+    t, width = x.shape
+    _check(norm_weight, "norm_weight", torch.float32, 1)
+    p = pending if pending is not None else ResidualUpdate()
+    for name, ten, shape, dtype in (("y", p.y, (t, width), None), ("scale", p.scale, (width,), torch.float32),
+                                    ("add_rows", p.add_rows, (t, width), torch.float32),
+                                    ("add_vec", p.add_vec, (width,), torch.float32), ("shift", shift, (width,), torch.float32),
+                                    ("norm_weight", norm_weight, (width,), torch.float32)):
+        if ten is not None and tuple(_check(ten, name, dtype).shape) != shape:
+            raise KernelError(f"residual_step: {name} has shape {tuple(ten.shape)}, not {shape}")
+    n = t if rows is None else _check(rows, "rows", torch.int32, 1).shape[0]
+    h = torch.empty((n, width), dtype=out_dtype, device=x.device)
+    changes = p.y is not None or p.add_rows is not None or p.add_vec is not None
+    fresh, stride = x, 0
+    if shift is not None:
+        if rows is not None or previous is None or step is None:
+            raise KernelError("residual_step: a token shift works on a whole step and needs the requests' state")
+        stride = _slot_stride(previous, width, "previous")
+        fresh = torch.empty_like(x) if changes and keep else x
+    stored = fresh.data_ptr() if changes and keep and rows is None else None
+    _run("hybrid", "ti_stream_step", x.data_ptr(), stored, _ptr(p.y), _ptr(p.scale), p.factor, _ptr(p.add_rows), _ptr(p.add_vec),
+         norm_weight.data_ptr(), float(eps), h.data_ptr(), _ptr(rows), n, _ptr(shift),
+         previous.data_ptr() if shift is not None else None, stride, _ptr(step.token_seq) if shift is not None else None,
+         _ptr(step.cu_seqlens) if shift is not None else None, _ptr(step.state_slots) if shift is not None else None, t, width,
+         _dtype_code(p.y) if p.y is not None else _dtype_code(h), _dtype_code(h), _stream())
+    return fresh, h
+
+
+def tanh_rows(x: torch.Tensor, offset: int, cols: int, out_dtype: torch.dtype) -> torch.Tensor:
+    """tanh of columns [offset, offset + cols) of the float32 rows ``x``, rounded once to ``out_dtype``."""
+    _check(x, "x", torch.float32, 2)
+    if offset < 0 or offset + cols > x.shape[1]:
+        raise KernelError("tanh_rows: the columns do not fit the rows")
+    out = torch.empty((x.shape[0], cols), dtype=out_dtype, device=x.device)
+    _run("hybrid", "ti_tanh_rows", out.data_ptr(), x.data_ptr(), x.shape[1], int(offset), x.shape[0], int(cols),
+         _dtype_code(out), _stream())
+    return out
 
 
 def gelu(x: torch.Tensor, tanh: bool = False, out: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -1379,7 +1480,7 @@ def _check_head_extras(q, head_sinks, gate, gate_offset) -> None:
 
 def attention_rows(q: torch.Tensor, cache: torch.Tensor, *, v_dim: int, positions: torch.Tensor, token_seq: torch.Tensor,
                    block_table: torch.Tensor, scale: float, sink: Optional[float] = None, window: Optional[int] = None,
-                   out_scale: float = 1.0, step=None, status: Optional[torch.Tensor] = None,
+                   chunk: Optional[int] = None, out_scale: float = 1.0, step=None, status: Optional[torch.Tensor] = None,
                    head_sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
                    gate_offset: int = 0, softcap: float = 0.0) -> torch.Tensor:
     """Causal attention of q [T, Hq, d] over pages whose rows are [k (d) | v (dv)] (``cache``
@@ -1387,7 +1488,7 @@ def attention_rows(q: torch.Tensor, cache: torch.Tensor, *, v_dim: int, position
     value (0.0: one is added to the sum of exp(score)); ``head_sinks`` float32 [Hq]: such a logit per query head
     instead. ``gate`` [T, cols] of q's dtype: the output of (token, head) is also multiplied by
     sigmoid(gate[token, gate_offset + head]). ``softcap`` > 0: a score s becomes softcap * tanh(s / softcap) before the
-    softmax. Returns [T, Hq * dv], multiplied by ``out_scale`` before its rounding."""
+    softmax. ``window``, ``chunk``: as in ``paged_attention``. Returns [T, Hq * dv], multiplied by ``out_scale`` before its rounding."""
     _check(q, "q", None, 3)
     _check(cache, "cache", q.dtype, 5)
     _check(positions, "positions", torch.int32, 1)
@@ -1402,7 +1503,7 @@ def attention_rows(q: torch.Tensor, cache: torch.Tensor, *, v_dim: int, position
     _check_head_extras(q, head_sinks, gate, gate_offset)
     _run("hybrid", "ti_attention_rows", out.data_ptr(), q.data_ptr(), cache.data_ptr(), positions.data_ptr(),
          token_seq.data_ptr(), block_table.data_ptr(), block_table.shape[1], t, hq, hkv, d, v_dim, page_size, num_pages,
-         planes, float(scale), int(window or 0), int(sink is not None), float(sink or 0.0), _ptr(head_sinks), _ptr(gate),
+         planes, float(scale), _mask_code(window, chunk), int(sink is not None), float(sink or 0.0), _ptr(head_sinks), _ptr(gate),
          gate.shape[1] if gate is not None else 0, int(gate_offset), float(out_scale), float(softcap or 0.0), _ptr(status),
          _dtype_code(q), _stream())
     return out
@@ -1576,6 +1677,98 @@ def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay_logits: 
              decay_logits.shape[1], int(decay_offset), beta_logits.data_ptr(), beta_logits.shape[1], int(beta_offset),
              a_log.data_ptr(), _ptr(dt_bias), float(q_scale), float(unit_eps), cu_seqlens.data_ptr(), state_slots.data_ptr(),
              int(num_seqs), t, heads, groups, key_dim, value_dim, work.data_ptr(), work.numel(), _dtype_code(q), _stream())
+    return out
+
+
+QKV_NORMS = {None: 0, "rows": 1, "head": 2, "head_after": 3}
+
+
+def qkv_prepare(qkv: torch.Tensor, *, num_heads: int, num_kv_heads: int, head_dim: int, v_dim: int, cache: torch.Tensor,
+                block_table: torch.Tensor, positions: torch.Tensor, token_seq: torch.Tensor, cu_seqlens: torch.Tensor,
+                state_slots: torch.Tensor, rotation: Optional[Rotation] = None, conv_weight: Optional[torch.Tensor] = None,
+                history: Optional[torch.Tensor] = None, shift_history: bool = False, norm: Optional[str] = None,
+                q_norm_weight: Optional[torch.Tensor] = None, k_norm_weight: Optional[torch.Tensor] = None, eps: float = 0.0,
+                offset: int = 0, status: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """What lies between the packed product and the attention, in one kernel, on columns [offset, ...) of ``qkv``
+    [T, row] = [q | k | v]: a short causal convolution per channel (``conv_weight`` float32 [taps, channels], tap by tap,
+    with ``history`` float32 [slots, taps - 1, channels]; None: none), then ``norm``: None, 'rows' (an RMS norm over all
+    rows of q, and of k, at once; weights [Hq d] and [Hkv d]), 'head' (per head, weights [d]) or 'head_after' (per head
+    after the rotation; weights [d] or None: a plain division by the root mean square), and the rotation. Returns q
+    [T, Hq, d]; k and v go to their token's place in ``cache`` (planes or rows, as ``head_rotation`` takes them).
+    ``shift_history``: as in ``short_conv``. Float32 arithmetic, one rounding."""
+    _check(qkv, "qkv", None, 2)
+    _check(cache, "cache", qkv.dtype, 5)
+    for name, ten, nd in (("positions", positions, 1), ("token_seq", token_seq, 1), ("block_table", block_table, 2)):
+        _check(ten, name, torch.int32, nd)
+    t, nq, nk = qkv.shape[0], num_heads * head_dim, num_kv_heads * head_dim
+    width = nq + nk + num_kv_heads * v_dim
+    if offset < 0 or offset + width > qkv.shape[1]:
+        raise KernelError("qkv_prepare: the packed rows do not fit the rows they lie in")
+    if norm not in QKV_NORMS:
+        raise KernelError(f"qkv_prepare: unknown norm {norm!r}; known: {sorted(map(str, QKV_NORMS))}")
+    for name, w, rows in (("q_norm_weight", q_norm_weight, nq), ("k_norm_weight", k_norm_weight, nk)):
+        if w is None and norm in ("rows", "head"):
+            raise KernelError(f"qkv_prepare: this norm needs {name}")
+        if w is not None and _check(w, name, torch.float32, 1).shape[0] != (rows if norm == "rows" else head_dim):
+            raise KernelError(f"qkv_prepare: {name} does not fit the norm")
+    if rotation is not None and rotation.rotary_dim > head_dim:
+        raise KernelError(f"qkv_prepare: rotary_dim {rotation.rotary_dim} exceeds head_dim {head_dim}")
+    taps, stride = 1, 0
+    if conv_weight is not None:
+        _check(conv_weight, "conv_weight", torch.float32, 2)
+        taps = conv_weight.shape[0]
+        if conv_weight.shape[1] != width:
+            raise KernelError("qkv_prepare: every tap has a weight per packed channel")
+        if taps > 1:
+            stride = _slot_stride(history, (taps - 1) * width, "history")
+    planes = _kv_planes(cache, num_kv_heads, head_dim, v_dim)
+    q = torch.empty((t, num_heads, head_dim), dtype=qkv.dtype, device=qkv.device)
+    if t:
+        inv_freq, table, table_positions, interleaved, rotary_dim, factor = _rotation_args(rotation)
+        _run("hybrid", "ti_qkv_prepare", q.data_ptr(), cache.data_ptr(), planes, qkv.data_ptr(), qkv.shape[1], int(offset),
+             _ptr(conv_weight), history.data_ptr() if taps > 1 else None, stride, taps, int(shift_history), QKV_NORMS[norm],
+             _ptr(q_norm_weight), _ptr(k_norm_weight), float(eps), inv_freq, table, table_positions, interleaved, rotary_dim,
+             factor, positions.data_ptr(), token_seq.data_ptr(), cu_seqlens.data_ptr(), state_slots.data_ptr(),
+             block_table.data_ptr(), block_table.shape[1], t, num_heads, num_kv_heads, head_dim, v_dim, cache.shape[3],
+             cache.shape[1], _ptr(status), _dtype_code(qkv), _stream())
+    return q
+
+
+def general_delta_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay_logits: torch.Tensor,
+                       rate_logits: torch.Tensor, *, decay_bias: Optional[torch.Tensor], rate_bias: Optional[torch.Tensor],
+                       decay_scale: float, state: torch.Tensor, heads: int, key_dim: int, value_dim: int, r_offset: int = 0,
+                       k_offset: int = 0, v_offset: int = 0, decay_offset: int = 0, rate_offset: int = 0,
+                       unit_eps: float = 1e-6, cu_seqlens: torch.Tensor, state_slots: torch.Tensor,
+                       num_seqs: int) -> torch.Tensor:
+    """The generalized delta rule with a decay and a removal rate per head and key channel. Per request and head, over the
+    step's tokens in order, with u = k / sqrt(k.k + unit_eps): S <- diag(w) S - (a * u)(u^T S) + k v^T (both terms read the
+    old S), o = S^T r, from and back into ``state`` float32 [slots, heads, value_dim, key_dim] (S transposed). r and k:
+    columns [offset, + heads * key_dim), v: [offset, + heads * value_dim) of their tensors;
+    w = exp(decay_scale * sigmoid(decay_logits + decay_bias)), a = sigmoid(rate_logits + rate_bias), from float32 rows.
+    Returns o float32 [T, heads * value_dim]."""
+    for name, ten in (("r", r), ("k", k), ("v", v)):
+        _check(ten, name, r.dtype, 2)
+    t, nk, nv = r.shape[0], heads * key_dim, heads * value_dim
+    for name, ten in (("decay_logits", decay_logits), ("rate_logits", rate_logits)):
+        _check(ten, name, torch.float32, 2)
+    for name, ten in (("decay_bias", decay_bias), ("rate_bias", rate_bias)):
+        if ten is not None and _check(ten, name, torch.float32, 1).shape[0] != nk:
+            raise KernelError(f"general_delta_scan: {name} has one entry per head and key channel")
+    if any(ten.shape[0] != t for ten in (k, v, decay_logits, rate_logits)):
+        raise KernelError("general_delta_scan: one row per token in r, k, v and the logits")
+    if (r_offset + nk > r.shape[1] or k_offset + nk > k.shape[1] or v_offset + nv > v.shape[1]
+            or decay_offset + nk > decay_logits.shape[1] or rate_offset + nk > rate_logits.shape[1] or decay_scale > 0):
+        raise KernelError("general_delta_scan: the tensors do not hold these heads, or the decay would grow")
+    stride = _slot_stride(state, heads * value_dim * key_dim, "state")
+    out = torch.empty((t, nv), dtype=torch.float32, device=r.device)
+    if t:
+        work = torch.empty(t * heads * (4 * key_dim + value_dim + 2) + 28, dtype=torch.float32, device=r.device)
+        _run("hybrid", "ti_general_delta_scan", out.data_ptr(), state.data_ptr(), stride, r.data_ptr(), r.shape[1], int(r_offset),
+             k.data_ptr(), k.shape[1], int(k_offset), v.data_ptr(), v.shape[1], int(v_offset), decay_logits.data_ptr(),
+             decay_logits.shape[1], int(decay_offset), rate_logits.data_ptr(), rate_logits.shape[1], int(rate_offset),
+             _ptr(decay_bias), _ptr(rate_bias), float(decay_scale), float(unit_eps), cu_seqlens.data_ptr(),
+             state_slots.data_ptr(), int(num_seqs), t, heads, key_dim, value_dim, work.data_ptr(), work.numel(),
+             _dtype_code(r), _stream())
     return out
 
 

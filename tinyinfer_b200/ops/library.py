@@ -44,9 +44,9 @@ LIBRARIES: Dict[str, dict] = {
     "experts": dict(sources=["runtime.cu", "experts.cu"], headers=["common.cuh", "mma_tile.cuh"], link=[]),
     # parts of designs with several residual streams, short convolutions, attention over [key | value] rows,
     # rotations of packed heads, and linear attention or the delta rule with a matrix state
-    "hybrid": dict(sources=["runtime.cu", "hyper_streams.cu", "conv_attention.cu", "linear_scan.cu", "head_rotation.cu",
-                            "delta_scan.cu"],
-                   headers=["common.cuh"], link=[]),
+    "hybrid": dict(sources=["runtime.cu", "hyper_streams.cu", "single_stream.cu", "conv_attention.cu", "qkv_prepare.cu",
+                            "linear_scan.cu", "head_rotation.cu", "delta_scan.cu"],
+                   headers=["common.cuh", "short_conv.cuh"], link=[]),
     # bfloat16 tensor-core kernels (tcgen05 + TMA); only a bfloat16 model loads it
     "sm100": dict(sources=["runtime.cu", "sm100_host.cu", "gemm_tcgen05.cu", "attention_mma.cu",
                            "attention_prefill_tcgen05.cu", "attention_prefill_pair_tcgen05.cu", "gemm_pair_tcgen05.cu",

@@ -10,16 +10,20 @@ only the first features of a head, a learned sink per query head in the softmax 
 output gate sigmoid(W_g x)_h per (token, head) (``head_gate``: W_g's rows ride in the packed projection), and a
 layer without key/value tensors that reads what another layer cached (``shares_cache``), biases on q, k and v alone
 (``qkv_bias``), scores capped smoothly by a tanh (``softcap``) and q and k divided by their root mean square after the
-rotation (``qk_unit_norm``); these may be combined with a window. Such a layer runs
+rotation (``qk_unit_norm``); these may be combined with a window, or with chunks (``chunk``: a query sees the keys of its
+own chunk of positions). Such a layer runs
 ``_attend_general``: packed product [q | k | v | g], per-head norm + rotation + append (``ops.head_rotation``),
-attention with the sinks and the gate in its epilogue.
+attention with the sinks and the gate in its epilogue. A short causal convolution over q, k and v (``conv_taps``) and a
+norm over all rows of q, and of k, at once (``qk_row_norm``) take the kernel that does everything between product and
+attention a token at a time (``ops.qkv_prepare``) in place of the per-head one; the convolution's last taps - 1 inputs are
+state of the request.
 """
 from __future__ import annotations
 
 import torch
 
 from .. import ops
-from .base import CacheNeed, Mixer, TensorSpec, build_position, register_mixer
+from .base import CacheNeed, Mixer, StateNeed, TensorSpec, build_position, register_mixer
 
 
 class Attention(Mixer):
@@ -32,14 +36,19 @@ class Attention(Mixer):
         self.position = build_position(spec.position, dtype, device)
         self._rotation = self.position.rotation()      # opaque here: the kernel reads it
         self.w_qkv = self.b_qkv = self.w_o = self.b_o = None
-        self.q_norm = self.k_norm = self.sinks = None
+        self.q_norm = self.k_norm = self.sinks = self.conv_w = None
+        self._by_token = spec.conv_taps > 0 or spec.qk_row_norm is not None      # prepared a token at a time, not a head
         self._general = bool(spec.value_dim != spec.head_dim or spec.head_sinks or spec.head_gate or spec.shares_cache
-                             or spec.qkv_bias or spec.softcap or spec.qk_unit_norm is not None
+                             or spec.qkv_bias or spec.softcap or spec.qk_unit_norm is not None or spec.chunk or self._by_token
                              or getattr(spec.position, "interleaved", False) or getattr(spec.position, "blend", None))
         if self._general and spec.bias:
             raise ValueError("biases on all four projections are not combined with value sizes, sinks, gates or shared caches")
-        if spec.qk_unit_norm is not None and spec.qk_norm is not None:
-            raise ValueError("q and k are normed before the rotation or after it, not both")
+        if sum(n is not None for n in (spec.qk_unit_norm, spec.qk_norm, spec.qk_row_norm)) > 1:
+            raise ValueError("q and k are normed once: per head before the rotation or after it, or all rows at once")
+        if spec.window and spec.chunk:
+            raise ValueError("an attention layer has a window or chunks, not both")
+        if spec.conv_taps < 0 or (self._by_token and (spec.shares_cache or not spec.short_names)):
+            raise ValueError("convolutions and row norms come with short tensor names and key/value tensors of the layer's own")
         if spec.qkv_bias and (spec.bias or spec.shares_cache or not spec.short_names):
             raise ValueError("biases on q, k and v alone come with short tensor names and key/value tensors of the layer's own")
         short = spec.short_names
@@ -51,8 +60,16 @@ class Attention(Mixer):
     def cache_need(self):
         s = self.spec
         if s.value_dim != s.head_dim:       # keys and values of different sizes lie side by side in one row a token
-            return CacheNeed(s.num_kv_heads, s.head_dim + s.value_dim, s.window, planes=1)
-        return CacheNeed(s.num_kv_heads, s.head_dim, s.window)
+            return CacheNeed(s.num_kv_heads, s.head_dim + s.value_dim, s.window, planes=1, chunk=s.chunk)
+        return CacheNeed(s.num_kv_heads, s.head_dim, s.window, chunk=s.chunk)
+
+    def _packed_width(self):
+        s = self.spec
+        return s.q_size + s.kv_size + s.num_kv_heads * s.value_dim
+
+    def state_need(self):
+        taps = self.spec.conv_taps
+        return StateNeed(((taps - 1) * self._packed_width(),), torch.float32) if taps > 1 else None
 
     def tensors(self):
         s, n = self.spec, self._n
@@ -65,6 +82,12 @@ class Attention(Mixer):
             t[n["q_norm"]] = TensorSpec((s.head_dim,), role="vector32", init="ones_noise")
             if not s.shares_cache:
                 t[n["k_norm"]] = TensorSpec((s.head_dim,), role="vector32", init="ones_noise")
+        if s.qk_row_norm is not None:
+            t[n["q_norm"]] = TensorSpec((s.q_size,), role="vector32", init="ones_noise")
+            t[n["k_norm"]] = TensorSpec((s.kv_size,), role="vector32", init="ones_noise")
+        if s.conv_taps:
+            for name, rows in ((n["q"], s.q_size), (n["k"], s.kv_size), (n["v"], s.num_kv_heads * s.value_dim)):
+                t[name + ".conv"] = TensorSpec((rows, s.conv_taps), role="vector32", init="ones_noise")
         if s.head_sinks:
             t[n["sink"]] = TensorSpec((s.num_heads,), role="vector32")
         if s.head_gate:
@@ -96,6 +119,11 @@ class Attention(Mixer):
         if s.qk_norm is not None:
             self.q_norm = tensors[n["q_norm"]]
             self.k_norm = None if s.shares_cache else tensors[n["k_norm"]]
+        if s.qk_row_norm is not None:
+            self.q_norm, self.k_norm = tensors[n["q_norm"]].contiguous(), tensors[n["k_norm"]].contiguous()
+        if s.conv_taps:
+            # tap by tap, [taps, channels]: neighbouring channels are neighbours in memory, as the kernel reads them
+            self.conv_w = torch.cat([tensors[n[p] + ".conv"] for p in ("q", "k", "v")], dim=0).t().contiguous()
         if s.head_sinks:
             self.sinks = tensors[n["sink"]].contiguous()
         if s.qkv_bias:              # zeros under the gate's and the filling rows
@@ -113,20 +141,41 @@ class Attention(Mixer):
             raise ValueError("a layer with key/value tensors writes its cache entry; one without them only reads")
         packed = ops.linear(x, self.w_qkv, bias=self.b_qkv)  # [T, q | (k | v) | (g) | fill]
         gate_at = s.q_size + ((s.kv_size + s.num_kv_heads * s.value_dim) if own else 0)
-        q = ops.head_rotation(packed, num_heads=s.num_heads, num_kv_heads=s.num_kv_heads, head_dim=s.head_dim,
+        q = self._prepare_by_token(packed, step, cache) if self._by_token else ops.head_rotation(
+                              packed, num_heads=s.num_heads, num_kv_heads=s.num_kv_heads, head_dim=s.head_dim,
                               v_dim=s.value_dim, has_kv=own, positions=step.positions, token_seq=step.token_seq,
                               q_norm_weight=self.q_norm, k_norm_weight=self.k_norm,
                               eps=(s.qk_norm.eps if s.qk_norm is not None else s.qk_unit_norm or 0.0),
                               rotation=self._rotation, norm_after=s.qk_unit_norm is not None,
                               cache=cache.kv if own else None, block_table=cache.block_table, status=step.status)
         extras = dict(head_sinks=self.sinks, gate=packed if s.head_gate else None, gate_offset=gate_at,
-                      window=s.window, softcap=s.softcap or 0.0)
+                      window=s.window, chunk=s.chunk, softcap=s.softcap or 0.0)
         if cache.kv.shape[0] == 2:          # keys and values of one size: the paged attention, tensor cores where the sizes allow
             return ops.paged_attention(q, cache.kv, positions=step.positions, token_seq=step.token_seq,
                                        block_table=cache.block_table, scale=s.scale, step=step, status=step.status,
                                        **extras)
         return ops.attention_rows(q, cache.kv, v_dim=s.value_dim, positions=step.positions, token_seq=step.token_seq,
                                   block_table=cache.block_table, scale=s.scale, step=step, status=step.status, **extras)
+
+    def _prepare_by_token(self, packed, step, cache):
+        s = self.spec
+        width = self._packed_width()
+        norm, eps = ((None, 0.0) if s.qk_norm is None else ("head", s.qk_norm.eps))
+        if s.qk_row_norm is not None:
+            norm, eps = "rows", s.qk_row_norm.eps
+        elif s.qk_unit_norm is not None:
+            norm, eps = "head_after", s.qk_unit_norm
+        history = cache.state.unflatten(1, (s.conv_taps - 1, width)) if s.conv_taps > 1 else None
+        single = step.num_tokens == step.num_seqs          # every request brings one token: the kernel keeps the history itself
+        q = ops.qkv_prepare(packed, num_heads=s.num_heads, num_kv_heads=s.num_kv_heads, head_dim=s.head_dim,
+                            v_dim=s.value_dim, cache=cache.kv, block_table=cache.block_table, positions=step.positions,
+                            token_seq=step.token_seq, cu_seqlens=step.cu_seqlens, state_slots=step.state_slots,
+                            rotation=self._rotation, conv_weight=self.conv_w, history=history, shift_history=single,
+                            norm=norm, q_norm_weight=self.q_norm, k_norm_weight=self.k_norm, eps=eps, status=step.status)
+        if history is not None and not single:
+            ops.conv_state_update(history, packed, offset=0, width=width, taps=s.conv_taps, cu_seqlens=step.cu_seqlens,
+                                  state_slots=step.state_slots, num_seqs=step.num_seqs)
+        return q
 
     def _attend(self, x, step, cache, link=None, link_eps=0.0):
         s = self.spec

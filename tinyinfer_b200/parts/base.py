@@ -33,11 +33,24 @@ class TensorSpec:
 class CacheNeed:
     """Paged keys and values a mixer wants per token: ``num_kv_heads * head_dim`` for K and V
     each. ``window`` None: every key stays; n: only the last n positions are ever read, older
-    pages may be given back."""
+    pages may be given back. ``chunk`` n: a position reads its own chunk of n positions only (chunks
+    counted from position 0 of the request), so the pages of earlier chunks may be given back."""
     num_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     planes: int = 2          # 2: keys and values; 1: one row per token (a latent that both are made from)
+    chunk: Optional[int] = None
+
+    @property
+    def keeps_all(self) -> bool:
+        """Every key stays to the end of its request."""
+        return self.window is None and self.chunk is None
+
+    def first_read(self, position: int) -> int:
+        """The lowest position that a query at ``position`` or later reads."""
+        if self.chunk is not None:
+            return position // self.chunk * self.chunk
+        return 0 if self.window is None else max(0, position - self.window + 1)
 
 
 @dataclass(frozen=True)
@@ -196,6 +209,10 @@ class Block:
 
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
         pass
+
+    def state_need(self) -> Optional[StateNeed]:
+        """Per-request state of the whole block: its mixer's, and what the arrangement keeps itself, if anything."""
+        return self.mixer.state_need()
 
     def forward(self, x, step, cache):
         raise NotImplementedError

@@ -120,6 +120,71 @@ class MultiStreamBlock(Block):
         return (streams, pending), None
 
 
+class ScaledResidualBlock(Block):
+    """x <- x + m * (s1 * mixer(shift(norm1(x)))), x <- x + m * (s2 * feed_forward(norm2(x))) around one float32 stream:
+    m a constant, s1 and s2 numbers per feature ("layer scale"), and a token shift that replaces h_t by
+    h_t + (h_(t-1) - h_t) * v per feature, h_(t-1) being the request's token before as it was before this replacement
+    (zeros at the start). Each of these may be missing. What travels between blocks is the pair (stream [T, width], update
+    still to be applied): one kernel applies what a sublayer left (and what the run order adds there), norms and shifts.
+    The last h of every request is state of the block: it lies behind the mixer's own in the request's slot."""
+
+    def _vectors(self):
+        s = self.spec
+        named = {"shift": s.token_shift, "s1": s.mixer_scale}
+        if self.feed_forward is not None:
+            named["s2"] = s.feed_forward_scale
+        return {what: tensor for what, tensor in named.items() if tensor is not None}
+
+    def tensors(self):
+        from .base import TensorSpec
+        return {tensor: TensorSpec((self.mixer_norm.spec.size,), role="vector32", init="ones_noise")
+                for tensor in self._vectors().values()}
+
+    def load(self, tensors):
+        self.vectors = {what: tensors[tensor].contiguous() for what, tensor in self._vectors().items()}
+
+    def _mixer_state(self):
+        """The mixer's own floats of a slot."""
+        need = self.mixer.state_need()
+        if need is None:
+            return 0
+        if len(need.shape) != 1 or need.dtype.itemsize != 4 or not need.dtype.is_floating_point:
+            raise ValueError("a block with a token shift takes mixers whose state is one row of float32")
+        return need.shape[0]
+
+    def state_need(self):
+        if self.spec.token_shift is None:
+            return self.mixer.state_need()
+        import torch
+        from .base import StateNeed
+        return StateNeed((self._mixer_state() + self.mixer_norm.spec.size,), torch.float32)
+
+    def forward(self, x, step, cache):
+        return self.forward_linked(x, None, None, step, cache)[0]
+
+    def forward_linked(self, x, link, next_norm, step, cache):
+        import dataclasses
+        from .. import ops
+        stream, pending = x
+        m, dtype = self.spec.residual_mult, self.mixer.dtype
+        shift, previous = self.vectors.get("shift"), None
+        if shift is not None:
+            if not cache.writes:
+                raise ValueError("a layer that reads another layer's cache entry has no state of its own for a token shift")
+            own = self._mixer_state()
+            previous = cache.state[:, own:own + stream.shape[1]]
+            cache = dataclasses.replace(cache, state=cache.state[:, :own] if own else None)
+        rms = self.mixer_norm.as_rms()
+        stream, h = ops.residual_step(stream, pending, rms[0], rms[1], dtype, shift=shift, previous=previous, step=step)
+        pending = ops.ResidualUpdate(self.mixer.forward(h, step, cache), self.vectors.get("s1"), m)
+        if self.feed_forward is not None:
+            rms = self.feed_forward_norm.as_rms()
+            stream, h = ops.residual_step(stream, pending, rms[0], rms[1], dtype)
+            pending = ops.ResidualUpdate(self.feed_forward.forward(h, step), self.vectors.get("s2"), m)
+        return (stream, pending), None
+
+
 register_block("pre_norm", PreNormBlock)
 register_block("multi_stream", MultiStreamBlock)
 register_block("output_norm", OutputNormBlock)
+register_block("scaled_residual", ScaledResidualBlock)

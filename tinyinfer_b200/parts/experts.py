@@ -10,7 +10,10 @@ weights are the chosen scores themselves) and ``router_input`` 'input' (the rout
 instead of the float32 stream), ``activation`` 'silu_glu' (down(silu(W_gate h) * (W_up h))), ``scoring`` 'sigmoid' (an
 expert's score is the sigmoid of its own router logit) and ``weight_input`` (a chosen expert runs on its weight times
 the token's row, expert(w h), and the outputs are summed as they are: the up product is linear, W (w h) = w (W h), so
-the weight multiplies both halves of the stored product inside the activation kernel and costs no pass of its own).
+the weight multiplies both halves of the stored product inside the activation kernel and costs no pass of its own),
+``groups`` (equal runs of neighbouring experts, of which the ``keep_groups`` with the best expert take part in the choice),
+``weight_scale`` (a factor on the weights) and ``shared_gate`` (the shared expert's output times one sigmoid a token; a
+shared expert of a silu-gated mixture is silu-gated too).
 
 A step's (token, choice) pairs are put in expert order on the device and the experts run as two grouped
 products over row tiles; nothing is read back to the host and no token is ever dropped, so a token's result
@@ -41,10 +44,17 @@ class Experts(FeedForward):
             raise ValueError("clamped_glu needs a positive limit")
         if spec.identity_experts < 0 or spec.top > spec.num_experts + spec.identity_experts:
             raise ValueError("top exceeds the number of router outputs")
-        if spec.shared_size and spec.activation != "relu_squared":
-            raise ValueError("a shared expert is built with the relu_squared activation only")
+        if spec.shared_size and spec.activation not in ("relu_squared", "silu_glu"):
+            raise ValueError("a shared expert is built with the relu_squared and silu_glu activations only")
+        if spec.shared_gate and (not spec.shared_size or spec.activation != "silu_glu"):
+            raise ValueError("the gate belongs to a silu-gated shared expert")
+        if spec.groups < 1 or (spec.num_experts + spec.identity_experts) % spec.groups or not 1 <= spec.keep_groups <= spec.groups:
+            raise ValueError("the groups of experts are equal, and one to all of them are kept")
+        if spec.keep_groups * ((spec.num_experts + spec.identity_experts) // spec.groups) < spec.top:
+            raise ValueError("the kept groups hold fewer experts than are chosen")
         self.glu = spec.activation in ("clamped_glu", "silu_glu")
         self.w_router = self.w_up = self.w_down = self.w_shared_up = self.w_shared_down = self.correction = None
+        self.w_shared_gate = None
 
     def tensors(self):
         s = self.spec
@@ -58,8 +68,12 @@ class Experts(FeedForward):
         if s.score_correction:
             t["correction"] = TensorSpec((s.num_experts + s.identity_experts,), role="vector32")
         if s.shared_size:
+            if self.glu:
+                t["shared.gate"] = TensorSpec((s.shared_size, s.hidden_size))
             t["shared.up"] = TensorSpec((s.shared_size, s.hidden_size))
             t["shared.down"] = TensorSpec((s.hidden_size, s.shared_size))
+        if s.shared_gate:
+            t["shared.sg"] = TensorSpec((1, s.hidden_size))
         return t
 
     def load(self, tensors):
@@ -74,8 +88,11 @@ class Experts(FeedForward):
         self.w_down = torch.stack([tensors[f"e{e}.down"] for e in range(s.num_experts)]).contiguous()
         self.w_router = tensors["router"].contiguous()
         if s.shared_size:
-            self.w_shared_up = tensors["shared.up"].contiguous()
+            self.w_shared_up = (torch.cat([tensors["shared.gate"], tensors["shared.up"]], dim=0) if self.glu
+                                else tensors["shared.up"]).contiguous()
             self.w_shared_down = tensors["shared.down"].contiguous()
+        if s.shared_gate:
+            self.w_shared_gate = tensors["shared.sg"].reshape(-1).contiguous()
 
     def _experts(self, x32, x):
         """(routing, float32 sorted rows of the experts' outputs, the shared expert's output or None)."""
@@ -84,7 +101,8 @@ class Experts(FeedForward):
         routing = ops.route_experts(x32, self.w_router, s.top, s.weight_eps,
                                     tile_rows=ops.expert_tile_rows(x, s.num_experts, s.top, s.expert_size),
                                     correction=self.correction, renormalize=s.renormalize, real_experts=s.num_experts,
-                                    scoring=s.scoring)
+                                    scoring=s.scoring, groups=s.groups, keep_groups=s.keep_groups,
+                                    weight_scale=s.weight_scale)
         if self.glu:
             gate_up = ops.expert_linear(x, self.w_up, routing, up=True, activation=False)
             hidden = (ops.silu_glu(gate_up, routing.slot_weight if s.weight_input else None) if s.activation == "silu_glu"
@@ -94,7 +112,8 @@ class Experts(FeedForward):
         down = ops.expert_linear(hidden, self.w_down, routing, up=False)
         shared = None
         if s.shared_size:
-            shared = ops.linear(ops.relu_squared(ops.linear(x, self.w_shared_up)), self.w_shared_down)
+            inner = ops.gated_linear(x, self.w_shared_up) if self.glu else ops.relu_squared(ops.linear(x, self.w_shared_up))
+            shared = ops.linear(inner, self.w_shared_down)
         return routing, down, shared
 
     def forward_stream(self, x32, x, norm, step):
@@ -103,9 +122,9 @@ class Experts(FeedForward):
         rms = norm.as_rms()
         if rms is None:
             raise ValueError("the experts' fused output needs an RMSNorm behind them")
-        if self.spec.identity_experts or self.spec.weight_input:
-            raise ValueError("identity experts and experts weighted at their input are not built into the fused output "
-                             "of this arrangement")
+        if self.spec.identity_experts or self.spec.weight_input or self.spec.shared_gate:
+            raise ValueError("identity experts, experts weighted at their input and gated shared experts are not built into "
+                             "the fused output of this arrangement")
         routing, down, shared = self._experts(x if self.spec.router_input == "input" else x32, x)
         return ops.experts_combine_norm_add(x32, down, shared, routing, rms[0], rms[1], self.dtype)
 
@@ -116,10 +135,8 @@ class Experts(FeedForward):
         if s.identity_experts and s.router_input != "input":
             raise ValueError("identity experts pass the sublayer's input on, which is also what the router must read")
         routing, down, shared = self._experts(x if s.router_input == "input" or x.dtype == torch.float32 else x.float(), x)
-        out = ops.experts_combine(down, x, routing, s.num_experts, weighted=not s.weight_input)
-        if shared is not None:
-            out = ops.add(out, shared)
-        return out
+        return ops.experts_combine(down, x, routing, s.num_experts, weighted=not s.weight_input, shared=shared,
+                                   shared_gate=self.w_shared_gate)
 
 
 register_feed_forward("experts", Experts)

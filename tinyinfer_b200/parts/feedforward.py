@@ -1,4 +1,4 @@
-"""Dense gated feed-forward (SwiGLU): down(silu(gate(x)) * up(x)), no bias
+"""Dense gated feed-forward: down(act(gate(x)) * up(x)), act silu (SwiGLU) or the tanh form of gelu, no bias
 (tinyinfer/models/qwen3.py:148-150,170-175 of the reference). Gate and up are packed as one
 [2I, H] matrix so that one matrix product feeds the activation, which acts on the float32
 accumulators as the reference's kernel does (tinyinfer/csrc/mlp.cu:116-141)."""
@@ -14,8 +14,8 @@ class GatedMLP(FeedForward):
     graph_safe = True
     def __init__(self, spec, dtype, device):
         super().__init__(spec, dtype, device)
-        if spec.activation != "silu":
-            raise ValueError(f"activation {spec.activation!r} is not supported (silu only)")
+        if spec.activation not in ops.GATED_ACTIVATIONS:
+            raise ValueError(f"activation {spec.activation!r} is not supported ({', '.join(ops.GATED_ACTIVATIONS)})")
         self.w_gate_up = self.w_down = None
 
     def tensors(self):
@@ -32,20 +32,23 @@ class GatedMLP(FeedForward):
         self.w_gate_up = torch.cat([tensors[gate], tensors[up]], dim=0).contiguous()
         self.w_down = tensors[down].contiguous()
 
+    def _hidden(self, x, **link):
+        return ops.gated_linear(x, self.w_gate_up, activation=self.spec.activation, **link)
+
     def forward(self, x, step=None):
-        return ops.linear(ops.gated_linear(x, self.w_gate_up), self.w_down)
+        return ops.linear(self._hidden(x), self.w_down)
 
     def forward_residual(self, x, residual, step=None):
-        return ops.linear(ops.gated_linear(x, self.w_gate_up), self.w_down, residual=residual)
+        return ops.linear(self._hidden(x), self.w_down, residual=residual)
 
     def forward_prenorm(self, x, norm, link, next_norm, step=None):
         rms = norm.as_rms()
         if rms is None or not ops.norm_link_ok(x):
             return super().forward_prenorm(x, norm, link, next_norm, step)
         if link is not None and link.weight is rms[0]:
-            hidden = ops.gated_linear(link.scaled, self.w_gate_up, link=link, link_eps=rms[1])
+            hidden = self._hidden(link.scaled, link=link, link_eps=rms[1])
         else:
-            hidden = ops.gated_linear(norm.forward(x), self.w_gate_up)
+            hidden = self._hidden(norm.forward(x))
         after = next_norm.as_rms() if next_norm is not None else None
         if after is None:
             return ops.linear(hidden, self.w_down, residual=x), None

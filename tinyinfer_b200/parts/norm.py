@@ -15,13 +15,16 @@ class RMSNorm(Norm):
     def tensors(self):
         # a weight stored around zero (the norm multiplies by offset + w) is drawn around zero too
         init = "ones_noise" if not getattr(self.spec, "offset", 0.0) else "normal"
-        return {self.spec.tensor: TensorSpec((self.spec.size,), role="vector32", init=init)}
+        shape = () if getattr(self.spec, "single_gain", False) else (self.spec.size,)
+        return {self.spec.tensor: TensorSpec(shape, role="vector32", init=init)}
 
     def load(self, tensors):
         self.weight = tensors[self.spec.tensor]
         offset = float(getattr(self.spec, "offset", 0.0))
         if offset:
             self.weight = (self.weight + offset).contiguous()      # float32: the sum is made once, here
+        if getattr(self.spec, "single_gain", False):               # the kernels take a number per coordinate
+            self.weight = self.weight.reshape(1).expand(self.spec.size).contiguous()
 
     def forward(self, x):
         return ops.rmsnorm(x, self.weight, self.spec.eps)
