@@ -1,0 +1,797 @@
+"""The Tarupel design in the engine against its plain statement (tests/plain_tarupel.py): the new kernels alone, each
+mechanism alone in a model, then whole models in every way of cutting the work (whole prompts, a decoded tail, portions
+down to two tokens, mixed batches with pages and state slots used again), keys at the edges of chunks, windows and pages and
+far back, long decoding through captured graphs, and greedy generation through the entry point and its scheduler. Cache
+pages are poisoned with NaN so that a read outside a request's own rows shows."""
+import copy
+import random
+
+import numpy as np
+import pytest
+import torch
+
+import helpers
+import plain_tarupel as plain
+import tarupel_helpers as th
+
+pytestmark = pytest.mark.gpu
+
+TOL = {"float32": 5e-5, "bfloat16": 4e-2}     # relative to the largest |logit| of the plain statement
+LENGTHS = [1, 7, 33, 90, 61, 47, 2, 70, 18, 120, 64, 65, 3]
+
+
+def row_errors(got, want):
+    scale = max(float(np.abs(w).max()) for w in want.values())
+    return np.array([float(np.abs(got[r][p].astype(np.float64) - want[r][p]).max()) / scale
+                     for r in sorted(got) for p in sorted(got[r])])
+
+
+def agrees(got, want, dtype):
+    """float32: every row within the tolerance; this is what judges the cache, the state and the batching.
+    bfloat16: activations rounded to 8 bits through several layers (and now and then an expert chosen otherwise on a close
+    call) leave a few rows further off than the typical row, so nearly all rows must be within the tolerance, the typical
+    row well within it, and none far outside."""
+    err = row_errors(got, want)
+    if not np.isfinite(err).all():
+        return False
+    if dtype == "float32":
+        return bool(err.max() <= TOL[dtype])
+    return bool((err > TOL[dtype]).mean() <= 0.05 and np.median(err) <= TOL[dtype] / 3 and err.max() <= 6 * TOL[dtype])
+
+
+def run(folder, dtype, steps, page, **kw):
+    from tinyinfer_b200.engine.replay import TraceSession
+    session = TraceSession(folder, dtype, helpers.peak_tokens(steps, max(64, page)), page_size=page, poison_cache=True, **kw)
+    got = helpers.collect(session, steps)
+    session.runner.check_status()
+    session.runner.manager.check_consistency()
+    return got, session
+
+
+def ints(values):
+    return torch.tensor(values, dtype=torch.int32).cuda()
+
+
+class Step:
+    """The device arrays of a step of the given portions, as the residual kernel reads them."""
+
+    def __init__(self, lens, slots):
+        cu = np.concatenate([[0], np.cumsum(lens)]).tolist()
+        self.cu_seqlens, self.state_slots = ints(cu), ints(slots)
+        self.token_seq = ints([i for i, n in enumerate(lens) for _ in range(n)])
+
+
+# ------------------------------------------------------------------ the kernels alone
+@pytest.mark.parametrize("heads,dk,dv", [(3, 24, 20), (1, 8, 70), (2, 130, 9), (4, 64, 64), (2, 128, 128), (5, 7, 5), (1, 300, 4), (1, 520, 3)])
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_general_delta_scan_against_plain(heads, dk, dv, dtype):
+    """Two requests of unequal length in three calls (a prompt's portion, then a portion beside one decoded token, then a
+    portion of many of the kernel's chunks beside a short one): the state goes through slots that lie inside a larger
+    state, with someone else's floats in front."""
+    from tinyinfer_b200 import ops
+    gen = torch.Generator().manual_seed(heads * dk + dv)
+    pad, nk, nv = 5, heads * dk, heads * dv
+    decay_b, rate_b = torch.randn(nk, generator=gen) - 2, 0.5 * torch.randn(nk, generator=gen)
+    state_d = torch.zeros(3, 11 + nk * dv).cuda()
+    view = state_d[:, 11:].unflatten(1, (heads, dv, dk))
+    S = [torch.zeros(heads, dk, dv, dtype=torch.float64) for _ in range(2)]
+    for lens in ([37, 5], [1, 22], [3, 141], [1, 1]):
+        T = sum(lens)
+        row = torch.randn(T, pad + 2 * nk + nv, generator=gen).to(dtype)
+        row[:, pad + nk:pad + 2 * nk] *= dk ** -0.5
+        a, b = torch.randn(T, 3 + nk, generator=gen), 2 * torch.randn(T, 2 + nk, generator=gen)
+        rd = row.cuda()
+        got = ops.general_delta_scan(rd, rd, rd, a.cuda(), b.cuda(), decay_bias=decay_b.cuda(), rate_bias=rate_b.cuda(),
+                                     decay_scale=-0.6, state=view, heads=heads, key_dim=dk, value_dim=dv, r_offset=pad,
+                                     k_offset=pad + nk, v_offset=pad + 2 * nk, decay_offset=3, rate_offset=2, unit_eps=1e-6,
+                                     cu_seqlens=ints([0, lens[0], T]), state_slots=ints([2, 0]), num_seqs=2).cpu()
+        x = row.double()
+        r, k, v = (x[:, o:o + n].reshape(T, heads, -1) for o, n in ((pad, nk), (pad + nk, nk), (pad + 2 * nk, nv)))
+        decay = torch.exp(-0.6 * torch.sigmoid(a[:, 3:].double() + decay_b.double())).reshape(T, heads, dk)
+        rate = torch.sigmoid(b[:, 2:].double() + rate_b.double()).reshape(T, heads, dk)
+        at = 0
+        for i, n in enumerate(lens):
+            part = slice(at, at + n)
+            want, S[i] = plain.general_delta_rule(r[part], k[part], v[part], decay[part], rate[part], S[i])
+            assert (got[part].double().reshape(n, heads, dv) - want).abs().max() <= 2e-5 * max(1.0, want.abs().max()), (i, lens)
+            at += n
+    kept = state_d.cpu()
+    assert (kept[:, :11] == 0).all() and (kept[1] == 0).all()
+    for i, slot in enumerate((2, 0)):
+        assert (kept[slot, 11:].reshape(heads, dv, dk).transpose(1, 2).double() - S[i]).abs().max() <= 2e-5 * max(1.0, S[i].abs().max())
+
+
+def conv_pages(lens, page, gen):
+    """A shuffled block table for requests of these lengths, and the number of pages of the pool."""
+    counts = [(n + page - 1) // page for n in lens]
+    perm = torch.randperm(sum(counts) + 3, generator=gen).tolist()
+    table, at = [], 0
+    for c in counts:
+        table.append(perm[at:at + c] + [-1] * (max(counts) - c))
+        at += c
+    return torch.tensor(table, dtype=torch.int32), sum(counts) + 3
+
+
+@pytest.mark.parametrize("hq,hkv,d,dv,rot,interleaved,taps,norm", [
+    (6, 2, 20, 12, 12, False, 4, "head_after"), (4, 2, 64, 64, 32, False, 2, "head_after"), (3, 3, 7, 5, 4, True, 3, "rows"),
+    (8, 2, 96, 96, 24, True, 0, "rows"), (4, 1, 128, 128, 128, True, 0, "rows"), (2, 1, 8, 24, 8, False, 1, "head"),
+    (5, 1, 256, 128, 0, False, 5, "head_after"), (2, 2, 16, 16, 16, True, 4, None), (16, 8, 128, 128, 64, False, 4, "head_after")])
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_qkv_prepare_against_plain(hq, hkv, d, dv, rot, interleaved, taps, norm, dtype):
+    """Two requests in five calls (portions, a portion beside a single token, single tokens, long portions): convolution
+    through the state, norms, rotation, and every key and value where its page says."""
+    from tinyinfer_b200 import ops
+    from tinyinfer_b200.config import PositionSpec
+    from tinyinfer_b200.parts.base import build_position
+    gen = torch.Generator().manual_seed(hq * d + rot + taps)
+    cq, ck, cv = hq * d, hkv * d, hkv * dv
+    width, off, page, total = cq + ck + cv, 8, 4, [128, 96]
+    spec = PositionSpec(kind="rope", theta=777.0, rotary_dim=rot, exact_frequencies=True, interleaved=interleaved) if rot else \
+        PositionSpec(kind="none")
+    rotation = build_position(spec, dtype, "cuda").rotation()
+    conv_w = torch.randn(width, taps, generator=gen) if taps else None
+    wq, wk = ((1 + 0.3 * torch.randn(n, generator=gen) for n in ((cq, ck) if norm == "rows" else (d, d)))
+              if norm in ("rows", "head") else (None, None))
+    rows = [torch.randn(n, width, generator=gen).to(dtype) for n in total]
+    table, pages = conv_pages(total, page, gen)
+    cache = torch.full((2, pages, hkv, page, d) if d == dv else (1, pages, hkv, page, d + dv), float("nan"), dtype=dtype).cuda()
+    state = torch.zeros(3, 5 + max(0, taps - 1) * width).cuda()
+    history = state[:, 5:].unflatten(1, (taps - 1, width)) if taps > 1 else None
+    status = torch.zeros(1, dtype=torch.int32, device="cuda")
+    done, got_q = [0, 0], [[], []]
+    for lens in ([3, 2], [1, 7], [1, 1], [90, 80], [33, 6]):
+        packed = torch.cat([torch.cat([torch.randn(n, off, generator=gen).to(dtype), rows[i][done[i]:done[i] + n]], dim=1)
+                            for i, n in enumerate(lens)]).cuda()
+        step = Step(lens, [2, 0])
+        single = lens == [1, 1]
+        q = ops.qkv_prepare(packed, num_heads=hq, num_kv_heads=hkv, head_dim=d, v_dim=dv, cache=cache, block_table=table.cuda(),
+                            positions=ints([done[i] + p for i, n in enumerate(lens) for p in range(n)]), token_seq=step.token_seq,
+                            cu_seqlens=step.cu_seqlens, state_slots=step.state_slots, rotation=rotation,
+                            conv_weight=conv_w.t().contiguous().cuda() if taps else None, history=history, shift_history=single,
+                            norm=norm, q_norm_weight=wq.cuda() if wq is not None else None,
+                            k_norm_weight=wk.cuda() if wk is not None else None, eps=1e-5, offset=off, status=status)
+        if taps > 1 and not single:
+            ops.conv_state_update(history, packed, offset=off, width=width, taps=taps, cu_seqlens=step.cu_seqlens,
+                                  state_slots=step.state_slots, num_seqs=2)
+        at = 0
+        for i, n in enumerate(lens):
+            got_q[i].append(q[at:at + n].cpu().double())
+            done[i] += n
+            at += n
+    assert int(status.item()) == 0 and done == total and bool((state[:, :5] == 0).all()) and bool((state[1] == 0).all())
+    cache = cache.cpu().double()
+    tol = 5e-5 if dtype == torch.float32 else 1.2e-2      # one rounding to bfloat16 of values of a few units
+    for i, n in enumerate(total):
+        y = rows[i].double()
+        if taps:
+            y = plain.short_conv(y, conv_w.double())
+        q, k, v = y[:, :cq].reshape(n, hq, d), y[:, cq:cq + ck].reshape(n, hkv, d), y[:, cq + ck:].reshape(n, hkv, dv)
+        if norm == "rows":
+            q, k = ((plain.rms(x.reshape(n, -1), 1e-5) * w.double()).reshape(x.shape) for x, w in ((q, wq), (k, wk)))
+        elif norm == "head":
+            q, k = plain.rms(q, 1e-5) * wq.double(), plain.rms(k, 1e-5) * wk.double()
+        q, k = (plain.rotated(x, 777.0, rot, interleaved) for x in (q, k))
+        if norm == "head_after":
+            q, k = plain.rms(q, 1e-5), plain.rms(k, 1e-5)
+        assert (torch.cat(got_q[i]) - q).abs().max() <= tol * max(1.0, q.abs().max()), i
+        for p in range(n):
+            slot = cache[:, table[i, p // page], :, p % page]
+            gk, gv = (slot[0], slot[1]) if d == dv else (slot[0, :, :d], slot[0, :, d:])
+            assert (gk - k[p]).abs().max() <= tol * max(1.0, k.abs().max()), (i, p)
+            assert (gv - v[p]).abs().max() <= tol * max(1.0, v.abs().max()), (i, p)
+
+
+def test_qkv_prepare_reports_a_token_without_a_page():
+    from tinyinfer_b200 import ops
+    qkv = torch.randn(2, 3 * 16).cuda()
+    cache = torch.zeros(2, 2, 1, 4, 16).cuda()
+    status = torch.zeros(1, dtype=torch.int32, device="cuda")
+    step = Step([2], [0])
+    ops.qkv_prepare(qkv, num_heads=1, num_kv_heads=1, head_dim=16, v_dim=16, cache=cache, block_table=ints([[0, -1]]),
+                    positions=ints([3, 4]), token_seq=step.token_seq, cu_seqlens=step.cu_seqlens, state_slots=step.state_slots,
+                    status=status)
+    assert int(status.item()) == 1
+    kept = cache.cpu()
+    assert torch.equal(kept[0, 0, 0, 3], qkv[0, 16:32].cpu()) and bool((kept[:, 1] == 0).all())
+
+
+@pytest.mark.parametrize("width", [72, 50, 1024, 5000])
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_residual_step_with_token_shift(width, dtype):
+    """Updates, what a pass starts with, the norm and the token shift through the slots, in portions that reach every form
+    of the kernel (one and three tokens a block, requests that start and end inside a block); the result of a token is the
+    same bits however its request is cut."""
+    from tinyinfer_b200 import ops
+    gen = torch.Generator().manual_seed(width)
+    total = [1000, 40, 3] if width <= 1024 else [40, 9, 3]
+    x = [torch.randn(n, width, generator=gen) for n in total]
+    y = [torch.randn(n, width, generator=gen).to(dtype) for n in total]
+    add = [torch.randn(n, width, generator=gen) for n in total]
+    scale, vec, shift = (torch.randn(width, generator=gen) for _ in range(3))
+    w = 1 + 0.2 * torch.randn(width, generator=gen)
+    want_x, want_h = [], []
+    for i, n in enumerate(total):
+        u = x[i].double() + 0.7 * (scale.double() * y[i].double()) + add[i].double() + vec.double()
+        want_x.append(u)
+        want_h.append(plain.shifted(plain.rms(u, 1e-5) * w.double(), shift.double()))
+    first = None
+    cuts = ([[total[0], total[1], total[2]]],
+            [[1, 2, 1], [1, 1, 1], [total[0] - 4, 5, 1], [1, 1, 0], [1, total[1] - 9, 0]])
+    for plan in cuts:
+        state = torch.zeros(4, 6 + width).cuda()
+        done, out = [0, 0, 0], [[], [], []]
+        for lens in plan:
+            who = [i for i in range(3) if lens[i]]
+            part = lambda src: torch.cat([src[i][done[i]:done[i] + lens[i]] for i in who]).cuda()
+            xin = part(x)
+            before = xin.clone()
+            fresh, h = ops.residual_step(xin, ops.ResidualUpdate(part(y), scale.cuda(), 0.7, part(add), vec.cuda()), w.cuda(), 1e-5,
+                                         dtype, shift=shift.cuda(), previous=state[:, 6:], step=Step([lens[i] for i in who],
+                                                                                                     [[3, 0, 2][i] for i in who]))
+            assert torch.equal(xin, before), "a shifted step leaves its input as it was"
+            at = 0
+            for i in who:
+                n = lens[i]
+                assert (fresh[at:at + n].cpu().double() - want_x[i][done[i]:done[i] + n]).abs().max() < 1e-5
+                out[i].append(h[at:at + n].cpu())
+                done[i] += n
+                at += n
+        assert done == total and bool((state[1] == 0).all()) and bool((state[:, :6] == 0).all())
+        out = [torch.cat(o) for o in out]
+        for i in range(3):
+            tol = 1e-5 if dtype == torch.float32 else 8e-3
+            assert (out[i].double() - want_h[i]).abs().max() <= tol * want_h[i].abs().max(), i
+            last = state[[3, 0, 2][i], 6:].cpu().double()
+            assert (last - plain.rms(want_x[i][-1], 1e-5) * w.double()).abs().max() < 1e-4
+        if first is None:
+            first = out
+        assert all(torch.equal(a, b) for a, b in zip(first, out)), "a token's result depends on the cut"
+
+
+def test_residual_step_without_a_shift():
+    """In place; chosen rows; nothing pending; a step that only adds."""
+    from tinyinfer_b200 import ops
+    gen = torch.Generator().manual_seed(1)
+    x, y, w, s = torch.randn(9, 52, generator=gen), torch.randn(9, 52, generator=gen), torch.randn(52, generator=gen), torch.randn(52, generator=gen)
+    for dtype in (torch.float32, torch.bfloat16):
+        yd = y.to(dtype)
+        u = x.double() + 0.5 * s.double() * yd.double()
+        want = plain.rms(u, 1e-6) * w.double()
+        xd = x.cuda()
+        same, h = ops.residual_step(xd, ops.ResidualUpdate(yd.cuda(), s.cuda(), 0.5), w.cuda(), 1e-6, dtype)
+        assert same is xd and (xd.cpu().double() - u).abs().max() < 1e-5
+        tol = 1e-5 if dtype == torch.float32 else 2e-2
+        assert (h.cpu().double() - want).abs().max() <= tol * want.abs().max()
+        xd = x.cuda()
+        rows = ints([8, 0, 3])
+        _, h = ops.residual_step(xd, ops.ResidualUpdate(yd.cuda(), s.cuda(), 0.5), w.cuda(), 1e-6, dtype, rows=rows)
+        assert torch.equal(xd.cpu(), x) and (h.cpu().double() - want[[8, 0, 3]]).abs().max() <= tol * want.abs().max()
+        _, h = ops.residual_step(xd, None, w.cuda(), 1e-6, dtype)
+        assert torch.equal(xd.cpu(), x) and (h.cpu().double() - plain.rms(x.double(), 1e-6) * w.double()).abs().max() <= tol * 5
+        ops.residual_step(xd, ops.ResidualUpdate(add_rows=x.cuda(), add_vec=s.cuda()), w.cuda(), 1e-6, dtype)
+        assert torch.allclose(xd.cpu(), 2 * x + s, atol=1e-6)
+
+
+ATTENTION_SHAPES = [
+    # hq, hkv, d, dv, page, [(context, q_len)]
+    (6, 2, 20, 12, 8, [(37, 37), (50, 1), (9, 2)]),                       # rows of [k | v]: the float32-arithmetic kernel
+    (3, 1, 8, 40, 4, [(130, 1), (17, 17)]),
+    (8, 2, 96, 96, 16, [(150, 150), (131, 1), (90, 3)]),                  # two planes, a size the tensor-core kernels refuse
+    (8, 2, 64, 64, 16, [(130, 130), (129, 1), (200, 2)]),                 # two planes: the tensor-core kernels
+    (8, 4, 128, 128, 64, [(1500, 1), (1, 1), (256, 1), (257, 1), (700, 513)]),
+    (4, 4, 128, 128, 64, [(1300, 897), (64, 64), (65, 1), (390, 130)]),
+    (6, 2, 64, 64, 32, [(600, 600), (131, 1), (90, 3)]),
+    (2, 1, 128, 128, 16, [(2400, 200), (2560, 1), (2561, 1), (640, 384)]),
+]
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("pairs", [False, True])
+@pytest.mark.parametrize("chunk,window", [(1, None), (7, None), (64, None), (120, None), (128, None), (300, None), (None, 65), (None, 1)])
+@pytest.mark.parametrize("hq,hkv,d,dv,page,work", ATTENTION_SHAPES)
+def test_attention_within_chunks(monkeypatch, dtype, pairs, chunk, window, hq, hkv, d, dv, page, work):
+    """Chunks smaller and larger than the kernels' tiles and pages, on their borders and off them, in every attention
+    kernel; keys and values of earlier chunks are NaN wherever no query of the step may read them (the pages a request has
+    given back), and their neighbours in a page are loud enough to show a key too many."""
+    from tinyinfer_b200 import ops
+    if pairs and (d != dv or d not in (64, 128) or dtype == torch.float32):
+        pytest.skip("one form of the prompt kernel")
+    monkeypatch.setattr(ops, "PAIR_MIN_CTAS", 0 if pairs else 1 << 30)
+    gen = torch.Generator().manual_seed(hq * d)
+    first = (lambda p: p // chunk * chunk) if chunk else (lambda p: max(0, p - window + 1))
+    lens = [c for c, _ in work]
+    table, total = conv_pages(lens, page, gen)
+    planes = d == dv
+    cache = torch.full((2, total, hkv, page, d) if planes else (1, total, hkv, page, d + dv), float("nan"), dtype=dtype)
+    ks = [torch.randn(n, hkv, d, generator=gen).to(dtype) for n in lens]
+    vs = [torch.randn(n, hkv, dv, generator=gen).to(dtype) for n in lens]
+    for i, (n, q_len) in enumerate(work):
+        kept = first(n - q_len) // page * page                     # pages below are given back
+        for p in range(kept, n):
+            pg = table[i, p // page]
+            if planes:
+                cache[0, pg, :, p % page], cache[1, pg, :, p % page] = ks[i][p], vs[i][p]
+            else:
+                cache[0, pg, :, p % page] = torch.cat([ks[i][p], vs[i][p]], dim=-1)
+        table[i, :kept // page] = -1
+    pos = torch.tensor([p for c, n in work for p in range(c - n, c)], dtype=torch.int32)
+    seq = torch.tensor([i for i, (c, n) in enumerate(work) for _ in range(n)], dtype=torch.int32)
+    q = (2.0 * torch.randn(pos.shape[0], hq, d, generator=gen)).to(dtype)
+    status = torch.zeros(1, dtype=torch.int32, device="cuda")
+    args = dict(positions=pos.cuda(), token_seq=seq.cuda(), block_table=table.cuda(), scale=d ** -0.5, status=status,
+                chunk=chunk, window=window)
+    out = ops.paged_attention(q.cuda(), cache.cuda(), **args) if planes else ops.attention_rows(q.cuda(), cache.cuda(), v_dim=dv, **args)
+    assert int(status.item()) == 0
+    ops.check_kernel_status()
+    out = out.cpu().double()
+    worst, at = 0.0, 0
+    for i, (n, q_len) in enumerate(work):
+        lo = first(n - q_len)
+        mask = (plain.chunk_mask(n, chunk) if chunk else plain.window_mask(n, window))[n - q_len:, lo:]
+        want = plain.softmax_attention(q[at:at + q_len].double(), ks[i][lo:].double(), vs[i][lo:].double(), d ** -0.5, mask)
+        worst = max(worst, float((out[at:at + q_len] - want).abs().max()))
+        at += q_len
+    assert worst <= (2e-5 if dtype == torch.float32 else 3e-2), worst
+
+
+@pytest.mark.parametrize("m,k,inter", [(1, 72, 56), (3, 128, 136), (16, 1024, 512), (64, 256, 384), (65, 96, 40), (300, 512, 640),
+                                       (700, 512, 6144)])
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_gated_product_with_tanh_gelu(m, k, inter, dtype):
+    from tinyinfer_b200 import ops
+    gen = torch.Generator().manual_seed(m + k)
+    x, w = torch.randn(m, k, generator=gen).to(dtype), (2 * torch.randn(2 * inter, k, generator=gen) / k ** 0.5).to(dtype)
+    got = ops.gated_linear(x.cuda(), w.cuda(), activation="gelu_tanh").cpu().double()
+    xd, wd = (x.double(), w.double()) if m < 300 else (x.cuda().double(), w.cuda().double())
+    want = (plain.gelu_tanh(xd @ wd[:inter].t()) * (xd @ wd[inter:].t())).cpu()
+    ops.check_kernel_status()
+    assert (got - want).abs().max() <= (2e-5 if dtype == torch.float32 else 8e-3) * want.abs().max()
+
+
+@pytest.mark.parametrize("experts,top,groups,keep,ff,shared,width,tokens", [
+    (6, 3, 3, 2, 24, 40, 72, 37), (1, 1, 1, 1, 16, 8, 40, 9), (8, 4, 8, 4, 8, 16, 40, 5), (16, 5, 4, 2, 64, 64, 128, 600),
+    (64, 6, 8, 3, 16, 24, 64, 50), (256, 8, 64, 5, 8, 8, 40, 33), (9, 3, 3, 1, 8, 16, 24, 20)])
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_experts_chosen_by_groups_with_a_gated_shared_expert(experts, top, groups, keep, ff, shared, width, tokens, dtype):
+    """The choice among the kept groups, weights over the chosen scores' sum times a factor, the weighted sum and the
+    shared expert times its gate, op by op as the experts' part strings them together."""
+    from tinyinfer_b200 import ops
+    gen = torch.Generator().manual_seed(experts * 7 + top)
+    draw = lambda *shape: torch.randn(*shape, generator=gen)
+    x = draw(tokens, width).to(dtype)
+    w = {"router": 3.0 * draw(experts, width), "shared.gate": draw(shared, width), "shared.up": draw(shared, width),
+         "shared.down": draw(width, shared), "shared.sg": 2.0 * draw(1, width)}
+    for e in range(experts):
+        w.update({f"e{e}.gate": draw(ff, width), f"e{e}.up": draw(ff, width), f"e{e}.down": draw(width, ff)})
+    w = {n: (t / t.shape[-1] ** 0.5).to(dtype) for n, t in w.items()}
+    xd = x.cuda()
+    routing = ops.route_experts(xd, w["router"].cuda(), top, 1e-20, tile_rows=ops.expert_tile_rows(xd, experts, top, ff),
+                                groups=groups, keep_groups=keep, weight_scale=1.7)
+    s = torch.softmax(x.double() @ w["router"].double().t(), dim=-1)
+    # rows on which neither the groups nor the experts are close to a tie
+    best = torch.sort(s.view(tokens, groups, -1).max(-1).values, dim=-1, descending=True)
+    allowed = torch.zeros(tokens, groups, dtype=torch.bool).scatter_(1, best.indices[:, :keep], True)
+    masked = s.masked_fill(~allowed.repeat_interleave(experts // groups, dim=1), -1.0)
+    ranked = torch.sort(masked, dim=-1, descending=True).values
+    clear = torch.ones(tokens, dtype=torch.bool)
+    if keep < groups:
+        clear &= (best.values[:, keep - 1] - best.values[:, keep]) > 1e-4 * best.values[:, keep]
+    if top < experts:
+        clear &= (ranked[:, top - 1] - ranked[:, top]) > 1e-4 * ranked[:, top - 1]
+    assert clear.float().mean() > 0.85
+    chosen = routing.chosen.cpu().long()
+    for t in torch.nonzero(clear).flatten().tolist():
+        assert sorted(chosen[t].tolist()) == sorted(plain.grouped_choice(s[t], top, groups, keep).tolist()), t
+    if top > keep and groups > keep:
+        assert any(sorted(chosen[t].tolist()) != sorted(torch.topk(s[t], top).indices.tolist()) for t in range(tokens)), "the groups never bind"
+    picked = torch.gather(s, 1, chosen)
+    assert (routing.weight.cpu().double() - 1.7 * picked / picked.sum(-1, keepdim=True)).abs().max() < 2e-5
+    up = torch.stack([torch.cat([w[f"e{e}.gate"], w[f"e{e}.up"]]) for e in range(experts)]).cuda()
+    down = torch.stack([w[f"e{e}.down"] for e in range(experts)]).cuda()
+    rows = ops.expert_linear(ops.silu_glu(ops.expert_linear(xd, up, routing, up=True, activation=False)), down, routing, up=False)
+    inner = ops.gated_linear(xd, torch.cat([w["shared.gate"], w["shared.up"]]).cuda())
+    got = ops.experts_combine(rows, xd, routing, experts, shared=ops.linear(inner, w["shared.down"].cuda()),
+                              shared_gate=w["shared.sg"].reshape(-1).contiguous().cuda()).cpu().double()
+    wd = {n: t.double() for n, t in w.items()}
+    f = th.moe(experts, top, ff, groups=(groups, keep), scale=1.7, shared=shared)
+    want = plain.experts(wd, f, x.double())
+    assert (got - want)[clear].abs().max() <= (5e-5 if dtype == torch.float32 else 3e-2) * max(1.0, want.abs().max())
+
+
+def test_tanh_of_columns():
+    from tinyinfer_b200 import ops
+    x = 3 * torch.randn(7, 21, generator=torch.Generator().manual_seed(0))
+    assert (ops.tanh_rows(x.cuda(), 5, 13, torch.float32).cpu().double() - torch.tanh(x[:, 5:18].double())).abs().max() < 1e-6
+    assert (ops.tanh_rows(x.cuda(), 20, 1, torch.bfloat16).cpu().double() - torch.tanh(x[:, 20:].double())).abs().max() < 4e-3
+
+
+# ------------------------------------------------------------------ each mechanism alone
+ALONE = {
+    "chunked": th.config([th.layer("attention", th.attention(6, 2, 20, 12, scale=0.35, rot=12, size=9, conv=4), None)]),
+    "chunked_planes": th.config([th.layer("attention", th.attention(4, 2, 64, 64, scale=0.2, rot=32, size=30, conv=2), None)]),
+    "windowed": th.config([th.layer("attention_2", th.attention(6, 2, 12, 20, scale=0.35, rot=8, size=9), None)]),
+    "windowed_planes": th.config([th.layer("attention_2", th.attention(4, 2, 64, 64, scale=0.2, rot=64, size=30), None)]),
+    "delta": th.config([th.layer("general_delta", th.delta(3, 20, gate_rank=7), None)]),
+    "dense": th.config([th.layer("general_delta", th.delta(1, 8), th.dense(56))]),
+    "experts": th.config([th.layer("general_delta", th.delta(1, 8), th.moe(9, 4, 24, groups=(3, 2), scale=2.2, shared=40))]),
+    "looped": th.config([th.layer("general_delta", th.delta(2, 8), None), th.layer("attention_2", th.attention(2, 1, 8, 8, size=6), None)],
+                        loop=(0, 2, 4)),
+}
+
+
+@pytest.mark.parametrize("name", sorted(ALONE))
+def test_one_mechanism_alone(tmp_path, name):
+    cfg = ALONE[name]
+    folder = th.write_folder(tmp_path / "m", cfg, seed=11)
+    requests = th.random_requests(cfg, [75, 1, 2, 19], seed=4)
+    want = th.plain_logits(folder, requests)
+    for steps in (helpers.trace_whole(requests), helpers.trace_chunked(requests, seed=3), helpers.trace_decode_tail(requests, tail=80)):
+        got, _ = run(folder, "float32", steps, page=8)
+        assert helpers.first_bad(got, want, TOL["float32"]) is None
+
+
+@pytest.mark.parametrize("name", ["MIX", "WIDE", "ONE"])
+def test_residual_after_every_layer_run(tmp_path, name):
+    """The float32 stream after every layer run of a prompt (a looped layer counts each time), not only the logits."""
+    from tinyinfer_b200.engine.replay import TraceSession
+    cfg = getattr(th, name)
+    folder = th.write_folder(tmp_path / "m", cfg, seed=2)
+    tokens = th.random_requests(cfg, [23], seed=1)["r0"]
+    c, w = th.read_folder(folder)
+    want = []
+    th.forward(c, w, tokens, residuals=want)
+    session = TraceSession(folder, "float32", 64, page_size=8, cuda_graphs=False)
+    got = []
+    for block in session.model.blocks:          # a block returns the stream and the update that the next norm applies
+        inner = block.forward_linked
+
+        def watched(x, link, next_norm, step, cache, _inner=inner):
+            out = _inner(x, link, next_norm, step, cache)
+            (stream, update), _ = out
+            got.append((stream + update.factor * update.scale * update.y).detach().cpu().double())
+            return out
+        block.forward_linked = watched
+    session.run_step({"step": 0, "entries": [{"id": "a", "tokens": tokens, "want": [len(tokens) - 1]}], "end": ["a"]})
+    assert len(got) == len(want) == len(plain.run_order(cfg))
+    for i, rows in enumerate(got):
+        assert (rows - want[i]).abs().max() <= 2e-5 * want[i].abs().max(), i
+
+
+# ------------------------------------------------------------------ whole models, every cut
+def traces_for(requests, max_live=4):
+    return {"whole": helpers.trace_whole(requests), "tail": helpers.trace_decode_tail(requests, tail=32),
+            "chunked": helpers.trace_chunked(requests, seed=1), "mixed": helpers.trace_mixed(requests, seed=2, max_live=max_live)}
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name,page", [("MIX", 8), ("WIDE", 16), ("ONE", 4)])
+def test_every_cut_matches_plain(tmp_path, name, page, dtype):
+    cfg = getattr(th, name)
+    folder = th.write_folder(tmp_path / name, cfg, seed=3, dtype=dtype)
+    requests = th.random_requests(cfg, LENGTHS, seed=5)
+    want = th.plain_logits(folder, requests)
+    results = {}
+    for tag, steps in traces_for(requests).items():
+        got, session = run(folder, dtype, steps, page, max_live=4)
+        assert {r: len(v) for r, v in got.items()} == {r: len(t) for r, t in requests.items()}, tag
+        assert agrees(got, want, dtype), (tag, helpers.first_bad(got, want, TOL[dtype]), np.sort(row_errors(got, want))[-8:])
+        if tag == "mixed":
+            stats = session.runner.manager.stats()
+            assert all(g["pages_taken"] > g["pages"] for g in stats["groups"]), "pages were not used again"
+        results[tag] = got
+    for tag in ("tail", "chunked", "mixed"):        # the cuts against each other: rounding only
+        assert agrees(results[tag], {r: np.stack([results["whole"][r][p] for p in range(len(t))]) for r, t in requests.items()},
+                      dtype), tag
+
+
+def test_two_state_slots_serve_many_requests(tmp_path):
+    """Slots (convolution histories, matrix states, the tokens before) and pages are handed from finished requests to new
+    ones; a slot that is taken again starts from zero, not from what its last owner left."""
+    cfg = th.MIX
+    folder = th.write_folder(tmp_path / "m", cfg, seed=8)
+    requests = th.random_requests(cfg, [30, 9, 41, 2, 17, 55, 5, 26], seed=9)
+    want = th.plain_logits(folder, requests)
+    steps = helpers.trace_mixed(requests, seed=4, max_live=2, decode_tail=6)
+    got, session = run(folder, "float32", steps, page=4, max_live=2)
+    assert helpers.first_bad(got, want, TOL["float32"]) is None
+    assert session.runner.manager.stats()["free_state_slots"] == 2
+
+
+def test_batch_of_unequal_requests_equals_each_alone(tmp_path):
+    cfg = th.WIDE
+    folder = th.write_folder(tmp_path / "m", cfg, seed=5)
+    requests = th.random_requests(cfg, [50, 3, 128, 17], seed=2)
+    together = [{"step": 0, "entries": [{"id": r, "tokens": t, "want": list(range(len(t)))} for r, t in requests.items()],
+                 "end": list(requests)}]
+    got, _ = run(folder, "float32", together, page=16)
+    alone, _ = run(folder, "float32", helpers.trace_whole(requests), page=16)
+    want = th.plain_logits(folder, requests)
+    assert helpers.first_bad(got, want, TOL["float32"]) is None
+    scale = max(float(np.abs(w).max()) for w in want.values())
+    assert max(float(np.abs(got[r][p] - alone[r][p]).max()) for r in requests for p in got[r]) / scale <= 1e-5
+
+
+def test_a_request_left_out_of_steps_goes_on(tmp_path):
+    """A request pauses for some steps while others run and end (their slots and pages change hands meanwhile)."""
+    cfg = th.MIX
+    folder = th.write_folder(tmp_path / "m", cfg, seed=4)
+    requests = th.random_requests(cfg, [40, 21, 33], seed=7)
+    a, b, c = (requests[f"r{i}"] for i in range(3))
+    want = th.plain_logits(folder, requests)
+    every = lambda toks, lo, hi: {"tokens": toks[lo:hi], "want": list(range(hi - lo))}
+    steps = [
+        {"step": 0, "entries": [dict(id="r0", **every(a, 0, 13)), dict(id="r1", **every(b, 0, 21))], "end": ["r1"]},
+        {"step": 1, "entries": [dict(id="r2", **every(c, 0, 2))], "end": []},
+        {"step": 2, "entries": [dict(id="r2", **every(c, 2, 33))], "end": ["r2"]},
+        {"step": 3, "entries": [dict(id="r0", **every(a, 13, 14))], "end": []},
+        {"step": 4, "entries": [dict(id="r0", **every(a, 14, 40))], "end": ["r0"]},
+    ]
+    got, _ = run(folder, "float32", steps, page=8, max_live=2)
+    assert helpers.first_bad(got, want, TOL["float32"]) is None
+
+
+# ------------------------------------------------------------------ edges of chunks and windows, far keys, first tokens
+def quiet(t):
+    """No token shift and a convolution of the current token alone: a key hangs on its own token only; and sharp scores."""
+    for name in t:
+        if name.endswith(".shift"):
+            t[name] = torch.zeros_like(t[name])
+        if name.endswith(".conv"):
+            t[name] = torch.zeros_like(t[name])
+            t[name][:, -1] = 1.0
+
+
+def edge_config(kind, size, planes):
+    d, dv = (64, 64) if planes else (12, 20)
+    m = th.attention(4, 2, d, dv, scale=4.0 / d ** 0.5, rot=d // 4 * 2, size=size, conv=3 if kind == "attention" else 0)
+    return th.config([th.layer(kind, m, None)], width=64)
+
+
+@pytest.mark.parametrize("dtype,planes", [("float32", False), ("float32", True), ("bfloat16", True)])
+@pytest.mark.parametrize("kind,size", [("attention", 24), ("attention", 37), ("attention_2", 24), ("attention_2", 37)])
+def test_keys_just_inside_and_outside(tmp_path, kind, size, planes, dtype):
+    """One token is replaced. At the positions that may see it the logits move and agree with the plain statement; at the
+    first position that may not, and at all behind it, they are what they were. In prompts and token by token, for tokens
+    at the edges of chunks, windows and pages."""
+    cfg = edge_config(kind, size, planes)
+    folder = th.write_folder(tmp_path / "m", cfg, seed=31, dtype=dtype, edit=quiet)
+    base = th.random_requests(cfg, [4 * size + 5], seed=3)["r0"]
+    n = len(base)
+    places = sorted({0, size - 1, size, 2 * size - 1, 2 * size, 15, 16, 47, 48, 2 * size + 3} - {n})
+    requests = {"base": base}
+    for p in places:
+        requests[f"p{p}"] = base[:p] + [(base[p] + 1) % cfg["vocab"]] + base[p + 1:]
+    want = th.plain_logits(folder, requests)
+    scale = np.abs(want["base"]).max()
+    for steps in (helpers.trace_whole(requests), helpers.trace_decode_tail(requests, tail=3 * size), helpers.trace_chunked(requests, seed=5)):
+        got, _ = run(folder, dtype, steps, page=16)
+        assert agrees(got, want, dtype)
+        for p in places:
+            last = (p // size + 1) * size - 1 if kind == "attention" else p + size - 1        # the last position that sees p
+            moved = [float(np.abs(got[f"p{p}"][i] - got["base"][i]).max()) / scale for i in range(n)]
+            should = [float(np.abs(want[f"p{p}"][i] - want["base"][i]).max()) / scale for i in range(n)]
+            assert max(moved[:p], default=0.0) <= 1e-6 and max(moved[last + 1:], default=0.0) <= 1e-6, p
+            assert max(should[last + 1:], default=0.0) == 0.0
+            if last < n and should[last] > 10 * TOL[dtype]:
+                assert moved[last] > 5 * TOL[dtype], p
+    # the premise: for some of these places the very last position that sees the token moves by far more than the tolerance
+    seen = 0
+    for p in places:
+        last = (p // size + 1) * size - 1 if kind == "attention" else p + size - 1
+        seen += last < n and np.abs(want[f"p{p}"][last] - want["base"][last]).max() / scale > 10 * TOL["float32"]
+    assert seen >= 2
+
+
+def far_config():
+    """Chunks, a window and a state that reach far back; scores sharp enough that one key takes nearly all of a head."""
+    return th.config([
+        th.layer("attention", th.attention(4, 2, 16, 24, scale=3.0, rot=8, size=640, conv=3), th.dense(48)),
+        th.layer("general_delta", th.delta(2, 16), None),
+        th.layer("attention_2", th.attention(4, 2, 16, 16, scale=3.0, rot=8, size=500), th.dense(48)),
+    ], width=64, loop=(1, 2, 2))
+
+
+def slow_decay(t):
+    t["l1.mix.w0"] = torch.full_like(t["l1.mix.w0"], -9.0)
+    t["l1.mix.w2"] = 0.1 * t["l1.mix.w2"]
+    t["l1.mix.a.b"] = torch.full_like(t["l1.mix.a.b"], -6.0)
+
+
+def test_far_tokens_carry_the_result(tmp_path):
+    """Positions around the borders of pages and of the kernels' key tiles are decoded one by one; cutting the first 64
+    tokens off moves the last logits by far more than the tolerance, so a missing or misplaced row, or a state lost on the
+    way, shows."""
+    cfg = far_config()
+    folder = th.write_folder(tmp_path / "m", cfg, seed=21, edit=slow_decay)
+    requests = th.random_requests(cfg, [700], seed=13)
+    tokens = requests["r0"]
+    want = th.plain_logits(folder, requests)
+    c, w = th.read_folder(folder)
+    other = [(t + 1) % cfg["vocab"] for t in tokens[:64]] + tokens[64:]
+    assert np.abs(th.forward(c, w, other)[-200:-60] - want["r0"][-200:-60]).max() > 100 * TOL["float32"] * np.abs(want["r0"]).max()
+    for steps in (helpers.trace_whole(requests), helpers.trace_decode_tail(requests, tail=140), helpers.trace_chunked(requests, seed=7)):
+        got, _ = run(folder, "float32", steps, page=16)
+        assert helpers.first_bad(got, want, 2 * TOL["float32"]) is None
+    folder16 = th.write_folder(tmp_path / "m16", cfg, seed=21, dtype="bfloat16", edit=slow_decay)
+    want16 = th.plain_logits(folder16, requests)
+    for steps in (helpers.trace_whole(requests), helpers.trace_decode_tail(requests, tail=140), helpers.trace_chunked(requests, seed=7)):
+        got, _ = run(folder16, "bfloat16", steps, page=16)
+        err = row_errors(got, want16)
+        assert np.isfinite(err).all() and np.median(err) <= 4e-2 and (err > 0.25).mean() <= 0.03, np.sort(err)[-5:]
+
+
+def test_one_far_key_among_hundreds(tmp_path):
+    """Query and key matrices are scaled so that one early key outscores all others of its chunk by a wide margin: the
+    logits at the end hang on that token's value. Replacing the token changes them; the engine agrees with the plain
+    statement on both, decoded through the cache, at several page sizes."""
+    cfg = th.config([th.layer("attention", th.attention(2, 1, 16, 16, scale=8.0, size=400), None)], width=32)
+    folder = th.write_folder(tmp_path / "m", cfg, seed=5, edit=quiet)
+    base = th.random_requests(cfg, [300], seed=3)["r0"]
+    c, w = th.read_folder(folder)
+    full = th.forward(c, w, base)
+    moves = {}
+    for p in (3, 15, 16, 17, 31, 32, 63, 64, 65, 100):
+        other = list(base)
+        other[p] = (other[p] + 1) % cfg["vocab"]
+        moves[p] = float(np.abs(th.forward(c, w, other)[-40:] - full[-40:]).max())
+    far = max(moves, key=moves.get)
+    assert moves[far] > 1e-2 * np.abs(full).max()
+    changed = list(base)
+    changed[far] = (changed[far] + 1) % cfg["vocab"]
+    requests = {"r0": base, "r1": changed}
+    want = th.plain_logits(folder, requests)
+    for page in (4, 16, 64):
+        got, _ = run(folder, "float32", helpers.trace_decode_tail(requests, tail=40), page=page)
+        assert helpers.first_bad(got, want, TOL["float32"]) is None, page
+
+
+def test_the_first_tokens(tmp_path):
+    """Position zero (no token before, no angle, an empty state, a convolution that sees only zeros behind it, a softmax of
+    one key), then the next few, as prompts of one to six tokens and decoded one by one from the start."""
+    cfg = th.MIX
+    folder = th.write_folder(tmp_path / "m", cfg, seed=12)
+    requests = th.random_requests(cfg, [1, 2, 3, 4, 5, 6], seed=8)
+    want = th.plain_logits(folder, requests)
+    got, _ = run(folder, "float32", helpers.trace_whole(requests), page=4)
+    assert helpers.first_bad(got, want, TOL["float32"]) is None
+    got, _ = run(folder, "float32", helpers.trace_decode_tail(requests, tail=6), page=4)
+    assert helpers.first_bad(got, want, TOL["float32"]) is None
+
+
+# ------------------------------------------------------------------ long decoding through graphs
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_long_decoding_replays_graphs(tmp_path, dtype):
+    cfg = th.MIX
+    folder = th.write_folder(tmp_path / "m", cfg, seed=6, dtype=dtype)
+    requests = th.random_requests(cfg, [160, 150, 155], seed=1)
+    want = th.plain_logits(folder, requests)
+    steps = [{"step": 0, "entries": [{"id": r, "tokens": t[:4], "want": [0, 1, 2, 3]} for r, t in requests.items()], "end": []}]
+    for p in range(4, 150):
+        steps.append({"step": p, "entries": [{"id": r, "tokens": [t[p]], "want": [0]} for r, t in requests.items()],
+                      "end": list(requests) if p == 149 else []})
+    got, session = run(folder, dtype, steps, page=8)
+    assert session.runner.graph_replays > 100
+    assert agrees(got, {r: w[:150] for r, w in want.items()}, dtype)
+
+
+# ------------------------------------------------------------------ generation through the entry point
+@pytest.mark.parametrize("dtype,tol", [("float32", 1e-4), ("bfloat16", 8e-2)])
+def test_greedy_generation_through_the_scheduler(tmp_path, dtype, tol):
+    from tinyinfer_b200 import LLM
+    from tinyinfer_b200.sampling import SamplingParams
+    cfg = th.MIX
+    folder = th.write_folder(tmp_path / "m", cfg, seed=3, dtype=dtype)
+    llm = LLM(folder, dtype=dtype, max_num_batched_tokens=24, max_num_seqs=3, kvcache_block_size=8,
+              num_kvcache_blocks=40, prefill_chunk=9, max_model_len=128)
+    assert llm.config.enable_prefix_caching is False          # a state cannot be rebuilt from pages
+    prompts = list(th.random_requests(cfg, [1, 7, 16, 33, 50], seed=6).values())
+    outs = llm.generate(prompts, SamplingParams(greedy=True, max_tokens=10))
+    c, w = th.read_folder(folder)
+    for p, o in zip(prompts, outs):
+        assert o["all_token_ids"] == p + o["token_ids"] and len(o["token_ids"]) == 10
+        logits = th.forward(c, w, p + o["token_ids"])
+        for i, tok in enumerate(o["token_ids"]):          # teacher forcing: the token has (nearly) the largest plain logit
+            row = logits[len(p) - 1 + i]
+            assert row.max() - row[tok] <= tol * np.abs(logits).max()
+    assert not llm.runner.manager.live_requests
+    llm.runner.manager.check_consistency()
+    llm.close()
+
+
+def test_command_line_generates_with_a_folder_and_with_a_preset(tmp_path):
+    import json
+    import subprocess
+    import sys
+    from pathlib import Path
+    root = Path(__file__).resolve().parent.parent
+    folder = th.write_folder(tmp_path / "m", th.ONE, seed=3)
+    common = ["--dtype", "fp32", "--prompt-ids", "5,17,3,200", "--prompt-len", "9", "--greedy", "--max-tokens", "6",
+              "--max-num-seqs", "2", "--max-num-batched-tokens", "16", "--block-size", "4", "--num-kvcache-blocks", "32",
+              "--max-model-len", "64"]
+    res = subprocess.run([sys.executable, str(root / "examples" / "generate.py"), "--model", str(folder)] + common,
+                         capture_output=True, text=True, timeout=600)
+    assert res.returncode == 0, res.stderr[-2000:]
+    rows = [json.loads(l) for l in res.stdout.splitlines() if l.startswith("{")]
+    assert len(rows) == 2 and all(len(r["token_ids"]) == 6 for r in rows)
+    c, w = th.read_folder(folder)
+    logits = th.forward(c, w, [5, 17, 3, 200] + rows[0]["token_ids"])
+    for i, tok in enumerate(rows[0]["token_ids"]):
+        assert logits[3 + i].max() - logits[3 + i][tok] <= 1e-4 * np.abs(logits).max()
+    res = subprocess.run([sys.executable, str(root / "examples" / "generate.py"), "--random-config", "tarupel-tiny"] + common,
+                         capture_output=True, text=True, timeout=600)
+    assert res.returncode == 0, res.stderr[-2000:]
+
+
+def test_trace_runner_program(tmp_path):
+    """The replay program itself: steps on standard input, a file of logits per step that wants some, 'done' lines."""
+    import json
+    import subprocess
+    from pathlib import Path
+    root = Path(__file__).resolve().parent.parent
+    cfg = th.ONE
+    folder = th.write_folder(tmp_path / "m", cfg, seed=9, dtype="bfloat16")
+    requests = th.random_requests(cfg, [20, 70, 9], seed=2)
+    steps = helpers.trace_mixed(requests, seed=1, max_live=3, decode_tail=5)
+    out = tmp_path / "out"
+    out.mkdir()
+    res = subprocess.run([str(root / "bin" / "trace_run"), "--model", str(folder), "--dtype", "float32", "--out", str(out),
+                          "--max-tokens", str(helpers.peak_tokens(steps))], input="".join(json.dumps(s) + "\n" for s in steps),
+                         capture_output=True, text=True, timeout=1200)
+    assert res.returncode == 0, res.stderr[-2000:]
+    assert [l for l in res.stdout.splitlines() if l.startswith("done ")] == [f"done {s['step']}" for s in steps]
+    want = th.plain_logits(folder, requests)
+    upto = {}
+    for s in steps:
+        wanted = [(e["id"], upto.get(e["id"], 0) + p) for e in s["entries"] for p in e["want"]]
+        for e in s["entries"]:
+            upto[e["id"]] = upto.get(e["id"], 0) + len(e["tokens"])
+        rows = np.fromfile(out / f"{s['step']}.f32", dtype="<f4").reshape(len(wanted), cfg["vocab"])
+        for row, (rid, p) in zip(rows, wanted):
+            assert np.abs(row - want[rid][p]).max() <= TOL["float32"] * np.abs(want[rid]).max()
+
+
+def random_config(seed):
+    """A model of random sizes and layer order: odd head counts and sizes, one to five taps or none, partial and no
+    rotation, chunks and windows from one key on or none, with and without feed-forward, experts with and without groups
+    and a shared expert, loops anywhere or none."""
+    rng = random.Random(seed)
+    layers = []
+    for _ in range(rng.randint(2, 6)):
+        roll = rng.random()
+        mlp = None if roll < 0.2 else th.dense(rng.choice([24, 56, 136]))
+        if roll > 0.5:
+            groups, per = rng.randint(1, 4), rng.randint(1, 4)
+            keep = rng.randint(1, groups)
+            mlp = th.moe(groups * per, rng.randint(1, min(6, keep * per)), rng.choice([8, 24, 40]),
+                         groups=(groups, keep) if rng.random() < 0.8 or keep < groups else None, scale=rng.uniform(0.5, 2.5),
+                         shared=rng.choice([None, 16, 40]))
+        kind = rng.choice(["attention", "attention_2", "general_delta"])
+        if kind == "general_delta":
+            layers.append(th.layer(kind, th.delta(rng.randint(1, 5), rng.choice([4, 8, 12, 36, 72]), gate_rank=rng.choice([1, 3, 8, 16])), mlp))
+            continue
+        kv, d = rng.randint(1, 3), rng.choice([8, 12, 20, 40, 64])
+        m = th.attention(kv * rng.randint(1, 3), kv, d, d if rng.random() < 0.4 else rng.choice([4, 8, 24, 36]), scale=rng.uniform(0.1, 0.5),
+                         rot=rng.choice([0, 4, d // 4 * 2, d]), base=rng.choice([100.0, 10000.0, 1e6]),
+                         size=rng.choice([None, 1, 2, 5, 16, 33, 64, 200]), conv=rng.randint(0, 5) if kind == "attention" else 0)
+        layers.append(th.layer(kind, m, mlp))
+    n = len(layers)
+    start = rng.randrange(n)
+    loop = None if rng.random() < 0.3 else (start, rng.randint(start + 1, n), rng.randint(1, 3))
+    return th.config(layers, vocab=rng.choice([97, 256, 300]), width=rng.choice([40, 72, 100, 136]), eps=rng.choice([1e-5, 1e-6]),
+                     scale=rng.choice([1.0, 3.0, 7.5]), mult=rng.choice([1.0, 0.5, 0.9]), loop=loop)
+
+
+@pytest.mark.parametrize("seed", [1, 2, 3, 4, 5, 6, 7, 8])
+def test_models_of_random_sizes_and_orders(tmp_path, seed):
+    cfg = random_config(seed)
+    page = [4, 8, 16, 32, 64, 16, 16, 8][seed - 1]
+    requests = th.random_requests(cfg, [70, 1, 37, 150, 2, 64], seed=seed)
+    folder = th.write_folder(tmp_path / "m", cfg, seed=seed)
+    want = th.plain_logits(folder, requests)
+    for steps in (helpers.trace_whole(requests), helpers.trace_mixed(requests, seed=seed, max_live=3, decode_tail=20)):
+        got, _ = run(folder, "float32", steps, page, max_live=3)
+        assert helpers.first_bad(got, want, TOL["float32"]) is None, cfg
+    folder16 = th.write_folder(tmp_path / "m16", cfg, seed=seed, dtype="bfloat16")
+    got, _ = run(folder16, "bfloat16", helpers.trace_mixed(requests, seed=seed, max_live=3, decode_tail=20), page, max_live=3)
+    err = row_errors(got, th.plain_logits(folder16, requests))
+    assert np.isfinite(err).all() and np.median(err) <= TOL["bfloat16"] / 2, (np.median(err), cfg)

@@ -265,7 +265,11 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap q_map, const _
                             moved = true;
                         }
                     }
-                    if (js[x] < t1x[x] && js[x] == jp[x]) {                // S of the next tile: behind the P V before it
+                    // S of the next tile: behind the P V before it. A barrier's parity only tells neighbouring rounds of
+                    // its buffer apart, so whoever waits for a buffer must know that its round before is over: tile B,
+                    // whose keys may begin any number of tiles after A's (its rows lie in the next chunk), starts its
+                    // first two tiles j only once A has issued P V of tile j - 2.
+                    if (js[x] < t1x[x] && js[x] == jp[x] && (x == 0 || js[1] >= t0x[1] + 2 || jp[0] + 1 >= js[1])) {
                         const int j = js[x], li = 2 * (j - tmin), b = li % NBUF;
                         if (mbar_test_wait(kv_full(b), (li / NBUF) & 1u)) {
                             tmem_fence_after();
