@@ -28,6 +28,9 @@ the Ravutar preset of the same width, the nearest design with matrix-state layer
 ``--design fezozen`` does it for the Fezozen design (capped, windowed and latent attention, sigmoid-scored experts
 weighted at their input, a norm before and after every sublayer), beside Qwen3 and the Gulisun preset of the same
 width, the nearest design with latent attention and routed experts around a float32 stream.
+``--design tarupel`` does it for the Tarupel design (chunked attention with short convolutions, windowed attention with
+whole-projection norms, the generalized delta rule, experts chosen by groups with a gated shared expert), beside Qwen3 and
+the Sinulix preset of the same width, the nearest design with a delta rule and gated experts.
 
 ``--impl reference`` runs the unmodified reference project from ``baseline/_ref`` through its own
 public API (``tinyinfer.LLM(Config(...))``, ``add_request``, ``step``) on a model folder of the same
@@ -654,11 +657,56 @@ def fezozen_numbers(cfg, batch, context):
     return dict(macs=macs, attn_per_key=0.0, attn_window_keys=per_layer, head=head, step_bytes=step_bytes)
 
 
+def tarupel_numbers(cfg, batch, context):
+    """As ``fezozen_numbers`` for the Tarupel design: matrix elements a token multiplies (active experts and the shared
+    one), attention flops per key with the keys a layer's chunk (a negative size in ``attn_window_keys``) or window holds,
+    flops a token spends in the delta rule (decay, u^T S, the removal, the write and the read-out), and the bytes a decode
+    step must move: dense weights, the experts a batch of this size is expected to touch, the head, the cached rows a
+    query at ``context`` reads, every request's matrix states read and written."""
+    w, macs, dense, expert_bytes, cache_bytes, scan_flops, state_bytes, per_layer = cfg.width, 0, 0, 0.0, 0.0, 0.0, 0, []
+    runs = [cfg.layers[e.layer] for e in cfg.execution()]
+    for layer in runs:
+        m, f = layer["mixer"], layer.get("mlp")
+        if layer["type"] == "general_delta":
+            n, rank = m["heads"] * m["dim"], m.get("gate_rank", 16)
+            part = 5 * w * n + rank * (w + n) + w * n
+            scan_flops += 9.0 * n * m["dim"]
+            state_bytes += n * m["dim"] * 4 * 2
+        else:
+            h, g, d, v = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            part = w * (h * d + g * (d + v)) + w * h * v
+            size = (m.get("mask") or {}).get("size") or 0
+            if layer["type"] == "attention":
+                seen = (context - 1) % size + 1 if size else context
+                per_layer.append((2.0 * h * (d + v), -size))
+            else:
+                seen = min(context, size) if size else context
+                per_layer.append((2.0 * h * (d + v), size))
+            cache_bytes += seen * g * (d + v) * 2
+        if f is not None and f["kind"] == "dense":
+            part += 3 * f["ff"] * w
+        elif f is not None:
+            e, top, ff = f["router"]["experts"], f["router"]["top"], f["expert"]["ff"]
+            part += e * w + (3 * f["shared"]["ff"] * w + w if f.get("shared") else 0)
+            macs += top * 3 * ff * w
+            touched = e * (1.0 - (1.0 - top / e) ** batch)
+            expert_bytes += touched * 3 * ff * w * 2
+        macs += part
+        dense += part
+    head = cfg.vocab * w
+    step_bytes = dense * 2 + expert_bytes + head * 2 + batch * cache_bytes + batch * state_bytes
+    return dict(macs=macs, attn_per_key=0.0, attn_window_keys=per_layer, head=head, step_bytes=step_bytes, scan_flops=scan_flops)
+
+
 def windowed_attention_flops(per_layer, t):
-    """Attention flops of a prompt of ``t`` tokens: position p sees min(p + 1, window) keys of a layer."""
+    """Attention flops of a prompt of ``t`` tokens: position p sees min(p + 1, window) keys of a layer, or, where the
+    size is negative, the p % size + 1 keys of its chunk."""
     total = 0.0
     for per_key, window in per_layer:
-        if window and window < t:
+        if window < 0:
+            whole, rest = divmod(t, -window)
+            total += per_key * (whole * window * (window - 1) / 2.0 + rest * (rest + 1) / 2.0)
+        elif window and window < t:
             total += per_key * (window * (window + 1) / 2.0 + (t - window) * window)
         else:
             total += per_key * t * (t + 1) / 2.0
@@ -670,9 +718,11 @@ DESIGNS = {      # design -> (what its numbers are made with, [(its preset, the 
     "gulisun": (gulisun_numbers, (("gulisun-1b", "0.6b"), ("gulisun-2b", "1.7b"))),
     "ravutar": (ravutar_numbers, (("ravutar-1b", "0.6b"), ("ravutar-2b", "1.7b"))),
     "sinulix": (sinulix_numbers, (("sinulix-1b", "0.6b"), ("sinulix-2b", "1.7b"))),
+    "tarupel": (tarupel_numbers, (("tarupel-1b", "0.6b"), ("tarupel-2b", "1.7b"))),
 }
 SIBLINGS = {"sinulix-1b": ("ravutar", "ravutar-1b"), "sinulix-2b": ("ravutar", "ravutar-2b"),   # also measured beside it
-            "fezozen-1b": ("gulisun", "gulisun-1b"), "fezozen-2b": ("gulisun", "gulisun-2b")}
+            "fezozen-1b": ("gulisun", "gulisun-1b"), "fezozen-2b": ("gulisun", "gulisun-2b"),
+            "tarupel-1b": ("sinulix", "sinulix-1b"), "tarupel-2b": ("sinulix", "sinulix-2b")}
 
 
 
@@ -740,7 +790,7 @@ def design_comparison(args) -> int:
     numbers_of, pairs = DESIGNS[design]
     for ours, theirs in pairs:
         g = preset_config(ours)
-        layers = len(g.run_order()) if hasattr(g, "run_order") else len(g.layers)
+        layers = len(g.run_order()) if hasattr(g, "run_order") else len(g.execution()) if hasattr(g, "execution") else len(g.layers)
         numbers = numbers_of(g, batch, context)
         t = prefill_tokens
         flops = (2.0 * numbers["macs"] * t + numbers["attn_per_key"] * t * (t + 1) / 2.0 + 2.0 * numbers["head"]
@@ -786,7 +836,7 @@ def main() -> int:
     ap.add_argument("--skip-points", action="store_true", help="only the headline batch")
     ap.add_argument("--skip-extras", action="store_true", help="leave out the 'configs' of the line")
     ap.add_argument("--extras", default="32b,mix,cpu", help="which of the other configurations to run")
-    ap.add_argument("--design", default="", choices=["", "gulisun", "ravutar", "sinulix", "fezozen"],
+    ap.add_argument("--design", default="", choices=["", "gulisun", "ravutar", "sinulix", "fezozen", "tarupel"],
                     help="instead of the headline: prefill and decode of this design beside Qwen3 at equal size")
     ap.add_argument("--ref-block-size", type=int, default=256, help="reference arm: its kvcache_block_size (its default)")
     ap.add_argument("--ref-step-tokens", type=int, default=32,

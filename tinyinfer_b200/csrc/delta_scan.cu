@@ -11,7 +11,7 @@
 //   delta_scan_kernel walks a request's tokens in order. The columns of S are independent of one another, and the
 //   update of a column is not a composition of diagonal maps (the transition I - beta k k^T is a full matrix), so
 //   the parallelism is requests x heads x value columns. A block is one request x one head x a few columns; a thread
-//   holds KPT neighbouring rows of one column, a column's rows are spread over KP lanes. With D = diag(g) S, the
+//   holds KPT neighbouring rows of one column (of two, in a walk of many tokens), a column's rows are spread over KP lanes. With D = diag(g) S, the
 //   read-out is o = D^T q + u (k.q): both sums over the rows, D^T k and D^T q, are taken in one pass and meet in
 //   one round of shuffles, and only S <- D + k u^T is carried to the next token. Chunks of tokens come into shared
 //   memory by cp.async, the next chunk while the current one is walked.
@@ -161,13 +161,15 @@ struct DeltaScanArgs {
     int vec_k, vec_v;             // rows of dk floats, and a block's columns of v, move in 16-byte pieces
 };
 
-template <int KPT, int KP, bool GENERAL>
+// NC: columns of S a lane holds. Two of them share every read of a token's rows from shared memory, which is what a walk of
+// many tokens spends most of its time on, and interleave their chains of dependent sums.
+template <int KPT, int KP, int NC, bool GENERAL>
 __global__ void __launch_bounds__(DS_MAX_WARPS * 32) delta_scan_kernel(DeltaScanArgs a) {
     extern __shared__ __align__(16) float smem[];
     constexpr int PITCH = KPT + 4;                       // floats from one lane part's rows to the next: no two lanes in a bank
     constexpr int trow = KP * PITCH;
     constexpr int ROWS = GENERAL ? 4 : 3;                // rows of channels a token brings: q, k, g and, in the general form, a
-    constexpr int cols_per_warp = 32 / KP;
+    constexpr int cols_per_warp = 32 / KP * NC;
     const int threads = blockDim.x, warps = threads >> 5;
     const int cpb = warps * cols_per_warp;
     const int col_blocks = (a.dv + cpb - 1) / cpb;
@@ -175,9 +177,8 @@ __global__ void __launch_bounds__(DS_MAX_WARPS * 32) delta_scan_kernel(DeltaScan
     const int seq = blockIdx.y;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int kpart = lane % KP;
-    const int lcol = warp * cols_per_warp + lane / KP;
-    const int col = cb * cpb + lcol;
-    const bool col_ok = col < a.dv;
+    const int lcol = warp * cols_per_warp + (lane / KP) * NC;          // the lane's first column in the block
+    const int col0 = cb * cpb + lcol;
     const int g = h / (a.heads / a.groups);
     const int buf_floats = (a.chunk * (ROWS * trow + cpb + 2) + 3) & ~3;
     for (int e = tid; e < 2 * buf_floats; e += threads) smem[e] = 0.f;   // the rows past dk stay zero
@@ -192,10 +193,13 @@ __global__ void __launch_bounds__(DS_MAX_WARPS * 32) delta_scan_kernel(DeltaScan
     __syncthreads();
     ti_grid_wait();
     const int row0 = a.cu_seqlens[seq], row1 = a.cu_seqlens[seq + 1];
-    float* srow = a.state + (size_t)a.state_slots[seq] * a.slot_stride + ((size_t)h * a.dv + (col_ok ? col : 0)) * a.dk;
-    float S[KPT];
+    float* shead = a.state + (size_t)a.state_slots[seq] * a.slot_stride + (size_t)h * a.dv * a.dk;
+    float S[NC][KPT];
 #pragma unroll
-    for (int r = 0; r < KPT; ++r) S[r] = (col_ok && kpart * KPT + r < a.dk) ? srow[kpart * KPT + r] : 0.f;
+    for (int c = 0; c < NC; ++c)
+#pragma unroll
+        for (int r = 0; r < KPT; ++r)
+            S[c][r] = (col0 + c < a.dv && kpart * KPT + r < a.dk) ? shead[(size_t)(col0 + c) * a.dk + kpart * KPT + r] : 0.f;
 
     // a chunk's tokens t0 .. t0 + n - 1 into one of the two buffers
     auto fetch = [&](int t0, int n, float* buf) {
@@ -256,67 +260,100 @@ __global__ void __launch_bounds__(DS_MAX_WARPS * 32) delta_scan_kernel(DeltaScan
         const float* sv = sq + (size_t)ROWS * a.chunk * trow;
         const float* sb = sv + (size_t)a.chunk * cpb;
         const float* sx = sb + a.chunk;
-        for (int tt = 0; tt < n; ++tt) {
-            const float vv = sv[tt * cpb + lcol], beta = sb[tt], kq = sx[tt];
-            const float4* pq = reinterpret_cast<const float4*>(sq + (size_t)tt * trow + kpart * PITCH);
-            const float4* pk = reinterpret_cast<const float4*>(sk + (size_t)tt * trow + kpart * PITCH);
-            const float4* pg = reinterpret_cast<const float4*>(sg + (size_t)tt * trow + kpart * PITCH);
-            float kr[KPT];
-            float dk0 = 0.f, dk1 = 0.f, dq0 = 0.f, dq1 = 0.f;
+        // in a walk a token's rows come to registers one token ahead of their use, so that no read of shared memory stands
+        // between the sums of one token and those of the next
+        struct Row { float k[KPT], q[KPT], g[KPT], a[GENERAL ? KPT : 1], v[NC], beta, kq; };
+        auto read_row = [&](int tt, Row& x) {
+            const size_t at = (size_t)tt * trow + kpart * PITCH;
 #pragma unroll
-            for (int r4 = 0; r4 < KPT / 4; ++r4) {
-                const float4 gv = pg[r4], kv = pk[r4], qv = pq[r4];
-                const float gr[4] = {gv.x, gv.y, gv.z, gv.w}, qr[4] = {qv.x, qv.y, qv.z, qv.w};
-                kr[r4 * 4] = kv.x; kr[r4 * 4 + 1] = kv.y; kr[r4 * 4 + 2] = kv.z; kr[r4 * 4 + 3] = kv.w;
-#pragma unroll
-                for (int j = 0; j < 4; ++j) {
-                    const int r = r4 * 4 + j;
-                    const float old = S[r];
-                    S[r] *= gr[j];
-                    if constexpr (GENERAL) {             // the removal reads the old state, the read-out the decayed one
-                        if (j & 1) { dk1 = fmaf(old, kr[r], dk1); dq1 = fmaf(S[r], qr[j], dq1); }
-                        else { dk0 = fmaf(old, kr[r], dk0); dq0 = fmaf(S[r], qr[j], dq0); }
-                    } else if (j & 1) { dk1 = fmaf(S[r], kr[r], dk1); dq1 = fmaf(S[r], qr[j], dq1); }
-                    else { dk0 = fmaf(S[r], kr[r], dk0); dq0 = fmaf(S[r], qr[j], dq0); }
+            for (int r4 = 0; r4 < KPT; r4 += 4) {
+                const float4 qv = *reinterpret_cast<const float4*>(sq + at + r4), kv = *reinterpret_cast<const float4*>(sk + at + r4);
+                const float4 gv = *reinterpret_cast<const float4*>(sg + at + r4);
+                x.q[r4] = qv.x; x.q[r4 + 1] = qv.y; x.q[r4 + 2] = qv.z; x.q[r4 + 3] = qv.w;
+                x.k[r4] = kv.x; x.k[r4 + 1] = kv.y; x.k[r4 + 2] = kv.z; x.k[r4 + 3] = kv.w;
+                x.g[r4] = gv.x; x.g[r4 + 1] = gv.y; x.g[r4 + 2] = gv.z; x.g[r4 + 3] = gv.w;
+                if constexpr (GENERAL) {
+                    const float4 av = *reinterpret_cast<const float4*>(sa + at + r4);
+                    x.a[r4] = av.x; x.a[r4 + 1] = av.y; x.a[r4 + 2] = av.z; x.a[r4 + 3] = av.w;
                 }
             }
-            float dot = dk0 + dk1, oq = dq0 + dq1;
 #pragma unroll
-            for (int off = 1; off < KP; off <<= 1) {
-                dot += __shfl_xor_sync(0xffffffffu, dot, off);
-                oq += __shfl_xor_sync(0xffffffffu, oq, off);
-            }
-            float o;
-            if constexpr (GENERAL) {
-                const float4* pa = reinterpret_cast<const float4*>(sa + (size_t)tt * trow + kpart * PITCH);
+            for (int c = 0; c < NC; ++c) x.v[c] = sv[tt * cpb + lcol + c];
+            x.beta = sb[tt];
+            x.kq = sx[tt];
+        };
+        auto token = [&](int tt, const Row& x) {
+            float dot[NC][2], oq[NC][2];                 // two chains a sum
 #pragma unroll
-                for (int r4 = 0; r4 < KPT / 4; ++r4) {
-                    const float4 av = pa[r4];
-                    const float ar[4] = {av.x, av.y, av.z, av.w};
+            for (int c = 0; c < NC; ++c) dot[c][0] = dot[c][1] = oq[c][0] = oq[c][1] = 0.f;
 #pragma unroll
-                    for (int j = 0; j < 4; ++j) {
-                        const int r = r4 * 4 + j;
-                        S[r] = fmaf(kr[r], fmaf(-ar[j], dot, vv), S[r]);
-                    }
+            for (int r = 0; r < KPT; ++r)
+#pragma unroll
+                for (int c = 0; c < NC; ++c) {
+                    // the general form removes along u of the old state and reads the decayed one
+                    const float old = S[c][r];
+                    S[c][r] = old * x.g[r];
+                    dot[c][r & 1] = fmaf(GENERAL ? old : S[c][r], x.k[r], dot[c][r & 1]);
+                    oq[c][r & 1] = fmaf(S[c][r], x.q[r], oq[c][r & 1]);
                 }
-                o = fmaf(vv, kq, fmaf(-dot, beta, oq));
-            } else {
-                const float u = beta * (vv - dot);
+            float d[NC], o[NC];
 #pragma unroll
-                for (int r = 0; r < KPT; ++r) S[r] = fmaf(kr[r], u, S[r]);
-                o = fmaf(u, kq, oq);
+            for (int c = 0; c < NC; ++c) {
+                d[c] = dot[c][0] + dot[c][1];
+                o[c] = oq[c][0] + oq[c][1];
             }
-            if (kpart == 0 && col_ok) a.y[(size_t)(t0 + tt) * a.heads * a.dv + h * a.dv + col] = o;
+#pragma unroll
+            for (int off = 1; off < KP; off <<= 1)
+#pragma unroll
+                for (int c = 0; c < NC; ++c) {
+                    d[c] += __shfl_xor_sync(0xffffffffu, d[c], off);
+                    o[c] += __shfl_xor_sync(0xffffffffu, o[c], off);
+                }
+#pragma unroll
+            for (int c = 0; c < NC; ++c) {
+                if constexpr (GENERAL) {
+#pragma unroll
+                    for (int r = 0; r < KPT; ++r) S[c][r] = fmaf(x.k[r], fmaf(-x.a[r], d[c], x.v[c]), S[c][r]);
+                    o[c] = fmaf(x.v[c], x.kq, fmaf(-d[c], x.beta, o[c]));
+                } else {
+                    const float u = x.beta * (x.v[c] - d[c]);
+#pragma unroll
+                    for (int r = 0; r < KPT; ++r) S[c][r] = fmaf(x.k[r], u, S[c][r]);
+                    o[c] = fmaf(u, x.kq, o[c]);
+                }
+            }
+            if (kpart == 0) {
+#pragma unroll
+                for (int c = 0; c < NC; ++c)
+                    if (col0 + c < a.dv) a.y[(size_t)(t0 + tt) * a.heads * a.dv + h * a.dv + col0 + c] = o[c];
+            }
+        };
+        if constexpr (NC == 1) {                         // steps of single tokens: nothing to read ahead, and fewer registers
+            for (int tt = 0; tt < n; ++tt) {
+                Row x;
+                read_row(tt, x);
+                token(tt, x);
+            }
+        } else {
+            Row even, odd;
+            read_row(0, even);
+            for (int tt = 0; tt < n; tt += 2) {
+                read_row(min(tt + 1, n - 1), odd);
+                token(tt, even);
+                if (tt + 1 >= n) break;
+                read_row(min(tt + 2, n - 1), even);
+                token(tt + 1, odd);
+            }
         }
         __syncthreads();                                 // the chunk has been read: its buffer may be filled again
     }
     ds_wait<0>();
     ti_grid_launch_dependents();                         // only now: the walk is long, and the next kernel's blocks would sit on the SMs through it
-    if (col_ok) {
+#pragma unroll
+    for (int c = 0; c < NC; ++c)
 #pragma unroll
         for (int r = 0; r < KPT; ++r)
-            if (kpart * KPT + r < a.dk) srow[kpart * KPT + r] = S[r];
-    }
+            if (col0 + c < a.dv && kpart * KPT + r < a.dk) shead[(size_t)(col0 + c) * a.dk + kpart * KPT + r] = S[c][r];
 }
 
 static inline size_t ds_round4(size_t n) { return (n + 3) & ~(size_t)3; }
@@ -327,37 +364,47 @@ static int ds_launch_scan(const DeltaWork& w, float* y, float* state, long long 
                           const int* state_slots, int num_seqs, int num_tokens, int heads, int groups, int dk, int dv,
                           cudaStream_t stream) {
     constexpr int rows_in = GENERAL ? 4 : 3;
+    // a walk of many tokens, or a step of single tokens
+    const bool walk = num_tokens != num_seqs;
     int kp = 1;
     const int rows = 8;                                  // most rows of a column that a lane holds
     while (kp < 32 && (dk + kp - 1) / kp > rows) kp <<= 1;
     const int per_lane = (dk + kp - 1) / kp;
     const int kpt = per_lane <= 4 ? 4 : per_lane <= 8 ? 8 : per_lane <= 16 ? 16 : 32;
-    // few columns a block when the step has few (request, head) pairs, so that every SM has a block; many columns a
-    // block otherwise, as every block fetches the head's q, k and g for itself
+    const int nc = walk && kpt <= 16 ? 2 : 1;
+    const int lane_cols = 32 / kp * nc;                  // columns of a warp
+    // few columns a block when the step has few (request, head) pairs, so that most SMs have a block; many columns a
+    // block otherwise, as every block fetches the head's rows for itself
     int warps = DS_MAX_WARPS;
-    while (warps > 1 && (long long)num_seqs * heads * ((dv + warps * (32 / kp) - 1) / (warps * (32 / kp))) < 148) warps >>= 1;
-    const int trow = kp * (kpt + 4), cpb = warps * (32 / kp);
-    // two buffers of `chunk` tokens within the 48 KB that need no opt-in; a step of single tokens stages no more than one
-    int chunk = 16;
-    while (chunk > 1 && 2 * ds_round4((size_t)chunk * (rows_in * trow + cpb + 2)) * sizeof(float) > 44 * 1024) chunk >>= 1;
-    if (num_tokens == num_seqs) chunk = 1;
+    const int least = walk ? 100 : 148;
+    while (warps > 1 && (long long)num_seqs * heads * ((dv + warps * lane_cols - 1) / (warps * lane_cols)) < least) warps >>= 1;
+    const int trow = kp * (kpt + 4), cpb = warps * lane_cols;
+    // two buffers of `chunk` tokens: a walk takes up to 100 KB, two blocks an SM; a step of single tokens stages no more than one
+    int chunk = walk ? 16 : 1;
+    while (chunk > 1 && 2 * ds_round4((size_t)chunk * (rows_in * trow + cpb + 2)) * sizeof(float) > 100 * 1024) chunk >>= 1;
     const size_t smem = 2 * ds_round4((size_t)chunk * (rows_in * trow + cpb + 2)) * sizeof(float);
     DeltaScanArgs args = {w, y, state, slot_stride, cu_seqlens, state_slots, heads, groups, dk, dv, chunk,
                           dk % 4 == 0, dv % 4 == 0 && cpb % 4 == 0};
     dim3 grid(heads * ((dv + cpb - 1) / cpb), num_seqs);
     // a walk of many tokens starts alone (see ti_launch_alone); a step of single tokens is short and starts early
-    const bool alone = num_tokens != num_seqs;
     bool launched = false;
-#define TI_DSCAN(KPT, KP)                                                                         \
-    if (!launched && kpt == KPT && kp == KP) {                                                    \
-        if (alone) ti_launch_alone(delta_scan_kernel<KPT, KP, GENERAL>, grid, warps * 32, smem, stream, args); \
-        else ti_launch(delta_scan_kernel<KPT, KP, GENERAL>, grid, warps * 32, smem, stream, args);         \
-        launched = true;                                                                          \
+#define TI_DSCAN_N(KPT, KP, NC)                                                                                       \
+    if (!launched && kpt == KPT && kp == KP && nc == NC) {                                                            \
+        if (smem > 44 * 1024) {                                                                                       \
+            const cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<KPT, KP, NC, GENERAL>,                       \
+                                                       cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);       \
+            TI_REQUIRE(e == cudaSuccess, "delta_scan: shared memory: %s", cudaGetErrorString(e));                     \
+        }                                                                                                             \
+        if (walk) ti_launch_alone(delta_scan_kernel<KPT, KP, NC, GENERAL>, grid, warps * 32, smem, stream, args);     \
+        else ti_launch(delta_scan_kernel<KPT, KP, NC, GENERAL>, grid, warps * 32, smem, stream, args);                \
+        launched = true;                                                                                              \
     }
+#define TI_DSCAN(KPT, KP) TI_DSCAN_N(KPT, KP, 1) TI_DSCAN_N(KPT, KP, 2)
 #define TI_DSCAN_ROWS(KPT) TI_DSCAN(KPT, 1) TI_DSCAN(KPT, 2) TI_DSCAN(KPT, 4) TI_DSCAN(KPT, 8) TI_DSCAN(KPT, 16) TI_DSCAN(KPT, 32)
-    TI_DSCAN_ROWS(4) TI_DSCAN_ROWS(8) TI_DSCAN_ROWS(16) TI_DSCAN(32, 32)
+    TI_DSCAN_ROWS(4) TI_DSCAN_ROWS(8) TI_DSCAN(16, 32) TI_DSCAN_N(32, 32, 1)
 #undef TI_DSCAN_ROWS
 #undef TI_DSCAN
+#undef TI_DSCAN_N
     TI_REQUIRE(launched, "delta_scan: no kernel for %d rows a lane over %d lanes", kpt, kp);
     TI_CHECK_LAUNCH("delta_scan");
     return 0;

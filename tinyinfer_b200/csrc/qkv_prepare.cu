@@ -1,4 +1,5 @@
-// Between the packed product [q | k | v] of an attention layer and its attention, all in one kernel, a block a token:
+// Between the packed product [q | k | v] of an attention layer and its attention, all in one kernel, a block a token (in
+// steps of few tokens several blocks a token, each with some of its heads):
 //   convolution : optional short causal convolution per channel of q, k and v (short_conv.cuh; weights float32
 //                 [taps][q | k | v], the earlier inputs in the request's state slot), before everything else
 //   norm        : 0 none; 1 RMS norm over ALL rows of q, and of k, at once with a weight per row; 2 RMS norm per head with a
@@ -22,6 +23,7 @@ struct QkvPrepareArgs {
     const float *inv_freq, *table; int table_positions, interleaved, rotary_dim; float rot_factor;
     const int *positions, *token_seq, *cu_seqlens, *state_slots, *block_table; int max_blocks;
     int hq, hkv, d, dv, page_size, num_pages;
+    int heads_per_block;          // of the token's hq + 2 hkv heads: q heads, then k heads, then v heads
     int* status;
 };
 
@@ -50,8 +52,11 @@ __global__ void __launch_bounds__(512) qkv_prepare_kernel(QkvPrepareArgs a) {
     extern __shared__ __align__(16) float qp_smem[];
     __shared__ float red[33];
     const int cq = a.hq * a.d, ck = a.hkv * a.d, width = cq + ck + a.hkv * a.dv;
-    float* buf = qp_smem;                                     // [q | k], float32
-    float* turn = qp_smem + cq + ck;                          // [cosines | sines] of the token's position
+    const int head0 = blockIdx.y * a.heads_per_block, head1 = min(a.hq + 2 * a.hkv, head0 + a.heads_per_block);
+    auto channel_of = [&](int head) { return head <= a.hq + a.hkv ? head * a.d : cq + ck + (head - a.hq - a.hkv) * a.dv; };
+    const int c_begin = channel_of(head0), c_end = channel_of(head1);    // the block's channels
+    float* turn = qp_smem;                                    // [cosines | sines] of the token's position
+    float* buf = qp_smem + ((a.rotary_dim + 3) & ~3);         // the block's share of [q | k], float32
     const int half = a.rotary_dim >> 1;
     ti_grid_launch_dependents();
     ti_grid_wait();
@@ -84,7 +89,7 @@ __global__ void __launch_bounds__(512) qkv_prepare_kernel(QkvPrepareArgs a) {
         turn[half + j] = s * a.rot_factor;
     }
     float ss_q = 0.f, ss_k = 0.f;
-    for (int c0 = tid * VEC; c0 < width; c0 += blockDim.x * VEC) {
+    for (int c0 = c_begin + tid * VEC; c0 < c_end; c0 += blockDim.x * VEC) {
         float v[VEC], newest[VEC];
         if constexpr (VEC == 1) {
             newest[0] = to_f32(in[(size_t)t * a.ld_in + a.in_off + c0]);
@@ -108,7 +113,7 @@ __global__ void __launch_bounds__(512) qkv_prepare_kernel(QkvPrepareArgs a) {
         }
 #pragma unroll
         for (int e = 0; e < VEC; ++e) {
-            buf[c0 + e] = v[e];
+            buf[c0 - c_begin + e] = v[e];
             if (c0 < cq) ss_q = fmaf(v[e], v[e], ss_q);
             else ss_k = fmaf(v[e], v[e], ss_k);
         }
@@ -121,9 +126,9 @@ __global__ void __launch_bounds__(512) qkv_prepare_kernel(QkvPrepareArgs a) {
     __syncthreads();
 
     const int warps = blockDim.x >> 5;
-    for (int head = warp; head < a.hq + a.hkv; head += warps) {
+    for (int head = head0 + warp; head < min(head1, a.hq + a.hkv); head += warps) {
         const bool is_q = head < a.hq;
-        float* x = buf + (size_t)head * a.d;                  // q heads, then k heads
+        float* x = buf + (size_t)(head - head0) * a.d;        // q heads, then k heads
         const float* w = is_q ? a.q_w : a.k_w;
         if (a.norm == 1 || a.norm == 2) {                     // each lane scales its own features; a partner is read below
             float inv = is_q ? inv_q : inv_k;
@@ -205,17 +210,26 @@ TI_API int ti_qkv_prepare(void* q_out, void* cache, int planes, const void* in, 
     QkvPrepareArgs a = {q_out, cache, planes, (long long)num_pages * hkv * page_size * d, in, ld_in, in_off, conv_w, hist,
                         slot_stride, taps, shift_history ? 1 : 0, norm, q_w, k_w, eps, inv_freq, cos_sin_table, table_positions,
                         interleaved, rotary_dim, rot_factor, positions, token_seq, cu_seqlens, state_slots, block_table,
-                        max_blocks, hq, hkv, d, dv, page_size, num_pages, status};
-    const size_t smem = (size_t)(cq + ck + rotary_dim) * sizeof(float);
+                        max_blocks, hq, hkv, d, dv, page_size, num_pages, hq + 2 * hkv, status};
+    const size_t smem = (size_t)(cq + ck + ((rotary_dim + 3) & ~3)) * sizeof(float);
     TI_REQUIRE(smem <= 200 * 1024, "qkv_prepare: %d rows of q and k do not fit shared memory", cq + ck);
     const int vec = dtype == TI_F32 ? 4 : 8;
-    const bool wide = d % vec == 0 && dv % vec == 0 && ld_in % vec == 0 && in_off % vec == 0 &&
+    // (few tokens with a history: a channel a thread, so that many threads read it side by side)
+    const bool wide = (taps == 1 || num_tokens > 128) && d % vec == 0 && dv % vec == 0 && ld_in % vec == 0 && in_off % vec == 0 &&
                       ((uintptr_t)q_out | (uintptr_t)cache | (uintptr_t)in | (uintptr_t)conv_w) % 16 == 0;
     const bool heads4 = d % 4 == 0 && dv % 4 == 0 && ((uintptr_t)q_out | (uintptr_t)cache) % 16 == 0;
     // few tokens: every channel group of a token at once; many: blocks enough to fill the machine anyway
+    // a token's heads over several blocks, unless the norm spans them
+    const int heads = hq + 2 * hkv;
+    int splits = 1;
+    if (norm != 1)
+        while (splits * 2 <= heads && splits * 2 * num_tokens <= 148) splits <<= 1;
+    a.heads_per_block = (heads + splits - 1) / splits;
+    splits = (heads + a.heads_per_block - 1) / a.heads_per_block;
+    const int share = splits > 1 ? a.heads_per_block * (d > dv ? d : dv) : width;
     int threads = 128;
     const int most = num_tokens <= 2 * 148 ? 512 : 256;
-    while (threads < most && threads * (wide ? vec : 1) < width) threads <<= 1;
+    while (threads < most && threads * (wide ? vec : 1) < share) threads <<= 1;
     typedef __nv_bfloat16 B;
 #define QP_GO(T, V, H)                                                                                                       \
     do {                                                                                                                     \
@@ -229,7 +243,7 @@ TI_API int ti_qkv_prepare(void* q_out, void* cache, int planes, const void* in, 
                                                        (int)smem);                                                           \
             TI_REQUIRE(e == cudaSuccess, "qkv_prepare: shared memory: %s", cudaGetErrorString(e));                           \
         }                                                                                                                    \
-        ti_launch(qkv_prepare_kernel<T, V, H, P>, num_tokens, threads, smem, stream, a);                                        \
+        ti_launch(qkv_prepare_kernel<T, V, H, P>, dim3(num_tokens, splits), threads, smem, stream, a);                                        \
     } while (0)
     if (dtype == TI_F32) { if (wide) QP_GO(float, 4, 4); else if (heads4) QP_GO(float, 1, 4); else QP_GO(float, 1, 1); }
     else if (dtype == TI_BF16) { if (wide) QP_GO(B, 8, 4); else if (heads4) QP_GO(B, 1, 4); else QP_GO(B, 1, 1); }
