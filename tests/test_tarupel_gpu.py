@@ -114,7 +114,7 @@ def conv_pages(lens, page, gen):
 
 @pytest.mark.parametrize("hq,hkv,d,dv,rot,interleaved,taps,norm", [
     (6, 2, 20, 12, 12, False, 4, "head_after"), (4, 2, 64, 64, 32, False, 2, "head_after"), (3, 3, 7, 5, 4, True, 3, "rows"),
-    (8, 2, 96, 96, 24, True, 0, "rows"), (4, 1, 128, 128, 128, True, 0, "rows"), (2, 1, 8, 24, 8, False, 1, "head"),
+    (6, 3, 80, 80, 20, True, 0, "rows"), (4, 1, 128, 128, 128, True, 0, "rows"), (2, 1, 8, 24, 8, False, 1, "head"),
     (5, 1, 256, 128, 0, False, 5, "head_after"), (2, 2, 16, 16, 16, True, 4, None), (16, 8, 128, 128, 64, False, 4, "head_after")])
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 def test_qkv_prepare_against_plain(hq, hkv, d, dv, rot, interleaved, taps, norm, dtype):
@@ -276,7 +276,7 @@ ATTENTION_SHAPES = [
     # hq, hkv, d, dv, page, [(context, q_len)]
     (6, 2, 20, 12, 8, [(37, 37), (50, 1), (9, 2)]),                       # rows of [k | v]: the float32-arithmetic kernel
     (3, 1, 8, 40, 4, [(130, 1), (17, 17)]),
-    (8, 2, 96, 96, 16, [(150, 150), (131, 1), (90, 3)]),                  # two planes, a size the tensor-core kernels refuse
+    (6, 3, 80, 80, 16, [(150, 150), (131, 1), (90, 3)]),                  # two planes, a size the tensor-core kernels refuse
     (8, 2, 64, 64, 16, [(130, 130), (129, 1), (200, 2)]),                 # two planes: the tensor-core kernels
     (8, 4, 128, 128, 64, [(1500, 1), (1, 1), (256, 1), (257, 1), (700, 513)]),
     (4, 4, 128, 128, 64, [(1300, 897), (64, 64), (65, 1), (390, 130)]),
@@ -287,7 +287,7 @@ ATTENTION_SHAPES = [
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("pairs", [False, True])
-@pytest.mark.parametrize("chunk,window", [(1, None), (7, None), (64, None), (120, None), (128, None), (300, None), (None, 65), (None, 1)])
+@pytest.mark.parametrize("chunk,window", [(1, None), (7, None), (64, None), (110, None), (128, None), (300, None), (None, 65), (None, 1)])
 @pytest.mark.parametrize("hq,hkv,d,dv,page,work", ATTENTION_SHAPES)
 def test_attention_within_chunks(monkeypatch, dtype, pairs, chunk, window, hq, hkv, d, dv, page, work):
     """Chunks smaller and larger than the kernels' tiles and pages, on their borders and off them, in every attention
