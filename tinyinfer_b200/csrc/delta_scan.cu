@@ -11,8 +11,8 @@
 //   delta_scan_kernel walks a request's tokens in order. The columns of S are independent of one another, and the
 //   update of a column is not a composition of diagonal maps (the transition I - beta k k^T is a full matrix), so
 //   the parallelism is requests x heads x value columns. A block is one request x one head x a few columns; a thread
-//   holds KPT neighbouring rows of one column (of two, in a walk of many tokens), a column's rows are spread over KP lanes. With D = diag(g) S, the
-//   read-out is o = D^T q + u (k.q): both sums over the rows, D^T k and D^T q, are taken in one pass and meet in
+//   holds KPT neighbouring rows of one column (of two, in a walk of many tokens), a column's rows are spread over KP
+//   lanes. With D = diag(g) S, the read-out is o = D^T q + u (k.q): both sums over the rows, D^T k and D^T q, are taken in one pass and meet in
 //   one round of shuffles, and only S <- D + k u^T is carried to the next token. Chunks of tokens come into shared
 //   memory by cp.async, the next chunk while the current one is walked.
 //
