@@ -47,12 +47,14 @@ def linear(x, w, bias=None, residual=None, out_float32=False):
     return y.to(torch.float32 if out_float32 else x.dtype)
 
 
-def gated_linear(x, w_gate_up, activation="silu"):
+def gated_linear(x, w_gate_up, activation="silu", bias=None):
     if activation != "silu":
         raise NotImplementedError(activation)
     inter = w_gate_up.shape[0] // 2
     g = _acc(x) @ _acc(w_gate_up[:inter]).T
     u = _acc(x) @ _acc(w_gate_up[inter:]).T
+    if bias is not None:
+        g, u = g + bias[:inter], u + bias[inter:]
     return ((g / (1.0 + torch.exp(-g))) * u).to(x.dtype)
 
 

@@ -324,7 +324,8 @@ class CacheManager:
                 raise RuntimeError("commit beyond the pages held")
             if g.need.keeps_all:
                 continue
-            for logical in range(min(self._first_needed_page(g, new_length), len(table))):
+            kept = (g.need.keep_first + self.page_size - 1) // self.page_size        # pages of kept first positions stay
+            for logical in range(kept, min(self._first_needed_page(g, new_length), len(table))):
                 if table[logical] >= 0:
                     g.pool.give_back(table[logical], request_id)
                     table[logical] = -1
@@ -352,7 +353,7 @@ class CacheManager:
             "prefix_queries": self.prefix_queries,
             "prefix_hit_tokens": self.prefix_hit_tokens,
             "kept_pages": len(self._page_key),
-            "groups": [{"window": g.need.window, "chunk": g.need.chunk, "entries": len(g.entries),
+            "groups": [{"window": g.need.window, "keep_first": g.need.keep_first, "chunk": g.need.chunk, "entries": len(g.entries),
                         "pages": g.pool.num_pages, "free_pages": g.pool.num_free,
                         "pages_taken": g.pool.pages_taken, "pages_returned": g.pool.pages_returned}
                        for g in self.groups],

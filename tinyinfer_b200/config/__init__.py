@@ -9,11 +9,12 @@ from .ravutar import RavutarConfig
 from .sinulix import SinulixConfig
 from .fezozen import FezozenConfig
 from .tarupel import TarupelConfig
+from .zetonex import ZetonexConfig
 
 __all__ = [
     "EngineConfig", "parse_dtype", "Architecture", "architecture_of", "known_architectures",
     "known_presets", "load_config", "lookup_architecture", "preset_config", "register_architecture", "AttentionSpec", "ExecStep",
     "GatedMLPSpec", "LayerSpec", "ModelSpec", "NormSpec", "PositionSpec", "TensorNames",
     "default_execution", "Qwen3Config", "GulisunConfig", "RavutarConfig", "SinulixConfig", "FezozenConfig",
-    "TarupelConfig",
+    "TarupelConfig", "ZetonexConfig",
 ]

@@ -38,6 +38,17 @@ class FrequencyBlend:
 
 
 @dataclass(frozen=True)
+class WavelengthBlend:
+    """Slows a rotary encoding's slow pairs down by their wavelength l = 2 pi / f (Llama 3.1's recipe): a pair keeps its
+    frequency f where l < original / high, turns at f / factor where l > original / low, and between the two at
+    (1 - s) f / factor + s f with s = (original / l - low) / (high - low)."""
+    factor: float
+    low: float
+    high: float
+    original: float
+
+
+@dataclass(frozen=True)
 class PositionSpec:
     """How positions enter a mixer. ``kind='rope'``: rotation of the first ``rotary_dim`` features of every head
     with inv_freq[j] = theta ** (-2j / rotary_dim), in pairs (j, j + rotary_dim / 2) or, ``interleaved``,
@@ -47,7 +58,8 @@ class PositionSpec:
     rotary_dim: int = 0
     exact_frequencies: bool = False         # inv_freq worked out in float64 and rounded once (default: in float32)
     interleaved: bool = False
-    blend: Optional[FrequencyBlend] = None  # frequencies slowed down for lengths beyond the original one
+    blend: Optional[object] = None          # frequencies slowed down for lengths beyond the original one: a FrequencyBlend or
+                                            # a WavelengthBlend
 
 
 @dataclass(frozen=True)
@@ -79,13 +91,27 @@ class AttentionSpec:
     qk_row_norm: Optional[NormSpec] = None  # norm of ALL rows of q, and of k, at once before the rotation (weights 'q.norm'
                                             # and 'k.norm' as long as the projections); its ``size`` is not used
 
+    keep_first: int = 0                     # with a window: the first so many positions stay visible too
+    values_are_keys: bool = False           # no value tensor: the values are the keys as projected, before norm and rotation
+    feature_gate: bool = False              # the heads side by side are multiplied by sigmoid(W_g x), feature by feature
+    difference: Optional[float] = None      # differential attention: a head's q and k are two maps of ``head_dim`` features
+                                            # each (side by side), with a softmax each over the same values;
+                                            # o = a1 - lam a2, divided by its root mean square over the head's values
+                                            # (``difference_eps``), times 1 - difference, where
+                                            # lam = exp(lq1 . lk1) - exp(lq2 . lk2) + difference is one number a layer
+    difference_eps: float = 0.0
+
+    @property
+    def maps(self) -> int:
+        return 1 if self.difference is None else 2
+
     @property
     def q_size(self) -> int:
-        return self.num_heads * self.head_dim
+        return self.num_heads * self.maps * self.head_dim
 
     @property
     def kv_size(self) -> int:
-        return self.num_kv_heads * self.head_dim
+        return self.num_kv_heads * self.maps * self.head_dim
 
     @property
     def value_dim(self) -> int:
@@ -94,12 +120,14 @@ class AttentionSpec:
 
 @dataclass(frozen=True)
 class GatedMLPSpec:
-    """Dense gated feed-forward: down(act(gate(x)) * up(x)), no bias; act 'silu' or 'gelu_tanh' (the tanh form)."""
+    """Dense gated feed-forward: down(act(gate(x)) * up(x)); act 'silu' or 'gelu_tanh' (the tanh form). ``bias``: all three
+    projections have one (the tensor's name with '.b' added)."""
     hidden_size: int
     intermediate_size: int
     activation: str = "silu"
     kind: str = "gated_mlp"
     names: Tuple[str, str, str] = ("gate_proj.weight", "up_proj.weight", "down_proj.weight")    # gate, up, down
+    bias: bool = False
 
 
 @dataclass(frozen=True)
@@ -167,6 +195,8 @@ class ExpertsSpec:
     groups: int = 1                         # the experts form this many equal groups of neighbours; a group's score is its
     keep_groups: int = 1                    # best expert's, and only experts of the best ``keep_groups`` groups can be chosen
     weight_scale: float = 1.0               # a factor on the weights
+    table_rows: int = 0                     # > 0: no router: row i of a table [table_rows, top] of integers ('table') names
+                                            # the experts of token id i, each of weight 1 / top
     shared_gate: bool = False               # the shared expert's output is multiplied by sigmoid(w_sg . h), one number a token
 
 
@@ -323,6 +353,8 @@ class LayerSpec:
     one float32 stream: m is ``residual_mult``, s1 and s2 are vectors named by ``mixer_scale`` and ``feed_forward_scale``
     behind the layer's prefix (None: no such factor), and shift, named by ``token_shift``, replaces h_t by
     h_t + (h_(t-1) - h_t) * v per feature, the h before a request's first token being zero (None: no shift).
+    ``arrangement='parallel_residual'``: x += m * (mixer(norm1(x)) + feed_forward(norm1(x))) around one float32 stream: one norm,
+    which both sublayers read (``feed_forward_norm`` None).
     ``feed_forward`` None (with ``feed_forward_norm`` None): the block has a mixer only.
     ``mixer_out_norm`` / ``feed_forward_out_norm`` ('multi_stream' only): a second norm on the sublayer's OUTPUT
     before it is added, x += norm_b(sublayer(norm(x))); its ``tensor`` is the name behind the LAYER's prefix.
@@ -338,7 +370,7 @@ class LayerSpec:
     mixer_out_norm: Optional[NormSpec] = None
     feed_forward_out_norm: Optional[NormSpec] = None
     index: Optional[int] = None
-    residual_mult: float = 1.0                  # 'scaled_residual' only, like the three names below
+    residual_mult: float = 1.0                  # 'scaled_residual' and 'parallel_residual'; the three names below: the former only
     mixer_scale: Optional[str] = None
     feed_forward_scale: Optional[str] = None
     token_shift: Optional[str] = None
@@ -355,6 +387,8 @@ class ExecStep:
     writes_cache: bool = True
     adds_embedding: bool = False
     adds_vector: Optional[int] = None
+    projects_embedding: bool = False        # x <- W [x; x0] right before the layer, x0 the embedding's output and W
+                                            # ``ModelSpec.entry_projection``
 
 
 @dataclass(frozen=True)
@@ -382,6 +416,7 @@ class ModelSpec:
     tie_embeddings: bool
     max_positions: int
     names: TensorNames = field(default_factory=TensorNames)
+    entry_projection: Optional[str] = None  # tensor [hidden, 2 hidden] that entries with ``projects_embedding`` apply
     step_vectors: Optional[Tuple[str, int]] = None      # (tensor name, rows): vectors that entries of the run order add
 
     def __post_init__(self):
@@ -389,6 +424,8 @@ class ModelSpec:
         rows = self.step_vectors[1] if self.step_vectors else 0
         if any(s.adds_vector is not None and not 0 <= s.adds_vector < rows for s in self.execution):
             raise ValueError(f"the run order adds a vector that is not among the model's {rows}")
+        if any(s.projects_embedding for s in self.execution) and self.entry_projection is None:
+            raise ValueError("the run order projects the embedding, and the model names no tensor for that")
         for step in self.execution:
             if not 0 <= step.layer < len(self.layers):
                 raise ValueError(f"execution names layer {step.layer}, the model has {len(self.layers)}")

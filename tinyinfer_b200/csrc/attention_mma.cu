@@ -40,6 +40,8 @@ struct AttnParams {
     const int* token_seq;
     const int* block_table;
     int max_blocks, hq, hkv, page_size, num_pages, window, num_rows;
+    int keep;                      // > 0: a window keeps the first so many positions
+    float share, diff_eps;         // differential attention: what of the second map is subtracted, and its norm's eps
     int num_ctas;                  // CTAs of the split kernel: the runs are cut for this many
     float scale_log2;              // softmax scale times log2(e)
     float cap_log2, cap_arg;       // scores capped by a tanh (ti_score_log2); 0: not
@@ -47,7 +49,7 @@ struct AttnParams {
     float sink_log2, out_scale;    // out_scale multiplies the output before its rounding
     const float* head_sinks;         // float32 [query heads]: a sink's logit per head in place of sink_log2 (or null)
     const __nv_bfloat16* gate;       // rows of ld_gate, first column gate_off: out *= sigmoid(gate[token][head]) (or null)
-    int ld_gate, gate_off;
+    int ld_gate, gate_off, gate_each;
     int* status;
 };
 
@@ -120,30 +122,32 @@ __device__ __forceinline__ void load_tile(const CUtensorMap* map, const AttnPara
     }
 }
 
-// Zeroes the value rows of a tile outside [keep_lo, keep_hi) (tile-local key indices): no query of
+// Zeroes the value rows of a tile outside [keep_lo, keep_hi) and not before `first` (tile-local key indices): no query of
 // this CTA may see them and what the stage holds there may be stale or unwritten. Called by the
 // `nthreads` threads that will read the tile, `tid` being the caller's index among them.
 template <int D>
-__device__ __forceinline__ void zero_value_rows(uint8_t* v_tile, int keep_lo, int keep_hi, int tid, int nthreads,
+__device__ __forceinline__ void zero_value_rows(uint8_t* v_tile, int keep_lo, int keep_hi, int first, int tid, int nthreads,
                                                 int row_begin, int row_end) {
     constexpr int CHUNKS = D / 8;
     for (int idx = tid; idx < (row_end - row_begin) * CHUNKS; idx += nthreads) {
         const int row = row_begin + idx / CHUNKS, chunk = idx % CHUNKS;
-        if (row >= keep_lo && row < keep_hi) continue;
+        if ((row >= keep_lo || row < first) && row < keep_hi) continue;
         *reinterpret_cast<uint4*>(v_tile + tile_off(row, chunk)) = make_uint4(0, 0, 0, 0);
     }
 }
 
 // ------------------------------------------------------------------------------------ decode
 // Key tiles a decoded row has to read: those from the one its window (if any) begins in to its last.
-struct RowTiles { int n, lo_tile, lo, ctx, row; };
-__device__ __forceinline__ RowTiles row_tiles(const AttnParams& p, int r) {
+// (number 0 .. n - 1: the tiles of kept first positions, if any, then the window's; see ti_nth_tile).
+struct RowTiles { int n, lo_tile, lo, ctx, row, kept; };
+template <bool KEEP> __device__ __forceinline__ RowTiles row_tiles(const AttnParams& p, int r) {
     RowTiles t;
     t.row = p.rows[r];
     t.ctx = p.positions[t.row] + 1;
     t.lo = ti_first_key(t.ctx - 1, p.window);
     t.lo_tile = t.lo / TK;
-    t.n = (t.ctx + TK - 1) / TK - t.lo_tile;
+    t.kept = KEEP ? ti_kept_tiles(p.keep, t.lo_tile, TK) : 0;
+    t.n = (t.ctx + TK - 1) / TK - t.lo_tile + t.kept;
     return t;
 }
 // Tiles per run for `total` tiles (all kv heads) on `ctas` CTAs. (The tiles of a step are counted in 32 bits: a
@@ -180,8 +184,9 @@ __device__ __forceinline__ void block_scan(int mine, int* warp_sums /* [NT / 32]
 }
 
 // A CTA's walk over the parts of its run: the loading warp and the consumers step through the same parts.
-struct Part { int r, row, kvh, tile0, tile1, tile_new, k_begin, k_end, slot, pair, cta0, cta1; };   // tile_new: the tile of the row's own token; cta0..cta1: the CTAs whose runs hold the pair's tiles
-struct RunWalk {
+// tile0, tile1: numbers of the row's tiles; lo, ctx: the keys the row sees are lo .. ctx - 1, and those before keep.
+struct Part { int r, row, kvh, tile0, tile1, kept, lo_tile, tile_new, lo, ctx, slot, pair, cta0, cta1; };   // tile_new: the tile of the row's own token; cta0..cta1: the CTAs whose runs hold the pair's tiles
+template <bool KEEP> struct RunWalk {
     int cur, end, base;            // global tile indices; base: that of (row r, kv head 0, its first tile)
     int r, per;
     RowTiles rt;
@@ -189,16 +194,17 @@ struct RunWalk {
         if (cur >= end) return false;
         while (cur - base >= p.hkv * rt.n) {                   // on to the next decoded row
             base += p.hkv * rt.n;
-            rt = row_tiles(p, ++r);
+            rt = row_tiles<KEEP>(p, ++r);
         }
         const int off = cur - base;
         const int kvh = off / rt.n, tl = off % rt.n;
         const int cnt = min(rt.n - tl, end - cur);
         part.r = r; part.row = rt.row; part.kvh = kvh;
-        part.tile0 = rt.lo_tile + tl; part.tile1 = part.tile0 + cnt;
+        part.tile0 = tl; part.tile1 = tl + cnt;
+        part.kept = rt.kept; part.lo_tile = rt.lo_tile;
         part.tile_new = (rt.ctx - 1) / TK;
-        part.k_begin = max(rt.lo, part.tile0 * TK);
-        part.k_end = min(rt.ctx, part.tile1 * TK);
+        part.lo = rt.lo;
+        part.ctx = rt.ctx;
         part.pair = r * p.hkv + kvh;
         part.slot = (int)blockIdx.x + part.pair;               // CTA and pair both only grow along the walk: no two parts share a slot
         const int first = base + kvh * rt.n;                   // the pair's first tile
@@ -220,10 +226,17 @@ struct RunWalk {
 // two CTAs of 8 or 9 query heads a kv head (head size 128) share an SM (32 requests x 8,192 keys, 64 query heads
 // over 8: 193 -> 170 us); with fewer query heads, where two CTAs fit anyway, the whole buffer's merge is shorter
 // (8 x 4,096 keys, 32 over 8: 26.9 us against 30.0).
-template <int D, int NS, bool SLIM, bool CAP>
+// MAPS 2, differential attention: a query head and a key head hold two maps' features side by side, D / 2 each, and every map
+// is a softmax of its own over the same values of D features. A row of the MMA then is a (query head, map), its query zero in
+// the other map's half: the product with a whole key row gives the map's own score, and the bytes of a key and a value serve
+// both maps. Every part is left to the merge kernel, which subtracts the maps of a head from one another.
+// FORM: 0 plain; 1 with what a window keeps and a gate per feature; 2 the same for two maps.
+template <int D, int NS, bool SLIM, bool CAP, int FORM>
 __global__ void __launch_bounds__(THREADS) decode_attention_kernel(const __grid_constant__ CUtensorMap kv_map,
                                                                    const AttnParams p) {
     using S = Smem<D>;
+    constexpr bool KEEP = FORM != 0;
+    constexpr int MAPS = FORM == 2 ? 2 : 1;
     constexpr int STAGES = NS;                             // hides the file's constant in this kernel
     constexpr int LDW = D + 2;                             // whole merge buffer row: D outputs, maximum, sum
     constexpr int OWN = D / 4, NB_OWN = OWN / 8;           // slim: features (and 8-wide blocks of them) a warp finishes
@@ -239,7 +252,7 @@ __global__ void __launch_bounds__(THREADS) decode_attention_kernel(const __grid_
     volatile int* abort_flag = &abort_sh;
 
     ti_grid_launch_dependents();
-    const int group = p.hq / p.hkv;
+    const int group = p.hq / p.hkv * MAPS;                 // rows of the MMA
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (threadIdx.x == 0) {
         abort_sh = 0;
@@ -251,7 +264,7 @@ __global__ void __launch_bounds__(THREADS) decode_attention_kernel(const __grid_
     const int stretch = (p.num_rows + THREADS - 1) / THREADS;
     const int my_r0 = min(p.num_rows, (int)threadIdx.x * stretch), my_r1 = min(p.num_rows, my_r0 + stretch);
     int mine = 0;
-    for (int r = my_r0; r < my_r1; ++r) mine += row_tiles(p, r).n;
+    for (int r = my_r0; r < my_r1; ++r) mine += row_tiles<KEEP>(p, r).n;
     int before, total;
     block_scan<THREADS>(mine, warp_sums, before, total);
     const int all_tiles = all_tiles_of(total, p.hkv);
@@ -266,17 +279,17 @@ __global__ void __launch_bounds__(THREADS) decode_attention_kernel(const __grid_
     if (run_begin < all_tiles && run_begin >= before * p.hkv && run_begin < (before + mine) * p.hkv) {
         int acc = before;
         for (int r = my_r0; r < my_r1; ++r) {
-            const int n = row_tiles(p, r).n;
+            const int n = row_tiles<KEEP>(p, r).n;
             if (run_begin < (acc + n) * p.hkv) { start_sh[0] = r; start_sh[1] = acc; break; }
             acc += n;
         }
     }
     __syncthreads();
     if (run_begin >= all_tiles) return;                    // more CTAs than runs
-    RunWalk walk;
+    RunWalk<KEEP> walk;
     walk.cur = run_begin; walk.end = run_end; walk.r = start_sh[0]; walk.per = per;
     walk.base = start_sh[1] * p.hkv;
-    walk.rt = row_tiles(p, walk.r);
+    walk.rt = row_tiles<KEEP>(p, walk.r);
 
     if (warp == 4) {
         // The kernel just before wrote this step's keys and values: for a decoded row that is its own token, in
@@ -289,7 +302,8 @@ __global__ void __launch_bounds__(THREADS) decode_attention_kernel(const __grid_
             Part it;
             while (ok && walk.next(p, it)) {
                 const int* table = p.block_table + (size_t)p.token_seq[it.row] * p.max_blocks;
-                for (int t = it.tile0; t < it.tile1; ++t, ++n) {
+                for (int v = it.tile0; v < it.tile1; ++v, ++n) {
+                    const int t = KEEP ? ti_nth_tile(v, it.kept, it.lo_tile) : it.lo_tile + v;
                     if (!waited && (n >= STAGES || t == it.tile_new)) { ti_grid_wait(); waited = true; }
                     const int s = n % STAGES;
                     if (!mbar_wait(bar0 + 8u * (STAGES + s), ((n / STAGES) & 1u) ^ 1u, abort_flag, p.status, 21)) { ok = false; break; }
@@ -309,7 +323,18 @@ __global__ void __launch_bounds__(THREADS) decode_attention_kernel(const __grid_
     while (walk.next(p, item)) {
         uint32_t qa[D / 16][4];
         {
-            const __nv_bfloat16* q0 = p.q + ((size_t)item.row * p.hq + (size_t)item.kvh * group) * D;
+            const __nv_bfloat16* q0 = p.q + ((size_t)item.row * p.hq + (size_t)item.kvh * (group / MAPS)) * D;
+            if constexpr (MAPS == 2) {                         // row g: map g & 1 of head g >> 1; rows g and g + 8 are one map
+#pragma unroll
+                for (int ks = 0; ks < D / 16; ++ks) {
+                    const bool own = (ks >= D / 32) == (g & 1);
+                    const __nv_bfloat16* qa0 = q0 + (size_t)(g >> 1) * D + ks * 16 + c;
+                    qa[ks][0] = own && g < group ? *reinterpret_cast<const uint32_t*>(qa0) : 0u;
+                    qa[ks][1] = own && g + 8 < group ? *reinterpret_cast<const uint32_t*>(qa0 + 4 * D) : 0u;
+                    qa[ks][2] = own && g < group ? *reinterpret_cast<const uint32_t*>(qa0 + 8) : 0u;
+                    qa[ks][3] = own && g + 8 < group ? *reinterpret_cast<const uint32_t*>(qa0 + 4 * D + 8) : 0u;
+                }
+            } else
 #pragma unroll
             for (int ks = 0; ks < D / 16; ++ks) {
                 qa[ks][0] = g < group ? *reinterpret_cast<const uint32_t*>(q0 + (size_t)g * D + ks * 16 + c) : 0u;
@@ -322,16 +347,17 @@ __global__ void __launch_bounds__(THREADS) decode_attention_kernel(const __grid_
 #pragma unroll
         for (int i = 0; i < D / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
         float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
-        const int k_begin = item.k_begin, k_end = item.k_end;
+        const int k_begin = item.lo, k_end = item.ctx, keep = KEEP ? p.keep : 0;
 
-        for (int t = item.tile0; t < item.tile1; ++t, ++n) {
+        for (int v = item.tile0; v < item.tile1; ++v, ++n) {
+            const int t = KEEP ? ti_nth_tile(v, item.kept, item.lo_tile) : item.lo_tile + v;
             const int s = n % STAGES;
             if (!mbar_wait(bar0 + 8u * s, (n / STAGES) & 1u, abort_flag, p.status, 22)) return;
             uint8_t* k_tile = smem + s * S::STAGE_BYTES;
             uint8_t* v_tile = k_tile + S::TILE_BYTES;
             const int w0 = warp * 16;                         // this warp's 16 keys of the tile
             const int tok0 = t * TK + w0;
-            if (tok0 < k_end && tok0 + 16 > k_begin) {
+            if (tok0 < k_end && (tok0 + 16 > k_begin || tok0 < keep)) {
                 float sc[2][4] = {};
 #pragma unroll
                 for (int ks = 0; ks < D / 16; ++ks) {
@@ -347,9 +373,9 @@ __global__ void __launch_bounds__(THREADS) decode_attention_kernel(const __grid_
 #pragma unroll
                     for (int j = 0; j < 4; ++j) {
                         const int tok = tok0 + nb * 8 + c + (j & 1);
-                        const float v = (tok >= k_begin && tok < k_end) ? ti_score_log2<CAP>(p, sc[nb][j]) : -INFINITY;
-                        sc[nb][j] = v;
-                        mx[j >> 1] = fmaxf(mx[j >> 1], v);
+                        const float s2 = ((tok >= k_begin || tok < keep) && tok < k_end) ? ti_score_log2<CAP>(p, sc[nb][j]) : -INFINITY;
+                        sc[nb][j] = s2;
+                        mx[j >> 1] = fmaxf(mx[j >> 1], s2);
                     }
                 float corr[2], m_use[2];
 #pragma unroll
@@ -373,7 +399,7 @@ __global__ void __launch_bounds__(THREADS) decode_attention_kernel(const __grid_
                 uint32_t pa[4] = {pack_bf16(sc[0][0], sc[0][1]), pack_bf16(sc[0][2], sc[0][3]),
                                   pack_bf16(sc[1][0], sc[1][1]), pack_bf16(sc[1][2], sc[1][3])};
                 if (tok0 < k_begin || tok0 + 16 > k_end) {    // warp-local: only this warp reads these rows
-                    zero_value_rows<D>(v_tile, k_begin - t * TK, k_end - t * TK, lane, 32, w0, w0 + 16);
+                    zero_value_rows<D>(v_tile, k_begin - t * TK, k_end - t * TK, keep - t * TK, lane, 32, w0, w0 + 16);
                     asm volatile("fence.proxy.async.shared::cta;" ::: "memory");   // a later TMA copy overwrites these rows
                     __syncwarp();
                 }
@@ -434,11 +460,12 @@ __global__ void __launch_bounds__(THREADS) decode_attention_kernel(const __grid_
                     acc += f * mbuf[((size_t)w4 * group + hrow) * LDW + d];
                     l_all += f * mbuf[((size_t)w4 * group + hrow) * LDW + D + 1];
                 }
-                if (item.cta0 == item.cta1) {                      // the pair lies inside this run: this is its result
+                if (MAPS == 1 && item.cta0 == item.cta1) {         // the pair lies inside this run: this is its result
                     const int head = item.kvh * group + hrow;
                     const float l_fin = p.has_sink ? l_all + exp2f(ti_sink_log2(p, head) - m_all) : l_all;
-                    p.out[((size_t)item.row * p.hq + head) * D + d] =
-                        __float2bfloat16_rn(l_fin > 0.f ? acc * ti_head_out_scale(p, item.row, head) / l_fin : 0.f);
+                    float res = l_fin > 0.f ? acc * ti_head_out_scale(p, item.row, head) / l_fin : 0.f;
+                    if constexpr (KEEP) ti_gate_features<1>(p, item.row, head, D, d, &res);
+                    p.out[((size_t)item.row * p.hq + head) * D + d] = __float2bfloat16_rn(res);
                 } else {
                     const size_t slot = (size_t)item.slot * group + hrow;
                     __stcg(p.part_o + slot * D + d, acc);
@@ -495,8 +522,9 @@ __global__ void __launch_bounds__(THREADS) decode_attention_kernel(const __grid_
 #pragma unroll
             for (int w4 = 0; w4 < 4; ++w4) { f[w4] = exp2f(mw[w4] - m_use); l_all += f[w4] * lw[w4]; }
             const int head = item.kvh * group + hrow;
-            const float l_fin = p.has_sink ? l_all + exp2f(ti_sink_log2(p, head) - m_all) : l_all;       // used where the result is final
-            const float inv = l_fin > 0.f ? (item.cta0 == item.cta1 ? ti_head_out_scale(p, item.row, head) : 1.f) / l_fin : 0.f;
+            const bool final_part = MAPS == 1 && item.cta0 == item.cta1;
+            const float l_fin = p.has_sink && MAPS == 1 ? l_all + exp2f(ti_sink_log2(p, head) - m_all) : l_all;       // used where the result is final
+            const float inv = l_fin > 0.f ? (final_part ? ti_head_out_scale(p, item.row, head) : 1.f) / l_fin : 0.f;
 #pragma unroll
             for (int nb = 0; nb < D / 8; ++nb) {               // every block, so that the accumulator's index is a constant
                 if (nb / NB_OWN != warp) continue;
@@ -510,15 +538,17 @@ __global__ void __launch_bounds__(THREADS) decode_attention_kernel(const __grid_
                     a0 += f[w4] * x0;
                     a1 += f[w4] * x1;
                 }
-                if (item.cta0 == item.cta1) {                  // the pair lies inside this run: this is its result
-                    *reinterpret_cast<__nv_bfloat162*>(p.out + ((size_t)item.row * p.hq + (size_t)item.kvh * group + hrow) * D + d) =
-                        __floats2bfloat162_rn(a0 * inv, a1 * inv);
+                if (final_part) {                              // the pair lies inside this run: this is its result
+                    float res[2] = {a0 * inv, a1 * inv};
+                    if constexpr (KEEP) ti_gate_features<2>(p, item.row, head, D, d, res);
+                    *reinterpret_cast<__nv_bfloat162*>(p.out + ((size_t)item.row * p.hq + head) * D + d) =
+                        __floats2bfloat162_rn(res[0], res[1]);
                 } else {
                     const size_t slot = (size_t)item.slot * group + hrow;
                     __stcg(reinterpret_cast<float2*>(p.part_o + slot * D + d), make_float2(a0, a1));
                 }
             }
-            if (item.cta0 != item.cta1 && warp == 0 && (lane & 3) == 0)
+            if (!final_part && warp == 0 && (lane & 3) == 0)
                 __stcg(reinterpret_cast<float2*>(p.part_ml + ((size_t)item.slot * group + hrow) * 2), make_float2(m_all, l_all));
         }
         }   // SLIM
@@ -532,14 +562,19 @@ __global__ void __launch_bounds__(THREADS) decode_attention_kernel(const __grid_
 // sum and output. (Merging inside the split kernel, by the CTA that counts itself in last, was slower by
 // 3 to 5 us at 1 to 8 long requests: while the kernel streams, the release that publishes a CTA's
 // partials waits microseconds for its stores.)
-template <int D>
+// MAPS 2: the block merges both maps of its head, whose parts every CTA has left here, and finishes the head: with a1 and a2
+// the maps' outputs, o = a1 - share * a2, divided by its root mean square over the D features, times the output's factor.
+template <int D, int FORM>
 __global__ void decode_merge_kernel(const AttnParams p) {
+    constexpr bool KEEP = FORM != 0;
+    constexpr int MAPS = FORM == 2 ? 2 : 1;
     __shared__ int warp_sums[D / 32];
+    __shared__ float red[33];
     ti_grid_launch_dependents();
     const int r = blockIdx.x, h = blockIdx.y, d = threadIdx.x;
     int mine = 0, mine_before = 0;
     for (int r2 = d; r2 < p.num_rows; r2 += D) {
-        const int n = row_tiles(p, r2).n;
+        const int n = row_tiles<KEEP>(p, r2).n;
         mine += n;
         if (r2 < r) mine_before += n;
     }
@@ -547,45 +582,61 @@ __global__ void decode_merge_kernel(const AttnParams p) {
     block_scan<D>(mine, warp_sums, skip, total);
     __syncthreads();
     block_scan<D>(mine_before, warp_sums, skip, tiles_before);
-    const RowTiles rt = row_tiles(p, r);
-    const int group = p.hq / p.hkv, kvh = h / group, hrow = h % group;
+    const RowTiles rt = row_tiles<KEEP>(p, r);
+    const int heads = p.hq / p.hkv, kvh = h / heads, hrow = h % heads, group = heads * MAPS;
     const int all_tiles = all_tiles_of(total, p.hkv);
     if (all_tiles < 0) return;                             // the split kernel has said so
     const int per = run_tiles(all_tiles, p.num_ctas);
     const int first = tiles_before * p.hkv + kvh * rt.n;                                   // the pair's tiles, globally
     const int c0 = first / per, c1 = (first + rt.n - 1) / per;
-    if (c0 == c1) return;
+    if (MAPS == 1 && c0 == c1) return;
     const int pair = r * p.hkv + kvh;
     ti_grid_wait();
-    float m_run = -INFINITY, acc = 0.f, l_all = 0.f;
-    for (int cb = c0; cb <= c1; cb += 8) {
-        float ms[8], ls[8], os[8];
+    float m_run[MAPS], acc[MAPS], l_all[MAPS];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
-            const bool in = cb + j <= c1;
-            const size_t slot = (size_t)(cb + j + pair) * group + hrow;
-            const float2 ml = in ? __ldcg(reinterpret_cast<const float2*>(p.part_ml + slot * 2)) : make_float2(-INFINITY, 0.f);
-            ms[j] = ml.x;
-            ls[j] = ml.y;
-            os[j] = in ? __ldcg(p.part_o + slot * D + d) : 0.f;
+    for (int mp = 0; mp < MAPS; ++mp) { m_run[mp] = -INFINITY; acc[mp] = 0.f; l_all[mp] = 0.f; }
+    constexpr int AT_ONCE = 8 / MAPS;
+    for (int cb = c0; cb <= c1; cb += AT_ONCE) {
+        float ms[MAPS][AT_ONCE], ls[MAPS][AT_ONCE], os[MAPS][AT_ONCE];
+#pragma unroll
+        for (int mp = 0; mp < MAPS; ++mp)
+#pragma unroll
+            for (int j = 0; j < AT_ONCE; ++j) {
+                const bool in = cb + j <= c1;
+                const size_t slot = (size_t)(cb + j + pair) * group + hrow * MAPS + mp;
+                const float2 ml = in ? __ldcg(reinterpret_cast<const float2*>(p.part_ml + slot * 2)) : make_float2(-INFINITY, 0.f);
+                ms[mp][j] = ml.x;
+                ls[mp][j] = ml.y;
+                os[mp][j] = in ? __ldcg(p.part_o + slot * D + d) : 0.f;
+            }
+#pragma unroll
+        for (int mp = 0; mp < MAPS; ++mp) {
+            float m_new = m_run[mp];
+#pragma unroll
+            for (int j = 0; j < AT_ONCE; ++j) m_new = fmaxf(m_new, ms[mp][j]);
+            const float m_use = m_new == -INFINITY ? 0.f : m_new;
+            const float keep = exp2f(m_run[mp] - m_use);      // 0 while nothing has been merged yet
+            acc[mp] *= keep;
+            l_all[mp] *= keep;
+#pragma unroll
+            for (int j = 0; j < AT_ONCE; ++j) {
+                const float f = exp2f(ms[mp][j] - m_use);      // 0 for a part that is not there
+                acc[mp] += f * os[mp][j];
+                l_all[mp] += f * ls[mp][j];
+            }
+            m_run[mp] = m_new;
         }
-        float m_new = m_run;
-#pragma unroll
-        for (int j = 0; j < 8; ++j) m_new = fmaxf(m_new, ms[j]);
-        const float m_use = m_new == -INFINITY ? 0.f : m_new;
-        const float keep = exp2f(m_run - m_use);          // 0 while nothing has been merged yet
-        acc *= keep;
-        l_all *= keep;
-#pragma unroll
-        for (int j = 0; j < 8; ++j) {
-            const float f = exp2f(ms[j] - m_use);          // 0 for a part that is not there
-            acc += f * os[j];
-            l_all += f * ls[j];
-        }
-        m_run = m_new;
     }
-    if (p.has_sink) l_all += exp2f(ti_sink_log2(p, h) - m_run);
-    p.out[((size_t)rt.row * p.hq + h) * D + d] = __float2bfloat16_rn(l_all > 0.f ? acc * ti_head_out_scale(p, rt.row, h) / l_all : 0.f);
+    float res;
+    if constexpr (MAPS == 1) {
+        if (p.has_sink) l_all[0] += exp2f(ti_sink_log2(p, h) - m_run[0]);
+        res = l_all[0] > 0.f ? acc[0] * ti_head_out_scale(p, rt.row, h) / l_all[0] : 0.f;
+    } else {
+        res = (l_all[0] > 0.f ? acc[0] / l_all[0] : 0.f) - (l_all[1] > 0.f ? acc[1] * p.share / l_all[1] : 0.f);
+        res *= ti_head_out_scale(p, rt.row, h) * rsqrtf(block_sum(res * res, red) / (float)D + p.diff_eps);
+    }
+    if constexpr (KEEP) ti_gate_features<1>(p, rt.row, h, D, d, &res);
+    p.out[((size_t)rt.row * p.hq + h) * D + d] = __float2bfloat16_rn(res);
 }
 
 template <typename K>
@@ -616,7 +667,7 @@ namespace {
 // is too. nullptr: no current device.
 int* configured_bytes(int which) {
     constexpr int MAX_DEVICES = 64;
-    static int bytes[8][MAX_DEVICES] = {};
+    static int bytes[24][MAX_DEVICES] = {};
     int dev = -1;
     if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= MAX_DEVICES) return nullptr;
     return &bytes[which][dev];
@@ -669,18 +720,24 @@ TI_API long long ti_attention_decode_scratch_floats(int num_rows, int hq, int hk
 // they must be complete when the call is made, not results of the kernels launched just before (those may
 // write q and the keys and values at the rows' own positions). Calls that share the scratch must not overlap.
 // has_sink: exp(sink) joins every softmax denominator without a value; out_scale: a factor on the output;
-// head_sinks, gate: a sink per query head, and a sigmoid gate per (token, query head) on the output (or null).
+// head_sinks, gate: a sink per query head, and a sigmoid gate per (token, query head) on the output (or null), per output
+// feature with gate_each; keep: a window keeps the first so many positions. maps 2: differential attention (share, diff_eps;
+// see decode_merge_kernel), hq query heads of two maps of d / 2 features, scratch for 2 hq heads.
 TI_API int ti_attention_decode_sink_bf16(void* out, const void* q, const void* kv_cache, float* scratch, long long scratch_floats,
                                          const int* rows, int num_rows, const int* positions, const int* token_seq,
                                          const int* block_table, int max_blocks, int hq, int hkv, int d, int page_size,
-                                         int num_pages, float scale, int window, int max_context, int has_sink, float sink,
+                                         int num_pages, float scale, int window, int keep, int max_context, int has_sink, float sink,
                                          float out_scale, const float* head_sinks, const void* gate, int ld_gate, int gate_off,
-                                         float softcap, int* status, cudaStream_t stream) {
-    if (check_shape(hq, hkv, d, page_size, "attention_decode")) return -1;
+                                         int gate_each, float softcap, int maps, float share, float diff_eps, int* status,
+                                         cudaStream_t stream) {
+    TI_REQUIRE(maps == 1 || (maps == 2 && !has_sink && !head_sinks), "attention_decode: one map, or two without sinks");
+    if (check_shape(hq * maps, hkv, d, page_size, "attention_decode")) return -1;
+    TI_REQUIRE(keep >= 0 && (!gate || !gate_each || (((uintptr_t)gate & 15) == 0 && ld_gate % 8 == 0 && gate_off % 8 == 0)),
+               "attention_decode: a gate per feature lies on 16-byte boundaries");
     TI_REQUIRE(num_rows >= 0 && num_rows <= 65535 && max_context > 0, "attention_decode: bad sizes");
     if (num_rows == 0) return 0;
-    const int group = hq / hkv;
-    const int ctas = ti_attention_decode_ctas(num_rows, hq, hkv, d, max_context, window);
+    const int group = hq / hkv * maps;
+    const int ctas = ti_attention_decode_ctas(num_rows, hq * maps, hkv, d, max_context, window);
     const long long slots = (long long)ctas + (long long)num_rows * hkv;
     TI_REQUIRE(slots * group * (d + 2) <= scratch_floats,
                "attention_decode: %d rows x %d kv heads on %d CTAs need %lld floats of scratch, %lld given",
@@ -696,35 +753,40 @@ TI_API int ti_attention_decode_sink_bf16(void* out, const void* q, const void* k
     TI_SET_SCORE_CAP(p, scale, softcap);
     p.has_sink = has_sink || head_sinks ? 1 : 0; p.sink_log2 = sink * 1.4426950408889634f; p.out_scale = out_scale;
     p.head_sinks = head_sinks; p.gate = (const __nv_bfloat16*)gate; p.ld_gate = ld_gate; p.gate_off = gate_off;
+    p.gate_each = gate_each; p.keep = keep; p.share = share; p.diff_eps = diff_eps;
     p.num_rows = num_rows; p.num_ctas = ctas;
-    // which: the record of configured_bytes; a capped kernel is another function and keeps a record of its own
-#define DEC_GO(D, NS, SLIM, CAP, which, bytes_expr)                                                                        \
+    // which: the record of configured_bytes; a capped kernel and the other forms are other functions and keep records of their own
+#define DEC_RUN(D, NS, SLIM, CAP, FORM, which, bytes_expr)                                                                 \
     do {                                                                                                                   \
         const int bytes = (bytes_expr);                                                                                    \
-        int* configured = configured_bytes((which) + ((CAP) ? 4 : 0));                                                     \
+        int* configured = configured_bytes((which) + ((CAP) ? 4 : 0) + 8 * (FORM));                                        \
         TI_REQUIRE(configured != nullptr, "attention_decode: no current device");                                          \
         if (*configured < bytes) {                                                                                         \
-            if (set_smem(decode_attention_kernel<D, NS, SLIM, CAP>, bytes, "attention_decode")) return -1;                 \
+            if (set_smem(decode_attention_kernel<D, NS, SLIM, CAP, FORM>, bytes, "attention_decode")) return -1;           \
             *configured = bytes;                                                                                           \
         }                                                                                                                  \
-        ti_launch(decode_attention_kernel<D, NS, SLIM, CAP>, ctas, THREADS, bytes, stream, map, p);                        \
+        ti_launch(decode_attention_kernel<D, NS, SLIM, CAP, FORM>, ctas, THREADS, bytes, stream, map, p);                  \
         TI_CHECK_LAUNCH("attention_decode");                                                                               \
-        ti_launch(decode_merge_kernel<D>, dim3(num_rows, hq), D, 0, stream, p);                                            \
+        ti_launch(decode_merge_kernel<D, FORM>, dim3(num_rows, hq), D, 0, stream, p);                                      \
+    } while (0)
+#define DEC_FORM(D, NS, SLIM, CAP, which, bytes_expr)                                    \
+    do {                                                                                 \
+        if (maps == 2) DEC_RUN(D, NS, SLIM, CAP, 2, which, bytes_expr);                  \
+        else if (keep > 0 || (gate && gate_each)) DEC_RUN(D, NS, SLIM, CAP, 1, which, bytes_expr); \
+        else DEC_RUN(D, NS, SLIM, CAP, 0, which, bytes_expr);                            \
+    } while (0)
+#define DEC_GO(D, NS, SLIM, which, bytes_expr)                           \
+    do {                                                                 \
+        if (capped) DEC_FORM(D, NS, SLIM, true, which, bytes_expr);      \
+        else DEC_FORM(D, NS, SLIM, false, which, bytes_expr);            \
     } while (0)
     const bool capped = p.cap_log2 > 0.f;
-    if (d == 128 && decode_form(group) == 2) {
-        if (capped) DEC_GO(128, 2 * STAGES, false, true, 2, Smem<128>::decode_bytes(group, 2 * STAGES));
-        else DEC_GO(128, 2 * STAGES, false, false, 2, Smem<128>::decode_bytes(group, 2 * STAGES));
-    } else if (d == 128 && decode_form(group) == 1) {
-        if (capped) DEC_GO(128, STAGES, true, true, 3, Smem<128>::decode_bytes(group, STAGES, true));
-        else DEC_GO(128, STAGES, true, false, 3, Smem<128>::decode_bytes(group, STAGES, true));
-    } else if (d == 128) {
-        if (capped) DEC_GO(128, STAGES, false, true, 0, Smem<128>::decode_bytes(group));
-        else DEC_GO(128, STAGES, false, false, 0, Smem<128>::decode_bytes(group));
-    } else {
-        if (capped) DEC_GO(64, STAGES, false, true, 1, Smem<64>::decode_bytes(group));
-        else DEC_GO(64, STAGES, false, false, 1, Smem<64>::decode_bytes(group));
-    }
+    if (d == 128 && decode_form(group) == 2) DEC_GO(128, 2 * STAGES, false, 2, Smem<128>::decode_bytes(group, 2 * STAGES));
+    else if (d == 128 && decode_form(group) == 1) DEC_GO(128, STAGES, true, 3, Smem<128>::decode_bytes(group, STAGES, true));
+    else if (d == 128) DEC_GO(128, STAGES, false, 0, Smem<128>::decode_bytes(group));
+    else DEC_GO(64, STAGES, false, 1, Smem<64>::decode_bytes(group));
+#undef DEC_FORM
+#undef DEC_RUN
 #undef DEC_GO
     TI_CHECK_LAUNCH("attention_decode_merge");
     return 0;
@@ -736,8 +798,8 @@ TI_API int ti_attention_decode_bf16(void* out, const void* q, const void* kv_cac
                                     int num_pages, float scale, int window, int max_context, int* status,
                                     cudaStream_t stream) {
     return ti_attention_decode_sink_bf16(out, q, kv_cache, scratch, scratch_floats, rows, num_rows, positions, token_seq,
-                                         block_table, max_blocks, hq, hkv, d, page_size, num_pages, scale, window, max_context,
-                                         0, 0.f, 1.f, nullptr, nullptr, 0, 0, 0.f, status, stream);
+                                         block_table, max_blocks, hq, hkv, d, page_size, num_pages, scale, window, 0, max_context,
+                                         0, 0.f, 1.f, nullptr, nullptr, 0, 0, 0, 0.f, 1, 0.f, 0.f, status, stream);
 }
 
 // ------------------------------------------------------------------------------------------------

@@ -37,6 +37,14 @@
 // share of the exponentials as a polynomial of degree 5 on the FMA pipe (every fourth: 547 us, every
 // eighth: 576, every second: 690; the softmax warps are short of issue slots as much as of the XU pipe).
 //
+// FORM 1, a window that keeps first positions, or a gate per feature: the key tiles are numbered without a gap, first the kept ones, which both
+// query tiles read, then the window's. FORM 2, differential attention: a query head and a key head hold two maps' features
+// side by side, D / 2 each. A CTA owns 128 query tokens; A and B are the two MAPS of the same rows, S_X multiplies only map
+// X's half of the features, both read the same values, and at the end two threads share a row: o = O_A / l_A - share *
+// O_B / l_B straight from tensor memory, divided by its root mean square, times the output's factor. Twice the softmax and
+// twice the P V of one map for one trip of the keys and values, with the tensor cores busy on one map while the other is in
+// its softmax, exactly as with two query tiles.
+//
 // Masked scores never reach an exponential (P is assigned 0 there), rows of V that no query of the CTA
 // may see are zeroed in shared memory before the second product (pages never written or given back cannot
 // leak NaNs through 0 * NaN), and every mbarrier wait is bounded (status word, abort flag, tensor memory
@@ -58,13 +66,16 @@ struct PairParams {
     const int* tiles;                // int4 {request index, first flat row, rows (<= 256), first position}
     const int* block_table;
     int max_blocks, hq, hkv, page_size, num_pages, window;
+    int keep;                        // > 0: a window keeps the first so many positions (FORM 1 and 2)
+    int halves;                      // FORM 2: 1: a tile entry has up to 256 rows and two CTAs take 128 each
+    float share, diff_eps;           // FORM 2: what of the second map is subtracted, and the norm's eps
     float scale_log2;
     float cap_log2, cap_arg;         // scores capped by a tanh (ti_score_log2); 0: not
     int has_sink;                    // the softmax denominator holds one more term 2^sink_log2 that has no value
     float sink_log2, out_scale;      // out_scale multiplies the output before its rounding
     const float* head_sinks;         // float32 [query heads]: a sink's logit per head in place of sink_log2 (or null)
     const __nv_bfloat16* gate;       // rows of ld_gate, first column gate_off: out *= sigmoid(gate[token][head]) (or null)
-    int ld_gate, gate_off;
+    int ld_gate, gate_off, gate_each;
     int* status;
 };
 
@@ -121,7 +132,7 @@ __device__ __forceinline__ void tmem_st32(uint32_t taddr, const uint32_t* r) {
 }
 __device__ __forceinline__ void tmem_wait_st() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 
-template <int D, bool CAP>
+template <int D, bool CAP, int FORM>
 __global__ void __launch_bounds__(PP_THREADS, 1)
 prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap kv_map,
                               const PairParams p) {
@@ -141,6 +152,7 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap q_map, const _
     auto o_full = [&](int x) { return bar0 + 8u * (5 + 2 * NBUF + x); };
     __shared__ uint32_t tmem_base_sh;
     __shared__ int abort_sh;
+    __shared__ float inv_sh[FORM == 2 ? 2 : 1][FORM == 2 ? QM : 1], ss_sh[FORM == 2 ? 2 : 1][FORM == 2 ? QM : 1];
     volatile int* abort_flag = &abort_sh;
 
     ti_grid_launch_dependents();
@@ -161,8 +173,11 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap q_map, const _
 
     // heads along x, tiles (longest key range first) along y: CTAs are handed out x first, so every head of
     // the longest tile starts before any shorter tile does, and the short ones fill in behind
-    const int4 td = reinterpret_cast<const int4*>(p.tiles)[blockIdx.y];
-    const int seq = td.x, row0 = td.y, nrows = td.z, pos0 = td.w;
+    const int4 td = reinterpret_cast<const int4*>(p.tiles)[FORM == 2 && p.halves ? blockIdx.y >> 1 : blockIdx.y];
+    const int half_off = FORM == 2 && p.halves ? (blockIdx.y & 1) * QM : 0;
+    const int seq = td.x, row0 = td.y + half_off, pos0 = td.w + half_off;
+    const int nrows = FORM == 2 ? min(td.z - half_off, QM) : td.z;       // FORM 2: may be none (an entry of at most 128 rows)
+    constexpr int ROWS_APART = FORM == 2 ? 0 : QM;                       // B's rows behind A's
     const int head = blockIdx.x;
     const int kvh = head / (p.hq / p.hkv);
     const int* table = p.block_table + (size_t)seq * p.max_blocks;
@@ -172,37 +187,47 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap q_map, const _
     int t0x[2], t1x[2];
 #pragma unroll
     for (int x = 0; x < 2; ++x) {
-        const int rows_x = min(QM, nrows - x * QM);
+        const int rows_x = min(QM, nrows - x * ROWS_APART);
         if (rows_x <= 0) { t0x[x] = 0; t1x[x] = 0; continue; }
-        const int first = pos0 + x * QM, hi_x = first + rows_x;
+        const int first = pos0 + x * ROWS_APART, hi_x = first + rows_x;
         const int lo_x = ti_first_key(first, p.window);
         t0x[x] = lo_x / KT;
         t1x[x] = (hi_x + KT - 1) / KT;
     }
     const bool has_b = t1x[1] > t0x[1];
     const int tmin = has_b ? min(t0x[0], t0x[1]) : t0x[0], tmax = has_b ? max(t1x[0], t1x[1]) : t1x[0];
+    // The CTA's tiles are numbered without a gap: 0 .. kept - 1 are those of kept first positions, number v >= kept is tile
+    // tmin + v - kept. Query tile X visits the kept ones and a run of the others that starts gap[X] tiles later (A's first key
+    // is never above B's, so gap[0] is 0): its i-th tile has number number_of(x, i), and it visits count[x] tiles.
+    const int kept = FORM == 0 ? 0 : ti_kept_tiles(p.keep, tmin, KT);
+    const int gap[2] = {t0x[0] - tmin, has_b ? t0x[1] - tmin : 0};
+    const int count[2] = {t1x[0] > t0x[0] ? kept + t1x[0] - t0x[0] : 0, has_b ? kept + t1x[1] - t0x[1] : 0};
+    auto number_of = [&](int x, int i) { return FORM != 0 && i < kept ? i : i + gap[x]; };
+    auto tile_of = [&](int v) { return FORM == 0 ? tmin + v : ti_nth_tile(v, kept, tmin); };
     const int lo = ti_first_key(pos0, p.window);                     // first key any query of the CTA sees
     const int hi = pos0 + nrows;                                     // one past the last
 
-    if (warp == 0) {
+    if (FORM == 2 && nrows <= 0) {
+        // nothing to do but the common exit
+    } else if (warp == 0) {
         // ------------------------------------------------------------ TMA producer
         if (lane == 0) {
-            mbar_expect_tx(q_full, (has_b ? 2u : 1u) * S::Q_BYTES);
+            mbar_expect_tx(q_full, (FORM != 2 && has_b ? 2u : 1u) * S::Q_BYTES);
 #pragma unroll
             for (int hh = 0; hh < S::HALVES; ++hh) {
                 tma_load_2d(smem_u32(q_tiles) + hh * (QM * 128), &q_map, q_full, head * D + hh * 64, row0);
-                if (has_b)
+                if (FORM != 2 && has_b)
                     tma_load_2d(smem_u32(q_tiles) + S::Q_BYTES + hh * (QM * 128), &q_map, q_full, head * D + hh * 64, row0 + QM);
             }
         }
-        // Load number i is K of tile tmin + i / 2 (i even) or V of it (i odd), into buffer i % NBUF. A tile is
+        // Load i is K of the tile number i / 2 (i even) or V of it (i odd), into buffer i % NBUF. A tile is
         // KT / piece_rows pieces (a piece lies in one page) x head halves: up to 16 copies, one a lane.
         const int piece_rows = p.page_size < 64 ? p.page_size : 64;
         const int num_copies = (KT / piece_rows) * S::HALVES;
         const int my_piece = lane / S::HALVES, my_half = lane % S::HALVES;
-        const int num_loads = 2 * (tmax - tmin);
+        const int num_loads = 2 * (kept + tmax - tmin);
         for (int i = 0; i < num_loads; ++i) {
-            const int j = tmin + (i >> 1), is_v = i & 1, b = i % NBUF;
+            const int j = tile_of(i >> 1), is_v = i & 1, b = i % NBUF;
             const int tok = j * KT + my_piece * piece_rows;
             const int logical = tok / p.page_size;
             int page = (lane < num_copies && logical < p.max_blocks) ? table[logical] : -1;
@@ -225,12 +250,18 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap q_map, const _
             constexpr uint32_t idesc_s = make_idesc(QM, KT);               // S = Q K^T: both operands K-major
             constexpr uint32_t idesc_o = make_idesc(QM, D, true);          // O = P V: V is MN-major (features contiguous)
             bool ok = mbar_wait(q_full, 0, abort_flag, p.status, 42);
-            int js[2] = {t0x[0], t0x[1]}, jp[2] = {t0x[0], t0x[1]};        // next S and next P V to issue, per query tile
+            int js[2] = {0, 0}, jp[2] = {0, 0};                            // next S and next P V to issue: query tile X's js[X]-th, jp[X]-th
             uint32_t spins = 0;
             unsigned long long idle_since = 0;
-            auto users = [&](int j) { return (j >= t0x[0] && j < t1x[0] ? 1 : 0) + (j >= t0x[1] && j < t1x[1] ? 1 : 0); };
-            auto issued = [&](const int* next, int j) { return (j >= t0x[0] && j < t1x[0] && next[0] > j ? 1 : 0) +
-                                                               (j >= t0x[1] && j < t1x[1] && next[1] > j ? 1 : 0); };
+            // which of X's tiles number v is, or -1 if X does not visit it
+            auto place_of = [&](int x, int v) {
+                const int i = FORM != 0 && v < kept ? v : v - gap[x];
+                return (FORM != 0 && v < kept ? count[x] > 0 : i >= kept && i < count[x]) ? i : -1;
+            };
+            auto all_issued = [&](const int* next, int v) {                // every query tile that visits number v has issued it
+                const int a = place_of(0, v), b = place_of(1, v);
+                return (a < 0 || next[0] > a) && (b < 0 || next[1] > b);
+            };
             // This one thread's instructions are what the tensor cores wait for between products (a descriptor made
             // from an address costs it as much as the MMA it describes costs the tensor pipe), so the descriptors
             // of the two query tiles and of the four key/value buffers are made once: a k step then is an addition.
@@ -242,47 +273,49 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap q_map, const _
                 v_desc[b] = make_sw128_desc_mn(smem_u32(kv_ring + b * S::KV_TILE), KT * 128, 1024);
             }
             auto pick = [&](const uint64_t* d, int b) { return b == 0 ? d[0] : (b == 1 ? d[1] : (b == 2 ? d[2] : d[3])); };
-            while (ok && (jp[0] < t1x[0] || jp[1] < t1x[1])) {
+            while (ok && (jp[0] < count[0] || jp[1] < count[1])) {
                 bool moved = false;
 #pragma unroll
                 for (int x = 0; x < 2; ++x) {
                     const uint32_t s_tmem = tmem_base + x * KT, o_tmem = tmem_base + 2 * KT + x * D;
                     if (jp[x] < js[x]) {                                   // P V of tile jp: P written, V landed
-                        const int j = jp[x], li = 2 * (j - tmin) + 1, b = li % NBUF;
-                        if (mbar_test_wait(p_full(x), (j - t0x[x]) & 1u) && mbar_test_wait(kv_full(b), (li / NBUF) & 1u)) {
+                        const int v = number_of(x, jp[x]), li = 2 * v + 1, b = li % NBUF;
+                        if (mbar_test_wait(p_full(x), jp[x] & 1u) && mbar_test_wait(kv_full(b), (li / NBUF) & 1u)) {
                             tmem_fence_after();
                             const uint64_t vd = pick(v_desc, b);
                             // A: 16 keys = 8 columns of packed bfloat16 pairs (P lies over the first 64 of the
                             // tile's 128 score columns); B: 16 key rows of V = 2048 bytes further on (128 in the
                             // descriptor's 16-byte units)
-                            umma_bf16_tmem_a(o_tmem, s_tmem, vd, idesc_o, j > t0x[x] ? 1u : 0u);
+                            umma_bf16_tmem_a(o_tmem, s_tmem, vd, idesc_o, jp[x] > 0 ? 1u : 0u);
 #pragma unroll
                             for (int ks = 1; ks < KT / 16; ++ks)
                                 umma_bf16_tmem_a(o_tmem, s_tmem + ks * 8, vd + (uint64_t)(ks * 128), idesc_o, 1u);
                             umma_commit(o_full(x));
                             ++jp[x];
-                            if (issued(jp, j) == users(j)) umma_commit(kv_empty(b));   // both tiles have read these values
+                            if (all_issued(jp, v)) umma_commit(kv_empty(b));   // both tiles have read these values
                             moved = true;
                         }
                     }
                     // S of the next tile: behind the P V before it. A barrier's parity only tells neighbouring rounds of
                     // its buffer apart, so whoever waits for a buffer must know that its round before is over: tile B,
                     // whose keys may begin any number of tiles after A's (its rows lie in the next chunk), starts its
-                    // first two tiles j only once A has issued P V of tile j - 2.
-                    if (js[x] < t1x[x] && js[x] == jp[x] && (x == 0 || js[1] >= t0x[1] + 2 || jp[0] + 1 >= js[1])) {
-                        const int j = js[x], li = 2 * (j - tmin), b = li % NBUF;
+                    // first two tiles (behind the kept ones, and of those) only once A has issued P V of the number two before.
+                    if (js[x] < count[x] && js[x] == jp[x] &&
+                        (x == 0 || js[1] >= (FORM != 0 && js[1] < kept ? 2 : kept + 2) || jp[0] + 1 >= number_of(1, js[1]))) {
+                        const int v = number_of(x, js[x]), li = 2 * v, b = li % NBUF;
                         if (mbar_test_wait(kv_full(b), (li / NBUF) & 1u)) {
                             tmem_fence_after();
-                            const uint64_t kd = pick(k_desc, b), qd = q_desc[x];
+                            const uint64_t kd = pick(k_desc, b), qd = q_desc[FORM == 2 ? 0 : x];
 #pragma unroll
-                            for (int ks = 0; ks < D / 16; ++ks) {
+                            for (int ks = 0; ks < D / (FORM == 2 ? 32 : 16); ++ks) {
                                 // half of the head, then 32 bytes a step: in the descriptor's 16-byte units
-                                const uint64_t off = (uint64_t)(((ks >> 2) * (QM * 128) + (ks & 3) * 32) >> 4);
+                                const int kstep = FORM == 2 ? x * (D / 32) + ks : ks;      // map x's share of the features
+                                const uint64_t off = (uint64_t)(((kstep >> 2) * (QM * 128) + (kstep & 3) * 32) >> 4);
                                 umma_bf16(s_tmem, qd + off, kd + off, idesc_s, ks > 0 ? 1u : 0u);
                             }
                             umma_commit(s_full(x));
                             ++js[x];
-                            if (issued(js, j) == users(j)) umma_commit(kv_empty(b));   // both tiles have read these keys
+                            if (all_issued(js, v)) umma_commit(kv_empty(b));   // both tiles have read these keys
                             moved = true;
                         }
                     }
@@ -306,8 +339,8 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap q_map, const _
         const int x = (warp - 2) >> 2;                                  // query tile of this warp
         const int lane_group = warp & 3;                                // tensor-memory lanes this warp may touch
         const int r = lane_group * 32 + lane;                           // query row of the tile = tensor-memory lane
-        const int num_x = t1x[x] - t0x[x];
-        const int first_pos = pos0 + x * QM;
+        const int num_x = count[x];
+        const int first_pos = pos0 + x * ROWS_APART;
         const int qpos = first_pos + r;
         const uint32_t lane_addr = tmem_base + ((uint32_t)(lane_group * 32) << 16);
         const uint32_t s_tmem = lane_addr + x * KT, o_tmem = lane_addr + 2 * KT + x * D;
@@ -316,13 +349,13 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap q_map, const _
         float m_ref = -INFINITY, l_run = 0.f;
         bool ok = true;
         for (int i = 0; i < num_x && ok; ++i) {
-            const int j = t0x[x] + i;
-            const int tk0 = j * KT;
+            const int tk0 = tile_of(number_of(x, i)) * KT;
             if (!mbar_wait(s_full(x), i & 1u, abort_flag, p.status, 44)) { ok = false; break; }
             tmem_fence_after();
             // columns of this tile the row may see: kmin < column <= kmax (tile-local)
             const int kmax = qpos - tk0;
             const int kmin = before_row - tk0;
+            const int kept_cols = FORM == 0 ? 0 : p.keep - tk0;             // columns below this one are kept positions
             const bool all_seen = KT - 1 <= kmax && kmin < 0;
             uint32_t sr[KT];
 #pragma unroll
@@ -339,7 +372,7 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap q_map, const _
             } else {
 #pragma unroll
                 for (int k = 0; k < KT; ++k) {
-                    if (!(k <= kmax && k > kmin)) sr[k] = 0xff800000u;             // -inf: masked by assignment
+                    if (!(k <= kmax && (k > kmin || (FORM != 0 && k < kept_cols)))) sr[k] = 0xff800000u;             // -inf: masked by assignment
                     m4[k & 3] = fmaxf(m4[k & 3], __uint_as_float(sr[k]));
                 }
             }
@@ -389,12 +422,12 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap q_map, const _
             tmem_wait_st();
             // value rows no query of the CTA may see: zero them once the tile has landed (first and last tiles only)
             if (tk0 < lo || tk0 + KT > hi) {
-                const int li = 2 * (j - tmin) + 1, b = li % NBUF;
+                const int li = 2 * number_of(x, i) + 1, b = li % NBUF;
                 if (!mbar_wait(kv_full(b), (li / NBUF) & 1u, abort_flag, p.status, 46)) { ok = false; break; }
                 uint8_t* v_tile = kv_ring + b * S::KV_TILE;
                 for (int idx = gtid; idx < KT * (D / 8); idx += 128) {
                     const int row = idx / (D / 8), chunk = idx % (D / 8);
-                    if (row >= lo - tk0 && row < hi - tk0) continue;
+                    if ((row >= lo - tk0 || (FORM != 0 && row < kept_cols)) && row < hi - tk0) continue;
                     *reinterpret_cast<uint4*>(v_tile + (chunk >> 3) * (KT * 128) + row * 128 + (((chunk & 7) ^ (row & 7)) << 4)) =
                         make_uint4(0, 0, 0, 0);
                 }
@@ -404,7 +437,51 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap q_map, const _
             __syncwarp();
             if (lane == 0) mbar_arrive(p_full(x));
         }
-        if (ok && num_x > 0) {
+        if constexpr (FORM == 2) {
+            // Thread r of A and of B share row r: A finishes features 0 .. D/2 - 1, B the rest, each from both maps' O in
+            // tensor memory. All 256 threads come by both barriers, whatever became of their waits.
+            constexpr int DH = D / 2;
+            inv_sh[x][r] = l_run > 0.f ? (x == 0 ? 1.f : p.share) / l_run : 0.f;
+#pragma unroll
+            for (int m = 0; m < 2; ++m)
+                if (ok) ok = mbar_wait(o_full(m), (num_x - 1) & 1u, abort_flag, p.status, 47);
+            tmem_fence_after();
+            asm volatile("bar.sync 1, 256;" ::: "memory");
+            const float inv_a = inv_sh[0][r], inv_b = inv_sh[1][r];
+            float o[DH], ss = 0.f;
+            __syncwarp();
+#pragma unroll
+            for (int c = 0; c < DH; c += 32) {
+                uint32_t oa[32], ob[32];
+                tmem_ld32_nowait(lane_addr + 2 * KT + x * DH + c, oa);
+                tmem_ld32_nowait(lane_addr + 2 * KT + D + x * DH + c, ob);
+                tmem_wait_ld();
+#pragma unroll
+                for (int k = 0; k < 32; ++k) {
+                    o[c + k] = __uint_as_float(oa[k]) * inv_a - __uint_as_float(ob[k]) * inv_b;
+                    ss = fmaf(o[c + k], o[c + k], ss);
+                }
+            }
+            ss_sh[x][r] = ss;
+            asm volatile("bar.sync 1, 256;" ::: "memory");
+            if (ok && r < nrows) {
+                const float f = ti_head_out_scale(p, (size_t)(row0 + r), head) * rsqrtf((ss_sh[0][r] + ss_sh[1][r]) / (float)D + p.diff_eps);
+                __nv_bfloat16* dst = p.out + ((size_t)(row0 + r) * p.hq + head) * D + x * DH;
+#pragma unroll
+                for (int c = 0; c < DH; c += 8) {
+                    float v[8];
+#pragma unroll
+                    for (int k = 0; k < 8; ++k) v[k] = o[c + k] * f;
+                    ti_gate_features<8>(p, (size_t)(row0 + r), head, D, x * DH + c, v);
+                    uint4 w;
+                    w.x = pack2(v[0], v[1]);
+                    w.y = pack2(v[2], v[3]);
+                    w.z = pack2(v[4], v[5]);
+                    w.w = pack2(v[6], v[7]);
+                    *reinterpret_cast<uint4*>(dst + c) = w;
+                }
+            }
+        } else if (ok && num_x > 0) {
             if (mbar_wait(o_full(x), (num_x - 1) & 1u, abort_flag, p.status, 47)) {
                 tmem_fence_after();
                 const float l_all = p.has_sink ? l_run + ex2(ti_sink_log2(p, head) - m_ref) : l_run;      // every score far below the sink: inf, 0
@@ -419,11 +496,15 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap q_map, const _
                     if (r < rows_x) {
 #pragma unroll
                         for (int q8 = 0; q8 < 4; ++q8) {
+                            float f[8];
+#pragma unroll
+                            for (int k = 0; k < 8; ++k) f[k] = __uint_as_float(orow[q8 * 8 + k]) * inv;
+                            if constexpr (FORM != 0) ti_gate_features<8>(p, (size_t)(row0 + x * QM + r), head, D, c + q8 * 8, f);
                             uint4 w;
-                            w.x = pack2(__uint_as_float(orow[q8 * 8]) * inv, __uint_as_float(orow[q8 * 8 + 1]) * inv);
-                            w.y = pack2(__uint_as_float(orow[q8 * 8 + 2]) * inv, __uint_as_float(orow[q8 * 8 + 3]) * inv);
-                            w.z = pack2(__uint_as_float(orow[q8 * 8 + 4]) * inv, __uint_as_float(orow[q8 * 8 + 5]) * inv);
-                            w.w = pack2(__uint_as_float(orow[q8 * 8 + 6]) * inv, __uint_as_float(orow[q8 * 8 + 7]) * inv);
+                            w.x = pack2(f[0], f[1]);
+                            w.y = pack2(f[2], f[3]);
+                            w.z = pack2(f[4], f[5]);
+                            w.w = pack2(f[6], f[7]);
                             *reinterpret_cast<uint4*>(dst + c + q8 * 8) = w;
                         }
                     }
@@ -449,12 +530,19 @@ TI_API int ti_attention_prefill_pair_rows() { return 2 * QM; }
 // first flat row, rows (<= 256), position of the first row}, every tile inside one request's portion.
 // q [T, Hq, D], out [T, Hq * D], kv_cache [2, num_pages, Hkv, page_size, D]; page_size 16, 32 or a multiple of 64.
 // has_sink: exp(sink) joins every softmax denominator without a value; out_scale: a factor on the output;
-// head_sinks, gate: a sink per query head, and a sigmoid gate per (token, query head) on the output (or null).
+// head_sinks, gate: a sink per query head, and a sigmoid gate per (token, query head) on the output (or null), per output
+// feature with gate_each; keep: a window keeps the first so many positions. maps 2: differential attention (FORM 2; share,
+// diff_eps; no sinks): tiles of at most 128 rows, or, with halves, of at most 256 that two CTAs share.
 TI_API int ti_attention_prefill_pair_sink_bf16(void* out, const void* q, const void* kv_cache, const int* tiles, int num_tiles,
                                                int num_tokens, const int* block_table, int max_blocks, int hq, int hkv, int d,
-                                               int page_size, int num_pages, float scale, int window, int has_sink,
+                                               int page_size, int num_pages, float scale, int window, int keep, int has_sink,
                                                float sink, float out_scale, const float* head_sinks, const void* gate,
-                                               int ld_gate, int gate_off, float softcap, int* status, cudaStream_t stream) {
+                                               int ld_gate, int gate_off, int gate_each, float softcap, int maps, int halves,
+                                               float share, float diff_eps, int* status, cudaStream_t stream) {
+    TI_REQUIRE(maps == 1 || (maps == 2 && !has_sink && !head_sinks), "attention_prefill_pair: one map, or two without sinks");
+    TI_REQUIRE(keep >= 0 && (!gate || !gate_each || (((uintptr_t)gate & 15) == 0 && ld_gate % 8 == 0 && gate_off % 8 == 0)),
+               "attention_prefill_pair: a gate per feature lies on 16-byte boundaries");
+    TI_REQUIRE(num_tiles <= 32767 || !halves, "attention_prefill_pair: more than 32767 tiles in one step");
     TI_REQUIRE(d == 64 || d == 128, "attention_prefill_pair: head_dim %d is not 64 or 128", d);
     TI_REQUIRE(hq > 0 && hkv > 0 && hq % hkv == 0, "attention_prefill_pair: bad head counts");
     TI_REQUIRE(num_tiles <= 65535, "attention_prefill_pair: more than 65535 tiles in one step");
@@ -471,21 +559,29 @@ TI_API int ti_attention_prefill_pair_sink_bf16(void* out, const void* q, const v
     TI_SET_SCORE_CAP(p, scale, softcap);
     p.has_sink = has_sink || head_sinks ? 1 : 0; p.sink_log2 = sink * 1.4426950408889634f; p.out_scale = out_scale;
     p.head_sinks = head_sinks; p.gate = (const __nv_bfloat16*)gate; p.ld_gate = ld_gate; p.gate_off = gate_off;
-    dim3 grid(hq, num_tiles);
-#define PP_GO(D, CAP)                                                                                                            \
+    p.gate_each = gate_each; p.keep = keep; p.halves = halves ? 1 : 0; p.share = share; p.diff_eps = diff_eps;
+    dim3 grid(hq, maps == 2 && halves ? 2 * num_tiles : num_tiles);
+#define PP_RUN(D, CAP, FORM)                                                                                                     \
     do {                                                                                                                         \
         static bool once = false;                                                                                                \
         if (!once) {                                                                                                             \
-            cudaError_t e = cudaFuncSetAttribute(prefill_attention_pair_kernel<D, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
-                                                 PpSmem<D>::BYTES);                                                              \
+            cudaError_t e = cudaFuncSetAttribute(prefill_attention_pair_kernel<D, CAP, FORM>,                                    \
+                                                 cudaFuncAttributeMaxDynamicSharedMemorySize, PpSmem<D>::BYTES);                 \
             TI_REQUIRE(e == cudaSuccess, "attention_prefill_pair: shared memory: %s", cudaGetErrorString(e));                    \
             once = true;                                                                                                         \
         }                                                                                                                        \
-        ti_launch(prefill_attention_pair_kernel<D, CAP>, grid, PP_THREADS, PpSmem<D>::BYTES, stream, q_map, kv_map, p);          \
+        ti_launch(prefill_attention_pair_kernel<D, CAP, FORM>, grid, PP_THREADS, PpSmem<D>::BYTES, stream, q_map, kv_map, p);    \
     } while (0)
-    const bool capped = p.cap_log2 > 0.f;
+#define PP_GO(D, CAP)                               \
+    do {                                            \
+        if (maps == 2) PP_RUN(D, CAP, 2);           \
+        else if (extended) PP_RUN(D, CAP, 1);       \
+        else PP_RUN(D, CAP, 0);                     \
+    } while (0)
+    const bool capped = p.cap_log2 > 0.f, extended = keep > 0 || (gate && gate_each);
     if (d == 128) { if (capped) PP_GO(128, true); else PP_GO(128, false); }
     else { if (capped) PP_GO(64, true); else PP_GO(64, false); }
+#undef PP_RUN
 #undef PP_GO
     TI_CHECK_LAUNCH("attention_prefill_pair");
     return 0;
@@ -496,5 +592,5 @@ TI_API int ti_attention_prefill_pair_bf16(void* out, const void* q, const void* 
                                           int page_size, int num_pages, float scale, int window, int* status,
                                           cudaStream_t stream) {
     return ti_attention_prefill_pair_sink_bf16(out, q, kv_cache, tiles, num_tiles, num_tokens, block_table, max_blocks, hq, hkv,
-                                               d, page_size, num_pages, scale, window, 0, 0.f, 1.f, nullptr, nullptr, 0, 0, 0.f, status, stream);
+                                               d, page_size, num_pages, scale, window, 0, 0, 0.f, 1.f, nullptr, nullptr, 0, 0, 0, 0.f, 1, 0, 0.f, 0.f, status, stream);
 }

@@ -31,6 +31,7 @@ struct PrefillParams {
     const int* tiles;                // int4 {request index, first flat row, rows (<= 128), first position}
     const int* block_table;
     int max_blocks, hq, hkv, page_size, num_pages, window;
+    int keep;                        // > 0: a window keeps the first so many positions
     int halves;                      // 1: a tile entry has up to 256 rows and two CTAs take 128 each
     int splits, split_keys;          // > 1: CTA z of a tile takes keys z * split_keys .. (a multiple of 128) and leaves a partial
     float* part_o;                   // [128-row tile][split][head][row][D] unnormalised outputs
@@ -41,7 +42,7 @@ struct PrefillParams {
     float sink_log2, out_scale;      // out_scale multiplies the output before its rounding
     const float* head_sinks;         // float32 [query heads]: a sink's logit per head in place of sink_log2 (or null)
     const __nv_bfloat16* gate;       // rows of ld_gate, first column gate_off: out *= sigmoid(gate[token][head]) (or null)
-    int ld_gate, gate_off;
+    int ld_gate, gate_off, gate_each;
     int* status;
 };
 
@@ -66,7 +67,29 @@ __device__ __forceinline__ uint32_t pack2(float lo, float hi) {
     return *reinterpret_cast<uint32_t*>(&v);
 }
 
-template <int D, bool CAP>
+// The key tiles that one share of the keys holds (all of them without a split): those of kept first positions, kept0 ..
+// kept0 + kept - 1, then the window's, tile0 .. tile1 - 1. Number j of them is tile(j).
+struct KeyTiles {
+    int kept0, kept, tile0, tile1;
+    __device__ __forceinline__ KeyTiles(const PrefillParams& p, int lo, int hi, int share) {
+        tile0 = lo / KT;
+        tile1 = (hi + KT - 1) / KT;
+        kept0 = 0;
+        kept = ti_kept_tiles(p.keep, tile0, KT);
+        if (p.splits > 1) {
+            const int first = share * (p.split_keys / KT), last = first + p.split_keys / KT;
+            kept0 = min(kept, first);
+            kept = min(kept, last) - kept0;
+            tile0 = max(tile0, first);
+            tile1 = max(tile0, min(tile1, last));
+        }
+    }
+    __device__ __forceinline__ int count() const { return kept + tile1 - tile0; }
+    __device__ __forceinline__ int tile(int j) const { return j < kept ? kept0 + j : tile0 + j - kept; }
+};
+
+// KEEP: with what a window keeps and a gate per feature (kernels of models without either are the code they were).
+template <int D, bool CAP, bool KEEP>
 __global__ void __launch_bounds__(PF_THREADS, 1)
 prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap kv_map,
                             const PrefillParams p) {
@@ -125,12 +148,9 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
     const int lo = ti_first_key(pos0, p.window);                     // first key the first query sees
     // With a split of the keys (few query tiles behind long prefixes: too few CTAs otherwise) this CTA takes the
     // key tiles of its share only and leaves an unnormalised partial result for the merge kernel.
-    int tile0 = lo / KT, tile1 = (hi + KT - 1) / KT;
-    if (p.splits > 1) {
-        tile0 = max(tile0, (int)blockIdx.z * (p.split_keys / KT));
-        tile1 = min(tile1, ((int)blockIdx.z + 1) * (p.split_keys / KT));
-    }
-    const int num_tiles = tile1 - tile0;
+    const KeyTiles own(p, lo, hi, blockIdx.z);
+    const int num_tiles = KEEP ? own.count() : own.tile1 - own.tile0;
+    auto nth_tile = [&](int j) { return KEEP ? own.tile(j) : own.tile0 + j; };
     const int* table = p.block_table + (size_t)seq * p.max_blocks;
 
     if (nrows <= 0 || num_tiles <= 0) {
@@ -151,7 +171,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
         const int num_copies = (KT / piece_rows) * S::HALVES * 2;
         const int my_piece = lane / (S::HALVES * 2), my_half = (lane >> 1) % S::HALVES, my_kv = lane & 1;
         auto page_of_tile = [&](int j) {                            // this lane's page of tile j, read ahead of its use
-            const int logical = ((tile0 + j) * KT + my_piece * piece_rows) / p.page_size;
+            const int logical = (nth_tile(j) * KT + my_piece * piece_rows) / p.page_size;
             const int page = (j < num_tiles && lane < num_copies && logical < p.max_blocks) ? table[logical] : -1;
             return page >= p.num_pages ? -1 : page;                 // never written, or given back by a window
         };
@@ -163,7 +183,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
             int ok = 1;
             if (lane == 0) ok = mbar_wait(kv_empty(s), ((j / KV_STAGES) & 1u) ^ 1u, abort_flag, p.status, 31) ? 1 : 0;
             if (!__shfl_sync(0xffffffffu, ok, 0)) break;
-            const int tok = (tile0 + j) * KT + my_piece * piece_rows;
+            const int tok = nth_tile(j) * KT + my_piece * piece_rows;
             const uint32_t copies = __popc(__ballot_sync(0xffffffffu, page >= 0));
             if (lane == 0) mbar_expect_tx(kv_full(s), copies * (uint32_t)piece_rows * 128u);
             __syncwarp();
@@ -245,7 +265,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
         bool ok = true;
         for (int j = 0; j < num_tiles && ok; ++j) {
             const int b = j & 1, s = j % KV_STAGES;
-            const int tk0 = (tile0 + j) * KT;
+            const int tk0 = nth_tile(j) * KT;
             if (!mbar_wait(s_full(b), (j >> 1) & 1u, abort_flag, p.status, 36)) { ok = false; break; }
             tmem_fence_after();
             // Columns of this tile the row may see: kmin < column <= kmax (tile-local). A chunk of 32
@@ -256,20 +276,23 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
             // same for the whole warp, because tcgen05.ld is a warp-wide instruction
             const int wmax0 = pos0 + lane_group * 32 - tk0, wmax1 = wmax0 + 31;
             const int wmin0 = before_first - tk0, wmin1 = before_last - tk0;
+            const int kept = KEEP ? p.keep - tk0 : 0;                      // columns below this one are kept positions
+            auto sees = [&](int col) { return col <= kmax && (col > kmin || (KEEP && col < kept)); };
+            auto unseen = [&](int c) { return c > wmax1 || (c + 31 <= wmin0 && (!KEEP || c >= kept)); };    // a chunk of 32
             float v[32];
             // pass 1: the row maximum of the visible scores (raw; the scale is positive)
             float mx = -INFINITY;
 #pragma unroll
             for (int cc = 0; cc < KH; cc += 32) {
                 const int c = half * KH + cc;
-                if (c > wmax1 || c + 31 <= wmin0) continue;
+                if (unseen(c)) continue;
                 tmem_ld32(lane_addr + b * KT + c, v);
                 if (c + 31 <= wmax0 && c > wmin1) {
 #pragma unroll
                     for (int i = 0; i < 32; ++i) mx = fmaxf(mx, v[i]);
                 } else {
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) mx = fmaxf(mx, (c + i <= kmax && c + i > kmin) ? v[i] : -INFINITY);
+                    for (int i = 0; i < 32; ++i) mx = fmaxf(mx, sees(c + i) ? v[i] : -INFINITY);
                 }
             }
             max_xch[b][half][r] = mx;
@@ -298,7 +321,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                 uint8_t* v_tile = kv_ring + s * S::STAGE + S::KV_TILE;
                 for (int idx = etid; idx < KT * (D / 8); idx += 256) {
                     const int row = idx / (D / 8), chunk = idx % (D / 8);
-                    if (row >= lo - tk0 && row < hi - tk0) continue;
+                    if ((row >= lo - tk0 || (KEEP && row < kept)) && row < hi - tk0) continue;
                     *reinterpret_cast<uint4*>(v_tile + (chunk >> 3) * (KT * 128) + row * 128 + (((chunk & 7) ^ (row & 7)) << 4)) =
                         make_uint4(0, 0, 0, 0);
                 }
@@ -307,7 +330,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
 #pragma unroll
             for (int cc = 0; cc < KH; cc += 32) {
                 const int c = half * KH + cc;
-                const bool none = c > wmax1 || c + 31 <= wmin0;
+                const bool none = unseen(c);
                 if (none) {
 #pragma unroll
                     for (int i = 0; i < 32; ++i) v[i] = 0.f;
@@ -322,7 +345,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                     } else {
 #pragma unroll
                         for (int i = 0; i < 32; ++i) {
-                            v[i] = (c + i <= kmax && c + i > kmin) ? ex2(ti_prob_log2<CAP>(p, v[i], m_use)) : 0.f;
+                            v[i] = sees(c + i) ? ex2(ti_prob_log2<CAP>(p, v[i], m_use)) : 0.f;
                             l_run += v[i];
                         }
                     }
@@ -373,11 +396,15 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __g
                     } else if (r < nrows) {
 #pragma unroll
                         for (int q8 = 0; q8 < 4; ++q8) {
+                            float f[8];
+#pragma unroll
+                            for (int i = 0; i < 8; ++i) f[i] = (o[c + q8 * 8 + i] + v[q8 * 8 + i]) * inv;
+                            if constexpr (KEEP) ti_gate_features<8>(p, (size_t)(row0 + r), head, D, half * DH + c + q8 * 8, f);
                             uint4 w;
-                            w.x = pack2((o[c + q8 * 8] + v[q8 * 8]) * inv, (o[c + q8 * 8 + 1] + v[q8 * 8 + 1]) * inv);
-                            w.y = pack2((o[c + q8 * 8 + 2] + v[q8 * 8 + 2]) * inv, (o[c + q8 * 8 + 3] + v[q8 * 8 + 3]) * inv);
-                            w.z = pack2((o[c + q8 * 8 + 4] + v[q8 * 8 + 4]) * inv, (o[c + q8 * 8 + 5] + v[q8 * 8 + 5]) * inv);
-                            w.w = pack2((o[c + q8 * 8 + 6] + v[q8 * 8 + 6]) * inv, (o[c + q8 * 8 + 7] + v[q8 * 8 + 7]) * inv);
+                            w.x = pack2(f[0], f[1]);
+                            w.y = pack2(f[2], f[3]);
+                            w.z = pack2(f[4], f[5]);
+                            w.w = pack2(f[6], f[7]);
                             *reinterpret_cast<uint4*>(dst + c + q8 * 8) = w;
                         }
                     }
@@ -409,9 +436,9 @@ __global__ void prefill_merge_kernel(const PrefillParams p) {
     if (r >= nrows) return;
     const int hi = pos0 + nrows;
     const int lo = ti_first_key(pos0, p.window);
-    const int tile0 = lo / KT, tile1 = (hi + KT - 1) / KT, per = p.split_keys / KT;
     float m_run = -INFINITY, acc = 0.f, l_all = 0.f;
-    for (int z = tile0 / per; z < p.splits && z * per < tile1; ++z) {
+    for (int z = 0; z < p.splits; ++z) {
+        if (KeyTiles(p, lo, hi, z).count() <= 0) continue;
         const size_t part = (((size_t)slot * p.splits + z) * p.hq + head) * QM + r;
         const float2 ml = __ldcg(reinterpret_cast<const float2*>(p.part_ml + part * 2));
         const float ov = __ldcg(p.part_o + part * D + d);
@@ -423,8 +450,9 @@ __global__ void prefill_merge_kernel(const PrefillParams p) {
         m_run = m_new;
     }
     if (p.has_sink) l_all += ex2(ti_sink_log2(p, head) - m_run);
-    p.out[((size_t)(row0 + r) * p.hq + head) * D + d] =
-        __float2bfloat16_rn(l_all > 0.f ? acc * ti_head_out_scale(p, (size_t)(row0 + r), head) / l_all : 0.f);
+    float res = l_all > 0.f ? acc * ti_head_out_scale(p, (size_t)(row0 + r), head) / l_all : 0.f;
+    ti_gate_features<1>(p, (size_t)(row0 + r), head, D, d, &res);
+    p.out[((size_t)(row0 + r) * p.hq + head) * D + d] = __float2bfloat16_rn(res);
 }
 
 }  // namespace
@@ -443,13 +471,16 @@ TI_API long long ti_attention_prefill_scratch_floats(int num_tiles, int halves, 
     return (long long)num_tiles * (halves ? 2 : 1) * splits * hq * QM * (d + 2);
 }
 // has_sink: exp(sink) joins every softmax denominator without a value; out_scale: a factor on the output;
-// head_sinks, gate: a sink per query head, and a sigmoid gate per (token, query head) on the output (or null).
+// head_sinks, gate: a sink per query head, and a sigmoid gate per (token, query head) on the output (or null), per output
+// feature with gate_each; keep: a window keeps the first so many positions.
 TI_API int ti_attention_prefill_tc_sink_bf16(void* out, const void* q, const void* kv_cache, const int* tiles, int num_tiles,
                                              int num_tokens, const int* block_table, int max_blocks, int hq, int hkv, int d,
-                                             int page_size, int num_pages, float scale, int window, int halves, int splits,
+                                             int page_size, int num_pages, float scale, int window, int keep, int halves, int splits,
                                              int split_keys, float* scratch, long long scratch_floats, int has_sink, float sink,
                                              float out_scale, const float* head_sinks, const void* gate, int ld_gate,
-                                             int gate_off, float softcap, int* status, cudaStream_t stream) {
+                                             int gate_off, int gate_each, float softcap, int* status, cudaStream_t stream) {
+    TI_REQUIRE(keep >= 0 && (!gate || !gate_each || (((uintptr_t)gate & 15) == 0 && ld_gate % 8 == 0 && gate_off % 8 == 0)),
+               "attention_prefill_tc: a gate per feature lies on 16-byte boundaries");
     TI_REQUIRE(splits >= 1 && splits <= 65535, "attention_prefill_tc: %d shares of the keys", splits);
     TI_REQUIRE(splits == 1 || (split_keys > 0 && split_keys % KT == 0 && scratch != nullptr &&
                                scratch_floats >= ti_attention_prefill_scratch_floats(num_tiles, halves, splits, hq, d)),
@@ -471,24 +502,31 @@ TI_API int ti_attention_prefill_tc_sink_bf16(void* out, const void* q, const voi
     TI_SET_SCORE_CAP(p, scale, softcap);
     p.has_sink = has_sink || head_sinks ? 1 : 0; p.sink_log2 = sink * 1.4426950408889634f; p.out_scale = out_scale;
     p.head_sinks = head_sinks; p.gate = (const __nv_bfloat16*)gate; p.ld_gate = ld_gate; p.gate_off = gate_off;
+    p.gate_each = gate_each; p.keep = keep;
     const int slots = halves ? 2 * num_tiles : num_tiles;
     p.splits = splits; p.split_keys = split_keys;
     p.part_o = scratch; p.part_ml = scratch ? scratch + (long long)slots * splits * hq * QM * d : nullptr;
     dim3 grid(hq, slots, splits);
-#define PF_GO(D, CAP)                                                                                                          \
+#define PF_RUN(D, CAP, KEEP)                                                                                                   \
     do {                                                                                                                       \
         static bool once = false;                                                                                              \
         if (!once) {                                                                                                           \
-            cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<D, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
-                                                 PfSmem<D>::BYTES);                                                            \
+            cudaError_t e = cudaFuncSetAttribute(prefill_attention_tc_kernel<D, CAP, KEEP>,                                    \
+                                                 cudaFuncAttributeMaxDynamicSharedMemorySize, PfSmem<D>::BYTES);               \
             TI_REQUIRE(e == cudaSuccess, "attention_prefill_tc: shared memory: %s", cudaGetErrorString(e));                    \
             once = true;                                                                                                       \
         }                                                                                                                      \
-        ti_launch(prefill_attention_tc_kernel<D, CAP>, grid, PF_THREADS, PfSmem<D>::BYTES, stream, q_map, kv_map, p);          \
+        ti_launch(prefill_attention_tc_kernel<D, CAP, KEEP>, grid, PF_THREADS, PfSmem<D>::BYTES, stream, q_map, kv_map, p);    \
     } while (0)
-    const bool capped = p.cap_log2 > 0.f;
-    if (d == 128) { if (capped) PF_GO(128, true); else PF_GO(128, false); }
-    else { if (capped) PF_GO(64, true); else PF_GO(64, false); }
+#define PF_GO(D)                                                                             \
+    do {                                                                                     \
+        if (capped) { if (extended) PF_RUN(D, true, true); else PF_RUN(D, true, false); }    \
+        else { if (extended) PF_RUN(D, false, true); else PF_RUN(D, false, false); }         \
+    } while (0)
+    const bool capped = p.cap_log2 > 0.f, extended = keep > 0 || (gate && gate_each);
+    if (d == 128) PF_GO(128);
+    else PF_GO(64);
+#undef PF_RUN
 #undef PF_GO
     TI_CHECK_LAUNCH("attention_prefill_tc");
     if (splits > 1) {
@@ -505,6 +543,6 @@ TI_API int ti_attention_prefill_tc_bf16(void* out, const void* q, const void* kv
                                         int split_keys, float* scratch, long long scratch_floats, int* status,
                                         cudaStream_t stream) {
     return ti_attention_prefill_tc_sink_bf16(out, q, kv_cache, tiles, num_tiles, num_tokens, block_table, max_blocks, hq, hkv, d,
-                                             page_size, num_pages, scale, window, halves, splits, split_keys, scratch,
-                                             scratch_floats, 0, 0.f, 1.f, nullptr, nullptr, 0, 0, 0.f, status, stream);
+                                             page_size, num_pages, scale, window, 0, halves, splits, split_keys, scratch,
+                                             scratch_floats, 0, 0.f, 1.f, nullptr, nullptr, 0, 0, 0, 0.f, status, stream);
 }

@@ -132,6 +132,13 @@ __device__ __forceinline__ int ti_first_key(int pos, int window) {
     return window < 0 ? pos - pos % -window : 0;
 }
 
+// A window may keep the request's first positions: a query at pos also sees every j < keep (j <= pos). The keys that are
+// seen then lie in two runs, [0, keep) and [ti_first_key(pos), pos]. Kernels that walk over tiles of `tile` keys number the
+// tiles they visit without a gap: first the kept tiles that lie before the window's first tile, then the window's.
+// Number v is the tile ti_nth_tile(v, kept, lo_tile).
+__device__ __forceinline__ int ti_kept_tiles(int keep, int lo_tile, int tile) { return min((keep + tile - 1) / tile, lo_tile); }
+__device__ __forceinline__ int ti_nth_tile(int v, int kept, int lo_tile) { return v < kept ? v : lo_tile + v - kept; }
+
 // Scores that level off smoothly: s -> cap * tanh(s / cap). P is an attention kernel's parameter block with scale_log2
 // (the softmax scale times log2 e), cap_log2 (cap * log2 e; 0: no cap) and cap_arg (scale / cap). The result is in log2
 // units, like raw * scale_log2; a masked score (-inf) stays -inf. These are the bfloat16 tensor-core kernels, whose
@@ -166,12 +173,31 @@ template <bool CAP, typename P> __device__ __forceinline__ float ti_prob_log2(co
 // A softmax sink and an output factor that may differ from head to head. P is an attention kernel's parameter block with
 // sink_log2 / head_sinks (float32 natural-log logits per query head, or null) and out_scale / gate (bfloat16 rows of
 // ld_gate elements, first column gate_off, one logit per (token, query head), or null: the output is also multiplied by
-// sigmoid(gate)).
+// sigmoid(gate)). gate_each != 0: the rows hold a logit per output FEATURE instead, head by head (ti_gate_features).
 template <typename P> __device__ __forceinline__ float ti_sink_log2(const P& p, int head) {
     return p.head_sinks ? p.head_sinks[head] * 1.4426950408889634f : p.sink_log2;
 }
 template <typename P> __device__ __forceinline__ float ti_head_out_scale(const P& p, size_t row, int head) {
-    if (!p.gate) return p.out_scale;
+    if (!p.gate || p.gate_each) return p.out_scale;
     const float z = __bfloat162float(p.gate[row * p.ld_gate + p.gate_off + head]);
     return p.out_scale / (1.f + expf(-z));
+}
+// Multiplies N neighbouring output features (from feature f of a head of d features on) by the sigmoids of their own gate
+// logits, if there are any. N 8: one 16-byte load; the launcher has seen to the alignment.
+template <int N, typename P> __device__ __forceinline__ void ti_gate_features(const P& p, size_t row, int head, int d, int f, float* v) {
+    if (!p.gate || !p.gate_each) return;
+    const __nv_bfloat16* g = p.gate + row * p.ld_gate + p.gate_off + head * d + f;
+    if constexpr (N == 8) {
+        const uint4 u = *reinterpret_cast<const uint4*>(g);
+        const __nv_bfloat162* z2 = reinterpret_cast<const __nv_bfloat162*>(&u);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const float2 z = __bfloat1622float2(z2[i]);
+            v[2 * i] *= 1.f / (1.f + expf(-z.x));
+            v[2 * i + 1] *= 1.f / (1.f + expf(-z.y));
+        }
+    } else {
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] *= 1.f / (1.f + expf(-__bfloat162float(g[i])));
+    }
 }

@@ -293,114 +293,165 @@ TI_API int ti_conv_qkv_append(void* q_out, void* cache, const void* qkv, int ld_
 // ------------------------------------------------------------------ attention over [k | v] rows, float32 arithmetic
 // One block per (token, query head). The running maximum starts at the sink's logit and the running sum at 1 when
 // there is a sink: the sink is a key without a value.
+// MAPS 2: differential attention. A query head and a key head hold two maps' features side by side; each map is a softmax of
+// its own over the same values. With a1 and a2 the maps' outputs, o = a1 - share * a2, divided by its root mean square over
+// the head's features (eps inside the root), times out_scale.
 constexpr int AR_THREADS = 128;
 constexpr int AR_MAX_D = 256;
 
-template <typename T>
-__global__ void __launch_bounds__(AR_THREADS) attention_rows_kernel(
-    T* __restrict__ out, const T* __restrict__ q, const T* __restrict__ cache, const int* __restrict__ positions,
-    const int* __restrict__ token_seq, const int* __restrict__ block_table, int max_blocks, int hq, int hkv, int d, int dv,
-    int page_size, int num_pages, int row, long long v_off, float scale, int window, int has_sink, float sink,
-    const float* __restrict__ head_sinks, const T* __restrict__ gate, int ld_gate, int gate_off,
-    float out_scale, float softcap, int* __restrict__ status) {
-    __shared__ float qs[AR_MAX_D];
-    __shared__ float p[AR_THREADS];
+struct AttentionRowsArgs {
+    void* out; const void *q, *cache;
+    const int *positions, *token_seq, *block_table; int max_blocks;
+    int hq, hkv, d, dv, page_size, num_pages, row; long long v_off;      // d: features of one map of a head
+    float scale; int window, keep, has_sink; float sink; const float* head_sinks;
+    const void* gate; int ld_gate, gate_off, gate_each;
+    float out_scale, softcap, share, diff_eps;
+    int* status;
+};
+
+template <typename T, int MAPS>
+__global__ void __launch_bounds__(AR_THREADS) attention_rows_kernel(AttentionRowsArgs a) {
+    __shared__ float qs[MAPS * AR_MAX_D];
+    __shared__ float p[MAPS][AR_THREADS];
     __shared__ long long row_off[AR_THREADS];
     __shared__ float red[33];
     ti_grid_launch_dependents();
     ti_grid_wait();
     const int tid = threadIdx.x;
     const int h = blockIdx.x, t = blockIdx.y;
-    const int pos = positions[t];
-    const int lo = ti_first_key(pos, window);
-    const int kvh = h / (hq / hkv);
-    const int* table = block_table + (size_t)token_seq[t] * max_blocks;
-    const T* qrow = q + ((size_t)t * hq + h) * d;
-    for (int i = tid; i < d; i += AR_THREADS) qs[i] = to_f32(qrow[i]);
+    const int d = a.d, dv = a.dv;
+    const int pos = a.positions[t];
+    const int lo = ti_first_key(pos, a.window);
+    const int kept = min(a.keep, lo);                      // first positions that are seen beside the window
+    const int seen = kept + pos + 1 - lo;
+    const int kvh = h / (a.hq / a.hkv);
+    const T* cache = (const T*)a.cache;
+    const int* table = a.block_table + (size_t)a.token_seq[t] * a.max_blocks;
+    const T* qrow = (const T*)a.q + ((size_t)t * a.hq + h) * (MAPS * d);
+    for (int i = tid; i < MAPS * d; i += AR_THREADS) qs[i] = to_f32(qrow[i]);
     __syncthreads();
 
-    float acc0 = 0.f, acc1 = 0.f;
-    if (head_sinks) { has_sink = 1; sink = head_sinks[h]; }            // a learned sink per query head
-    if (gate) {                                                          // a sigmoid gate per (token, query head)
-        const float z = to_f32(gate[(size_t)t * ld_gate + gate_off + h]);
+    float acc[MAPS][2], m[MAPS], l[MAPS];
+    int has_sink = a.has_sink;
+    float sink = a.sink, out_scale = a.out_scale;
+    if (a.head_sinks) { has_sink = 1; sink = a.head_sinks[h]; }            // a learned sink per query head
+    const T* gate = (const T*)a.gate;
+    if (gate && !a.gate_each) {                                              // a sigmoid gate per (token, query head)
+        const float z = to_f32(gate[(size_t)t * a.ld_gate + a.gate_off + h]);
         out_scale *= 1.f / (1.f + expf(-z));
     }
-    float m = has_sink ? sink : -INFINITY, l = has_sink ? 1.f : 0.f;
-    for (int tile0 = lo; tile0 <= pos; tile0 += AR_THREADS) {
-        const int j = tile0 + tid;
-        float s = -INFINITY;
+#pragma unroll
+    for (int mp = 0; mp < MAPS; ++mp) {
+        acc[mp][0] = acc[mp][1] = 0.f;
+        m[mp] = has_sink ? sink : -INFINITY;
+        l[mp] = has_sink ? 1.f : 0.f;
+    }
+    for (int n0 = 0; n0 < seen; n0 += AR_THREADS) {        // the seen keys without a gap: the kept ones, then the window's
+        const int n = n0 + tid;
+        float s[MAPS];
+#pragma unroll
+        for (int mp = 0; mp < MAPS; ++mp) s[mp] = -INFINITY;
         long long off = -1;
-        if (j <= pos) {
-            const int logical = j / page_size;
-            const int page = logical < max_blocks ? table[logical] : -1;
-            if (page >= 0 && page < num_pages) {
-                off = (((long long)page * hkv + kvh) * page_size + j % page_size) * row;
+        if (n < seen) {
+            const int j = ti_nth_tile(n, kept, lo);
+            const int logical = j / a.page_size;
+            const int page = logical < a.max_blocks ? table[logical] : -1;
+            if (page >= 0 && page < a.num_pages) {
+                off = (((long long)page * a.hkv + kvh) * a.page_size + j % a.page_size) * a.row;
                 const T* krow = cache + off;
-                float dot = 0.f;
-                for (int i = 0; i < d; ++i) dot = fmaf(qs[i], to_f32(krow[i]), dot);
-                s = dot * scale;
-                if (softcap > 0.f) s = softcap * tanhf(s / softcap);      // scores level off smoothly at +-softcap
-            } else if (status) {
-                atomicExch(status, 2);                 // a visible key without a page
+#pragma unroll
+                for (int mp = 0; mp < MAPS; ++mp) {
+                    float dot = 0.f;
+                    for (int i = 0; i < d; ++i) dot = fmaf(qs[mp * d + i], to_f32(krow[mp * d + i]), dot);
+                    s[mp] = dot * a.scale;
+                    if (a.softcap > 0.f) s[mp] = a.softcap * tanhf(s[mp] / a.softcap);      // scores level off smoothly at +-softcap
+                }
+            } else if (a.status) {
+                atomicExch(a.status, 2);                 // a visible key without a page
             }
         }
-        const float tile_max = block_max(s, red);
-        const float m_new = fmaxf(m, tile_max);
-        const float corr = (m == -INFINITY) ? 0.f : expf(m - m_new);
-        const float pj = (s == -INFINITY) ? 0.f : expf(s - m_new);
-        p[tid] = pj;
         row_off[tid] = off;
-        const float tile_sum = block_sum(pj, red);      // also orders the writes of p and row_off
-        l = l * corr + tile_sum;
-        acc0 *= corr;
-        acc1 *= corr;
-        m = m_new;
-        const int n = min(AR_THREADS, pos + 1 - tile0);
+#pragma unroll
+        for (int mp = 0; mp < MAPS; ++mp) {
+            const float tile_max = block_max(s[mp], red);
+            const float m_new = fmaxf(m[mp], tile_max);
+            const float corr = (m[mp] == -INFINITY) ? 0.f : expf(m[mp] - m_new);
+            const float pj = (s[mp] == -INFINITY) ? 0.f : expf(s[mp] - m_new);
+            p[mp][tid] = pj;
+            const float tile_sum = block_sum(pj, red);      // also orders the writes of p and row_off
+            l[mp] = l[mp] * corr + tile_sum;
+            acc[mp][0] *= corr;
+            acc[mp][1] *= corr;
+            m[mp] = m_new;
+        }
+        const int count = min(AR_THREADS, seen - n0);
         if (tid < dv) {
-            for (int jj = 0; jj < n; ++jj) {
+            for (int jj = 0; jj < count; ++jj) {
                 const long long o = row_off[jj];
                 if (o < 0) continue;
-                const float pv = p[jj];
-                acc0 = fmaf(pv, to_f32(cache[o + v_off + tid]), acc0);
-                if (tid + AR_THREADS < dv) acc1 = fmaf(pv, to_f32(cache[o + v_off + tid + AR_THREADS]), acc1);
+                const float v0 = to_f32(cache[o + a.v_off + tid]);
+                const float v1 = tid + AR_THREADS < dv ? to_f32(cache[o + a.v_off + tid + AR_THREADS]) : 0.f;
+#pragma unroll
+                for (int mp = 0; mp < MAPS; ++mp) {
+                    acc[mp][0] = fmaf(p[mp][jj], v0, acc[mp][0]);
+                    acc[mp][1] = fmaf(p[mp][jj], v1, acc[mp][1]);
+                }
             }
         }
         __syncthreads();
     }
-    T* orow = out + ((size_t)t * hq + h) * dv;
-    const float inv = l > 0.f ? out_scale / l : 0.f;
-    if (tid < dv) orow[tid] = from_f32<T>(acc0 * inv);
-    if (tid + AR_THREADS < dv) orow[tid + AR_THREADS] = from_f32<T>(acc1 * inv);
+    float o[2];
+    const float inv = l[0] > 0.f ? (MAPS == 1 ? out_scale : 1.f) / l[0] : 0.f;
+    o[0] = acc[0][0] * inv;
+    o[1] = acc[0][1] * inv;
+    if constexpr (MAPS == 2) {
+        const float inv2 = l[1] > 0.f ? a.share / l[1] : 0.f;
+        o[0] -= acc[1][0] * inv2;
+        o[1] -= acc[1][1] * inv2;
+        const float ss = (tid < dv ? o[0] * o[0] : 0.f) + (tid + AR_THREADS < dv ? o[1] * o[1] : 0.f);
+        const float r = out_scale * rsqrtf(block_sum(ss, red) / (float)dv + a.diff_eps);
+        o[0] *= r;
+        o[1] *= r;
+    }
+    T* orow = (T*)a.out + ((size_t)t * a.hq + h) * dv;
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+        const int f = tid + e * AR_THREADS;
+        if (f >= dv) break;
+        if (gate && a.gate_each) o[e] *= 1.f / (1.f + expf(-to_f32(gate[(size_t)t * a.ld_gate + a.gate_off + (size_t)h * dv + f])));
+        orow[f] = from_f32<T>(o[e]);
+    }
 }
 
-// planes 1: cache [pages][hkv][page_size][d + dv]; planes 2 (d == dv): [2][pages][hkv][page_size][d].
+// planes 1: cache [pages][hkv][page_size][maps d + dv]; planes 2 (maps d == dv): [2][pages][hkv][page_size][maps d].
 // out: [T][hq * dv], multiplied by out_scale before its one rounding. head_sinks (float32 [hq], or null): a sink's
 // logit per query head in place of the one `sink`; gate (compute dtype, rows of ld_gate, first column gate_off, or
-// null): the output of (token, head) is also multiplied by sigmoid(gate[token][head]). softcap > 0: a score s becomes
-// softcap * tanh(s / softcap) before the softmax.
+// null): the output of (token, head) is also multiplied by sigmoid(gate[token][head]), or, gate_each, feature by feature by
+// sigmoid(gate[token][head * dv + feature]). softcap > 0: a score s becomes softcap * tanh(s / softcap) before the
+// softmax. keep > 0: a window keeps the first `keep` positions. maps 2: differential attention with share and diff_eps.
 TI_API int ti_attention_rows(void* out, const void* q, const void* cache, const int* positions, const int* token_seq,
                              const int* block_table, int max_blocks, int num_tokens, int hq, int hkv, int d, int dv,
-                             int page_size, int num_pages, int planes, float scale, int window, int has_sink, float sink,
-                             const float* head_sinks, const void* gate, int ld_gate, int gate_off,
-                             float out_scale, float softcap, int* status, int dtype, cudaStream_t stream) {
-    TI_REQUIRE(planes == 1 || (planes == 2 && d == dv), "attention_rows: two planes need keys and values of one size");
-    const int row = planes == 2 ? d : d + dv;
-    const long long v_off = planes == 2 ? (long long)num_pages * hkv * page_size * d : d;
+                             int page_size, int num_pages, int planes, float scale, int window, int keep, int has_sink, float sink,
+                             const float* head_sinks, const void* gate, int ld_gate, int gate_off, int gate_each,
+                             float out_scale, float softcap, int maps, float share, float diff_eps, int* status, int dtype,
+                             cudaStream_t stream) {
+    TI_REQUIRE(maps == 1 || maps == 2, "attention_rows: %d maps (1 or 2)", maps);
+    const int kd = maps * d;
+    TI_REQUIRE(planes == 1 || (planes == 2 && kd == dv), "attention_rows: two planes need keys and values of one size");
     TI_REQUIRE(d > 0 && d <= AR_MAX_D && dv > 0 && dv <= AR_MAX_D, "attention_rows: head sizes %d / %d not in 1..%d", d, dv, AR_MAX_D);
     TI_REQUIRE(hq > 0 && hkv > 0 && hq % hkv == 0, "attention_rows: %d query heads do not group over %d kv heads", hq, hkv);
-    TI_REQUIRE(page_size > 0 && num_tokens >= 0 && softcap >= 0.f, "attention_rows: bad sizes");
+    TI_REQUIRE(page_size > 0 && num_tokens >= 0 && softcap >= 0.f && keep >= 0, "attention_rows: bad sizes");
     TI_REQUIRE(num_tokens <= 65535, "attention_rows: more than 65535 tokens in one step");
     if (num_tokens == 0) return 0;
+    AttentionRowsArgs a = {out, q, cache, positions, token_seq, block_table, max_blocks, hq, hkv, d, dv, page_size, num_pages,
+                           planes == 2 ? kd : kd + dv, planes == 2 ? (long long)num_pages * hkv * page_size * kd : kd,
+                           scale, window, keep, has_sink, sink, head_sinks, gate, ld_gate, gate_off, gate_each,
+                           out_scale, softcap, share, diff_eps, status};
     dim3 grid(hq, num_tokens);
-    if (dtype == TI_F32)
-        ti_launch(attention_rows_kernel<float>, grid, AR_THREADS, 0, stream, (float*)out, (const float*)q, (const float*)cache,
-                  positions, token_seq, block_table, max_blocks, hq, hkv, d, dv, page_size, num_pages, row, v_off, scale, window,
-                  has_sink, sink, head_sinks, (const float*)gate, ld_gate, gate_off, out_scale, softcap, status);
-    else if (dtype == TI_BF16)
-        ti_launch(attention_rows_kernel<__nv_bfloat16>, grid, AR_THREADS, 0, stream, (__nv_bfloat16*)out, (const __nv_bfloat16*)q,
-                  (const __nv_bfloat16*)cache, positions, token_seq, block_table, max_blocks, hq, hkv, d, dv, page_size,
-                  num_pages, row, v_off, scale, window, has_sink, sink, head_sinks, (const __nv_bfloat16*)gate, ld_gate, gate_off,
-                  out_scale, softcap, status);
+    if (dtype == TI_F32 && maps == 1) ti_launch(attention_rows_kernel<float, 1>, grid, AR_THREADS, 0, stream, a);
+    else if (dtype == TI_F32) ti_launch(attention_rows_kernel<float, 2>, grid, AR_THREADS, 0, stream, a);
+    else if (dtype == TI_BF16 && maps == 1) ti_launch(attention_rows_kernel<__nv_bfloat16, 1>, grid, AR_THREADS, 0, stream, a);
+    else if (dtype == TI_BF16) ti_launch(attention_rows_kernel<__nv_bfloat16, 2>, grid, AR_THREADS, 0, stream, a);
     else TI_REQUIRE(false, "attention_rows: unknown dtype %d", dtype);
     TI_CHECK_LAUNCH("attention_rows");
     return 0;

@@ -11,6 +11,9 @@
 //   plan     : one block: where every expert's rows start in the sorted order, and the list of row tiles
 //              [expert, first row, rows] that the grouped product walks
 //   place    : slot of every (token, choice) in the sorted order and the token of every slot
+//   route by table : no router. A row of a table names the experts of a token id, so the routing of every such layer is known
+//              from the step's token ids alone: one launch makes it for all layers at once, a block a layer (count, plan and
+//              place in shared memory), before the first layer runs
 //   grouped product : for every tile, rows x W[expert]^T with float32 FMA accumulation in a fixed k order; the up
 //              form gathers its rows from the tokens and applies max(v, 0)^2, the down form reads the sorted rows
 //   combine_norm_add : y = sum_k weight_k * down[slot_k] (+ the shared expert's output), in choice order, then the
@@ -255,6 +258,87 @@ TI_API int ti_moe_route(int* chosen, float* weight, int* rank, int* counts, int*
     return 0;
 }
 
+// ------------------------------------------------------------------ route by table
+constexpr int RT_THREADS = 1024;
+constexpr int RT_MAX_EXPERTS = 1024;
+
+struct RouteTableArgs {
+    const int *token_ids, *tables;         // tables [layers][vocab][top]
+    int *chosen, *slot_of, *token_of, *tiles, *num_tiles;      // [layers][tokens top] x 3, [layers][max_tiles][3], [layers]
+    int num_tokens, vocab, top, experts, tile_rows, max_tiles;
+};
+
+__global__ void __launch_bounds__(RT_THREADS) moe_route_table_kernel(RouteTableArgs a) {
+    __shared__ int counts[RT_MAX_EXPERTS], starts[RT_MAX_EXPERTS], first_tile[RT_MAX_EXPERTS];
+    __shared__ int total_tiles;
+    ti_grid_launch_dependents();
+    ti_grid_wait();
+    const int layer = blockIdx.x, tid = threadIdx.x, lane = tid & 31;
+    const int n = a.num_tokens * a.top;
+    const int* table = a.tables + (size_t)layer * a.vocab * a.top;
+    int* chosen = a.chosen + (size_t)layer * n;
+    int* slot_of = a.slot_of + (size_t)layer * n;
+    int* token_of = a.token_of + (size_t)layer * n;
+    int* tiles = a.tiles + (size_t)layer * a.max_tiles * 3;
+    for (int e = tid; e < a.experts; e += RT_THREADS) counts[e] = 0;
+    __syncthreads();
+#pragma unroll 4
+    for (int i = tid; i < n; i += RT_THREADS) {
+        const int token = min(max(a.token_ids[i / a.top], 0), a.vocab - 1);
+        const int e = min(max(table[(size_t)token * a.top + i % a.top], 0), a.experts - 1);     // a table is checked when it is loaded
+        chosen[i] = e;
+        atomicAdd(&counts[e], 1);
+    }
+    __syncthreads();
+    if (tid < 32) {                                        // where every expert's rows and tiles start
+        int rows = 0, tls = 0;
+        for (int e0 = 0; e0 < a.experts; e0 += 32) {
+            const int e = e0 + lane, c = e < a.experts ? counts[e] : 0, k = (c + a.tile_rows - 1) / a.tile_rows;
+            int ci = c, ki = k;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int cv = __shfl_up_sync(0xffffffffu, ci, o), kv = __shfl_up_sync(0xffffffffu, ki, o);
+                if (lane >= o) { ci += cv; ki += kv; }
+            }
+            if (e < a.experts) { starts[e] = rows + ci - c; first_tile[e] = tls + ki - k; }
+            rows += __shfl_sync(0xffffffffu, ci, 31);
+            tls += __shfl_sync(0xffffffffu, ki, 31);
+        }
+        if (lane == 0) total_tiles = min(tls, a.max_tiles);
+    }
+    __syncthreads();
+    for (int e = tid; e < a.experts; e += RT_THREADS) {
+        const int c = counts[e];
+        for (int r = 0, k = first_tile[e]; r < c && k < a.max_tiles; r += a.tile_rows, ++k) {
+            tiles[3 * k] = e;
+            tiles[3 * k + 1] = starts[e] + r;
+            tiles[3 * k + 2] = min(a.tile_rows, c - r);
+        }
+    }
+    if (tid == 0) a.num_tiles[layer] = total_tiles;
+    __syncthreads();                                       // starts[] now turn into cursors
+#pragma unroll 4
+    for (int i = tid; i < n; i += RT_THREADS) {            // each thread reads back what it wrote itself
+        const int slot = atomicAdd(&starts[chosen[i]], 1);
+        slot_of[i] = slot;
+        token_of[slot] = i / a.top;
+    }
+}
+
+// tables int32 [layers][vocab][top] with entries below `experts`; the outputs of layer l start at l times their length a layer.
+TI_API int ti_moe_route_table(int* chosen, int* slot_of, int* token_of, int* tiles, int* num_tiles, const int* token_ids,
+                              const int* tables, int layers, int num_tokens, int vocab, int top, int experts, int tile_rows,
+                              int max_tiles, cudaStream_t stream) {
+    TI_REQUIRE(layers >= 0 && num_tokens >= 0 && vocab > 0 && top > 0 && tile_rows > 0, "moe_route_table: bad sizes");
+    TI_REQUIRE(experts > 0 && experts <= RT_MAX_EXPERTS && top <= experts, "moe_route_table: %d of %d experts (at most %d)", top,
+               experts, RT_MAX_EXPERTS);
+    if (layers == 0 || num_tokens == 0) return 0;
+    RouteTableArgs a = {token_ids, tables, chosen, slot_of, token_of, tiles, num_tiles, num_tokens, vocab, top, experts, tile_rows, max_tiles};
+    ti_launch(moe_route_table_kernel, layers, RT_THREADS, 0, stream, a);
+    TI_CHECK_LAUNCH("moe_route_table");
+    return 0;
+}
+
 // ------------------------------------------------------------------ grouped product
 constexpr int EG_BM = 32, EG_BN = 64, EG_BK = 16, EG_THREADS = 128;
 
@@ -489,13 +573,42 @@ __global__ void moe_clamped_glu_kernel(T* __restrict__ out, const T* __restrict_
     }
 }
 
+// The same, eight features (bfloat16, 16 bytes) a thread: a row's halves start on 16-byte boundaries.
+__global__ void moe_clamped_glu_vec_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ in, size_t rows, int ff,
+                                           float limit, float alpha) {
+    ti_grid_launch_dependents();
+    ti_grid_wait();
+    const int vecs = ff / 8;
+    const size_t n = rows * vecs, stride = (size_t)gridDim.x * blockDim.x;
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += stride) {
+        const size_t r = i / vecs;
+        const int c = (int)(i % vecs);
+        const uint4 g4 = reinterpret_cast<const uint4*>(in + r * 2 * ff)[c], u4 = reinterpret_cast<const uint4*>(in + r * 2 * ff + ff)[c];
+        const __nv_bfloat162 *g2 = reinterpret_cast<const __nv_bfloat162*>(&g4), *u2 = reinterpret_cast<const __nv_bfloat162*>(&u4);
+        uint4 o4;
+        __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&o4);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            const float2 g = __bfloat1622float2(g2[k]), u = __bfloat1622float2(u2[k]);
+            const float ga = fminf(g.x, limit), gb = fminf(g.y, limit);
+            const float ua = fminf(fmaxf(u.x, -limit), limit), ub = fminf(fmaxf(u.y, -limit), limit);
+            o2[k] = __floats2bfloat162_rn(ga / (1.f + expf(-alpha * ga)) * (ua + 1.f), gb / (1.f + expf(-alpha * gb)) * (ub + 1.f));
+        }
+        reinterpret_cast<uint4*>(out + r * ff)[c] = o4;
+    }
+}
+
 TI_API int ti_moe_clamped_glu(void* out, const void* in, long long rows, int ff, float limit, float alpha, int dtype,
                               cudaStream_t stream) {
     TI_REQUIRE(rows >= 0 && ff > 0, "moe_clamped_glu: bad sizes");
     if (rows == 0) return 0;
     const long long want = (rows * ff + 255) / 256;
     const int blocks = (int)(want < 148 * 16 ? want : 148 * 16);
-    if (dtype == TI_F32) ti_launch(moe_clamped_glu_kernel<float>, blocks, 256, 0, stream, (float*)out, (const float*)in, (size_t)rows, ff, limit, alpha);
+    if (dtype == TI_BF16 && ff % 8 == 0 && (((uintptr_t)out | (uintptr_t)in) & 15) == 0) {
+        const long long vwant = (rows * (ff / 8) + 255) / 256;
+        ti_launch(moe_clamped_glu_vec_kernel, (int)(vwant < 148 * 16 ? vwant : 148 * 16), 256, 0, stream, (__nv_bfloat16*)out,
+                  (const __nv_bfloat16*)in, (size_t)rows, ff, limit, alpha);
+    } else if (dtype == TI_F32) ti_launch(moe_clamped_glu_kernel<float>, blocks, 256, 0, stream, (float*)out, (const float*)in, (size_t)rows, ff, limit, alpha);
     else if (dtype == TI_BF16) ti_launch(moe_clamped_glu_kernel<__nv_bfloat16>, blocks, 256, 0, stream, (__nv_bfloat16*)out, (const __nv_bfloat16*)in, (size_t)rows, ff, limit, alpha);
     else TI_REQUIRE(false, "moe_clamped_glu: unknown dtype %d", dtype);
     TI_CHECK_LAUNCH("moe_clamped_glu");

@@ -341,6 +341,12 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constan
                     float* v = reinterpret_cast<float*>(rg);
                     const float* u = reinterpret_cast<const float*>(ru);
                     __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)m * p.N + j0;
+                    if (p.bias) {
+                        float* uw = reinterpret_cast<float*>(ru);
+#pragma unroll
+                        for (int i = 0; i < 32; ++i)
+                            if (j0 + i < p.N) { v[i] += p.bias[j0 + i]; uw[i] += p.bias[p.N + j0 + i]; }
+                    }
 #pragma unroll
                     for (int i = 0; i < 32; ++i) v[i] = glu_mul(v[i], u[i], gelu);
                     if (j0 + 32 <= p.N && (((size_t)m * p.N + j0) & 7) == 0) {
@@ -382,12 +388,12 @@ TI_API int ti_gemm_pair_supported(int M, int N, int K, int gated) {
 }
 
 // y = x . w^T in bfloat16 with float32 accumulation, in the pair form; for steps of many tokens. gated: w is
-// [2N, K] (gate rows, then up rows), out [M, N] = act(x.gate) * (x.up) (gated 1: silu, 2: the tanh form of gelu). out_f32: out is float32.
+// [2N, K] (gate rows, then up rows), out [M, N] = act(x.gate) * (x.up) (gated 1: silu, 2: the tanh form of gelu), with bias [2N] on both halves. out_f32: out is float32.
 // status: device word set if a wait ran out.
 TI_API int ti_gemm_pair_bf16(void* out, const void* x, const void* w, const float* bias, const void* residual,
                              int M, int N, int K, int gated, int out_f32, int* status, cudaStream_t stream) {
     TI_REQUIRE(ti_gemm_pair_supported(M, N, K, gated), "gemm_pair: shape %d x %d x %d not supported", M, N, K);
-    TI_REQUIRE(!(gated && (bias || residual || out_f32)), "gemm_pair: the gated form takes no bias, residual or float32 output");
+    TI_REQUIRE(!(gated && (residual || out_f32)), "gemm_pair: the gated form takes no residual or float32 output");
     CUtensorMap map_x, map_w;
     if (!ti_get_bf16_map(x, M, K, BM, &map_x)) return -1;
     if (!ti_get_bf16_map(w, gated ? 2 * N : N, K, BN / 2, &map_w)) return -1;

@@ -66,6 +66,7 @@ __global__ void __launch_bounds__(GS_THREADS) gemm_simt_kernel(
             if (n >= N) continue;
             float v = acc[i][j];
             if constexpr (GATED != 0) {
+                if (bias) { v += bias[n]; acc2[i][j] += bias[gate_rows + n]; }
                 if constexpr (GATED == 1) v = v / (1.f + expf(-v));
                 else v = 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
                 v *= acc2[i][j];
@@ -79,27 +80,27 @@ __global__ void __launch_bounds__(GS_THREADS) gemm_simt_kernel(
 }
 
 // out_f32 != 0: the result is stored as float32 whatever the input dtype (logits).
-// gated != 0 (1: silu, 2: the tanh form of gelu): w is [2N, K], rows 0..N-1 the gate and N..2N-1 the up projection; out is [M, N].
+// gated != 0 (1: silu, 2: the tanh form of gelu): w is [2N, K], rows 0..N-1 the gate and N..2N-1 the up projection, bias [2N]; out is [M, N].
 TI_API int ti_gemm_simt(void* out, const void* x, const void* w, const float* bias, const void* residual,
                         int M, int N, int K, int gated, int out_f32, int dtype, cudaStream_t stream) {
     TI_REQUIRE(M >= 0 && N > 0 && K > 0, "gemm: bad sizes M=%d N=%d K=%d", M, N, K);
-    TI_REQUIRE(!(gated && (bias || residual || out_f32)), "gemm: the gated form takes no bias, residual or float32 output");
+    TI_REQUIRE(!(gated && (residual || out_f32)), "gemm: the gated form takes no residual or float32 output");
     if (M == 0) return 0;
     dim3 grid((N + GS_BN - 1) / GS_BN, (M + GS_BM - 1) / GS_BM);
     TI_REQUIRE(grid.y <= 65535, "gemm: too many rows");
     if (dtype == TI_F32) {
         if (gated == 2)
-            ti_launch(gemm_simt_kernel<float, float, 2>, grid, GS_THREADS, 0, stream, (float*)out, (const float*)x, (const float*)w, nullptr, nullptr, M, N, K, N);
+            ti_launch(gemm_simt_kernel<float, float, 2>, grid, GS_THREADS, 0, stream, (float*)out, (const float*)x, (const float*)w, bias, nullptr, M, N, K, N);
         else if (gated)
-            ti_launch(gemm_simt_kernel<float, float, 1>, grid, GS_THREADS, 0, stream, (float*)out, (const float*)x, (const float*)w, nullptr, nullptr, M, N, K, N);
+            ti_launch(gemm_simt_kernel<float, float, 1>, grid, GS_THREADS, 0, stream, (float*)out, (const float*)x, (const float*)w, bias, nullptr, M, N, K, N);
         else
             ti_launch(gemm_simt_kernel<float, float, 0>, grid, GS_THREADS, 0, stream, (float*)out, (const float*)x, (const float*)w, bias, (const float*)residual, M, N, K, 0);
     } else if (dtype == TI_BF16) {
         typedef __nv_bfloat16 B;
         if (gated == 2)
-            ti_launch(gemm_simt_kernel<B, B, 2>, grid, GS_THREADS, 0, stream, (B*)out, (const B*)x, (const B*)w, nullptr, nullptr, M, N, K, N);
+            ti_launch(gemm_simt_kernel<B, B, 2>, grid, GS_THREADS, 0, stream, (B*)out, (const B*)x, (const B*)w, bias, nullptr, M, N, K, N);
         else if (gated)
-            ti_launch(gemm_simt_kernel<B, B, 1>, grid, GS_THREADS, 0, stream, (B*)out, (const B*)x, (const B*)w, nullptr, nullptr, M, N, K, N);
+            ti_launch(gemm_simt_kernel<B, B, 1>, grid, GS_THREADS, 0, stream, (B*)out, (const B*)x, (const B*)w, bias, nullptr, M, N, K, N);
         else if (out_f32)
             ti_launch(gemm_simt_kernel<B, float, 0>, grid, GS_THREADS, 0, stream, (float*)out, (const B*)x, (const B*)w, bias, (const B*)residual, M, N, K, 0);
         else

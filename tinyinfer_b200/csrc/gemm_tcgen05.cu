@@ -341,12 +341,12 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_c
                 // hold gate rows j.., lanes 16..31 the up rows of the same outputs, which reach the
                 // gate's lanes by a shuffle.
                 if (SWAP && (p.N & 3) == 0 &&
-                    (p.gated ? ((uintptr_t)p.out & 7) == 0
+                    (p.gated ? ((uintptr_t)p.out & 7) == 0 && ((uintptr_t)p.bias & 15) == 0
                              : ((uintptr_t)p.out & 15) == 0 && ((uintptr_t)p.residual & 7) == 0 && ((uintptr_t)p.bias & 15) == 0)) {
                     const int n0 = r0 + 4 * (p.gated ? (lane & 15) : lane);
                     const bool n_ok = n0 < p.N;                        // N is a multiple of 4: all four rows or none
                     float4 b4 = make_float4(0.f, 0.f, 0.f, 0.f), g4 = make_float4(0.f, 0.f, 0.f, 0.f);
-                    if (p.bias && n_ok) b4 = *reinterpret_cast<const float4*>(p.bias + n0);
+                    if (p.bias && n_ok) b4 = *reinterpret_cast<const float4*>(p.bias + n0 + (p.gated && lane >= 16 ? p.N : 0));
                     if (p.emit_g && n_ok) g4 = *reinterpret_cast<const float4*>(p.emit_g + n0);
                     const int cols_real = min(BN, p.M - c0);
                     // the tokens this unit finishes: all of them, or with a shared sum those with
@@ -394,6 +394,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_c
 #pragma unroll
                                 for (int i = 0; i < G; ++i) {
                                     const int col = g0 + 4 * i * col_step;              // the same for the whole warp
+                                    if (p.bias) { acc[i].x += b4.x; acc[i].y += b4.y; acc[i].z += b4.z; acc[i].w += b4.w; }   // no row scale then
                                     float4 up;
                                     up.x = __shfl_xor_sync(0xffffffffu, acc[i].x, 16); up.y = __shfl_xor_sync(0xffffffffu, acc[i].y, 16);
                                     up.z = __shfl_xor_sync(0xffffffffu, acc[i].z, 16); up.w = __shfl_xor_sync(0xffffffffu, acc[i].w, 16);
@@ -654,6 +655,11 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_c
                         const int j0 = c0 + c;
                         if (!row_ok || j0 >= p.N) continue;
                         __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(p.out) + (size_t)m * p.N + j0;
+                        if (p.bias) {
+#pragma unroll
+                            for (int i = 0; i < 16; ++i)
+                                if (j0 + i < p.N) { v[i] += p.bias[j0 + i]; u[i] += p.bias[p.N + j0 + i]; }
+                        }
 #pragma unroll
                         for (int i = 0; i < 16; ++i) v[i] = glu_mul(v[i], u[i], gelu);
                         if (j0 + 16 <= p.N && (((size_t)m * p.N + j0) & 7) == 0) {
@@ -704,10 +710,11 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_c
                     // the up half goes through shared memory to the threads that hold the gate
                     const bool is_up = row_in_tile >= 64;
                     const int jj = row_in_tile & 63;
+                    const float b = p.bias && r0 + jj < p.N ? p.bias[(is_up ? p.N : 0) + r0 + jj] : 0.f;
                     for (int c = 0; c < BN; c += 16) {
                         load_chunk(c, v);
 #pragma unroll
-                        for (int i = 0; i < 16; ++i) v[i] *= row_scale_sh[c + i];        // gate and up alike
+                        for (int i = 0; i < 16; ++i) v[i] = fmaf(v[i], row_scale_sh[c + i], b);        // gate and up alike
                         if (is_up) {
 #pragma unroll
                             for (int i = 0; i < 16; ++i) exch[jj * 17 + i] = v[i];
@@ -801,7 +808,7 @@ int launch(const CUtensorMap& rows_map, const CUtensorMap& cols_map, const GemmP
 TI_API int ti_gemm_bf16_supported(int M, int N, int K) { return (M > 0 && N > 0 && K > 0 && K % 8 == 0) ? 1 : 0; }
 
 // y = x . w^T in bfloat16 with float32 accumulation. gated: w is [2N, K] (gate rows, then up rows),
-// out [M, N] = act(x.gate) * (x.up), act being silu (gated 1) or the tanh form of gelu (gated 2). out_f32: out is float32. status: device word set if a wait ran out.
+// out [M, N] = act(x.gate) * (x.up), act being silu (gated 1) or the tanh form of gelu (gated 2), with bias [2N] on both halves. out_f32: out is float32. status: device word set if a wait ran out.
 // workspace / counters: float32 scratch and zeroed int32 words for the split-k path of small M (may be
 // null: then no tile is split). Calls that share them must be ordered on one stream.
 struct NormLink {                  // an RMSNorm spread over two products (see GemmParams)
@@ -870,7 +877,8 @@ static int gemm_entry(void* out, const void* x, const void* w, const float* bias
     TI_REQUIRE(link.scale_sums == nullptr || (M <= 64 && link.scale_parts > 0 && link.scale_dim > 0),
                "gemm_bf16: rows can be scaled by their rms for at most 64 tokens");
     TI_REQUIRE(K % 8 == 0, "gemm_bf16: K=%d is not a multiple of 8 (rows must start on 16-byte boundaries)", K);
-    TI_REQUIRE(!(gated && (bias || residual || out_f32)), "gemm_bf16: the gated form takes no bias, residual or float32 output");
+    TI_REQUIRE(!(gated && (residual || out_f32)), "gemm_bf16: the gated form takes no residual or float32 output");
+    TI_REQUIRE(!(gated && bias && link.scale_sums), "gemm_bf16: the gated form takes a bias or a norm link, not both");
     TI_REQUIRE(((uintptr_t)x & 15) == 0 && ((uintptr_t)w & 15) == 0, "gemm_bf16: operands must be 16-byte aligned");
     if (M == 0) return 0;
     GemmParams p;
@@ -898,7 +906,7 @@ static int gemm_entry(void* out, const void* x, const void* w, const float* bias
         // one trip and sharing only adds the wait: measured). Needs every unit running at once, and the
         // 16-byte path of the sum.
         const bool may_share = M >= 16 && (N & 3) == 0 &&
-                               (gated ? ((uintptr_t)out & 7) == 0
+                               (gated ? ((uintptr_t)out & 7) == 0 && ((uintptr_t)bias & 15) == 0
                                       : ((uintptr_t)out & 15) == 0 && ((uintptr_t)residual & 7) == 0 && ((uintptr_t)bias & 15) == 0);
         if (workspace && counters)
             p.splits = choose_splits(tiles, (K + BK - 1) / BK, bn, workspace_floats, num_counters, may_share);

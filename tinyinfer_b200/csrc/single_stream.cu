@@ -1,6 +1,9 @@
 // The residual of a pre-norm decoder kept as ONE float32 stream, with everything that may lie between two sublayers in one
 // kernel. With y the output of the sublayer before (compute dtype or float32):
 //     x <- x + factor * (scale * y)          scale: a number per feature ("layer scale"), factor: a constant
+//     x <- x + factor * y2                   y2: the output of a second sublayer that read the same input, either rows like y or
+//                                            a mixture's experts: moe_weight * sum_c moe_rows[moe_slots[t][c]] (float32 rows in
+//                                            expert order, the weighted sum with equal weights, made here and never stored)
 //     x <- x + add_rows[t] + add_vec         what a pass over a stretch of layers starts with (both optional)
 //     h  = norm_w * x / sqrt(mean(x^2) + eps)
 // and, with a token shift, h_t <- h_t + (h_(t-1) - h_t) * shift per feature, where h_(t-1) is the request's token before as
@@ -19,6 +22,8 @@ struct StreamStepArgs {
     const float* x_in;
     float* x_out;                          // may be x_in without a shift; null: the updated rows are not kept
     const void* y; const float* y_scale; float y_factor;
+    const void* y2;
+    const float* moe_rows; const int* moe_slots; int moe_top; float moe_weight;
     const float *add_rows, *add_vec;
     const float* norm_w; float eps;
     void* h;
@@ -71,6 +76,23 @@ __device__ __forceinline__ void updated_row(const StreamStepArgs& a, size_t t, i
         }
 #pragma unroll
         for (int e = 0; e < VEC; ++e) u[e] = fmaf(a.y_factor, y[e], u[e]);
+    }
+    if (a.y2) {
+        float y[VEC];
+        SsVec<VEC>::load((const TY*)a.y2 + t * a.width + i, y);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) u[e] = fmaf(a.y_factor, y[e], u[e]);
+    }
+    if (a.moe_rows) {
+        float y[VEC] = {};
+        for (int c = 0; c < a.moe_top; ++c) {
+            float r[VEC];
+            SsVec<VEC>::load(a.moe_rows + (size_t)a.moe_slots[t * a.moe_top + c] * a.width + i, r);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) y[e] += r[e];
+        }
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) u[e] = fmaf(a.y_factor * a.moe_weight, y[e], u[e]);
     }
     if (a.add_rows) {
         float r[VEC];
@@ -226,6 +248,35 @@ __global__ void __launch_bounds__(SS_MAX_THREADS) stream_shift_kernel(StreamStep
     }
 }
 
+// What a pass over a stretch of layers projects: the updated row beside the embedding's, as the operand row of a product. In
+// bfloat16 the float32 row travels as two halves, u = hi + lo (16 bits of mantissa instead of 8; the product's weight has the
+// columns for it twice): out row [hi | lo | x0]. In float32: [u | x0]. x0 = scale * table[token].
+template <typename TY, typename TO, int VEC>
+__global__ void __launch_bounds__(SS_MAX_THREADS) stream_enter_kernel(StreamStepArgs a, TO* __restrict__ out, const TO* __restrict__ table,
+                                                                      const int* __restrict__ token_ids, int vocab, float scale) {
+    ti_grid_launch_dependents();
+    ti_grid_wait();
+    const size_t t = blockIdx.x;
+    const int token = token_ids[t];
+    const bool known = token >= 0 && token < vocab;
+    constexpr int PARTS = sizeof(TO) == 4 ? 2 : 3;
+    TO* row = out + t * PARTS * a.width;
+    for (int i = threadIdx.x * VEC; i < a.width; i += blockDim.x * VEC) {
+        float u[VEC], x0[VEC] = {};
+        updated_row<TY, VEC>(a, t, i, u);
+        if (known) SsVec<VEC>::load(table + (size_t)token * a.width + i, x0);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x0[e] *= scale;
+        SsVec<VEC>::store(row + i, u);
+        if constexpr (PARTS == 3) {
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) u[e] -= to_f32(from_f32<TO>(u[e]));
+            SsVec<VEC>::store(row + a.width + i, u);
+        }
+        SsVec<VEC>::store(row + (PARTS - 1) * a.width + i, x0);
+    }
+}
+
 template <typename K>
 static int ss_smem(K kernel, size_t bytes) {
     if (bytes <= 40 * 1024) return 0;             // with the static arrays still under what needs no opt-in
@@ -234,12 +285,43 @@ static int ss_smem(K kernel, size_t bytes) {
     return 0;
 }
 
+// out [num_tokens][3 width] (bfloat16) or [num_tokens][2 width] (float32, dtype); the updates as in ti_stream_step.
+TI_API int ti_stream_enter(void* out, const float* x_in, const void* y, const float* y_scale, float y_factor, const void* y2,
+                           const float* moe_rows, const int* moe_slots, int moe_top, float moe_weight, const float* add_rows,
+                           const float* add_vec, const void* table, const int* token_ids, int vocab, float scale, int num_tokens,
+                           int width, int y_dtype, int dtype, cudaStream_t stream) {
+    TI_REQUIRE(num_tokens >= 0 && width > 0 && vocab > 0 && out && x_in && table && token_ids, "stream_enter: bad arguments");
+    TI_REQUIRE(!moe_rows || (moe_slots && moe_top > 0), "stream_enter: experts' rows come with their slots");
+    if (num_tokens == 0) return 0;
+    StreamStepArgs a = {x_in, nullptr, y, y_scale, y_factor, y2, moe_rows, moe_slots, moe_top, moe_weight, add_rows, add_vec, nullptr,
+                        0.f, nullptr, nullptr, nullptr, nullptr, 0, nullptr, nullptr, nullptr, num_tokens, width};
+    const uintptr_t all = (uintptr_t)x_in | (uintptr_t)y | (uintptr_t)y_scale | (uintptr_t)y2 | (uintptr_t)moe_rows |
+                          (uintptr_t)add_rows | (uintptr_t)add_vec | (uintptr_t)table | (uintptr_t)out;
+    const bool wide = width % 4 == 0 && all % 16 == 0;
+    int threads = 64;
+    while (threads < SS_MAX_THREADS && threads * 4 < width) threads <<= 1;
+    typedef __nv_bfloat16 B;
+#define SE_GO(TY, TO)                                                                                                             \
+    do {                                                                                                                          \
+        if (wide) ti_launch(stream_enter_kernel<TY, TO, 4>, num_tokens, threads, 0, stream, a, (TO*)out, (const TO*)table, token_ids, vocab, scale); \
+        else ti_launch(stream_enter_kernel<TY, TO, 1>, num_tokens, threads, 0, stream, a, (TO*)out, (const TO*)table, token_ids, vocab, scale);      \
+    } while (0)
+    if (y_dtype == TI_F32 && dtype == TI_F32) SE_GO(float, float);
+    else if (y_dtype == TI_F32 && dtype == TI_BF16) SE_GO(float, B);
+    else if (y_dtype == TI_BF16 && dtype == TI_BF16) SE_GO(B, B);
+    else TI_REQUIRE(false, "stream_enter: unknown dtypes %d, %d", y_dtype, dtype);
+#undef SE_GO
+    TI_CHECK_LAUNCH("stream_enter");
+    return 0;
+}
+
 // x_in, x_out float32 [num_tokens][width] (x_out null: not kept; with a shift it is not x_in). y (or null) with y_scale
-// (float32 [width], or null) and y_factor; add_rows float32 [num_tokens][width], add_vec float32 [width] (or null). h:
+// (float32 [width], or null) and y_factor; y2 (of y's dtype, or null), moe_rows float32 [slots][width] with moe_slots
+// [num_tokens][moe_top] and moe_weight (or null); add_rows float32 [num_tokens][width], add_vec float32 [width] (or null). h:
 // [num_rows][width]. shift (float32 [width], or null) with prev (slots of `width` floats, prev_stride apart), token_seq,
 // cu_seqlens and state_slots of the step.
-TI_API int ti_stream_step(const float* x_in, float* x_out, const void* y, const float* y_scale, float y_factor,
-                          const float* add_rows, const float* add_vec, const float* norm_w, float eps, void* h, const int* rows,
+TI_API int ti_stream_step(const float* x_in, float* x_out, const void* y, const float* y_scale, float y_factor, const void* y2,
+                          const float* moe_rows, const int* moe_slots, int moe_top, float moe_weight, const float* add_rows, const float* add_vec, const float* norm_w, float eps, void* h, const int* rows,
                           int num_rows, const float* shift, float* prev, long long prev_stride, const int* token_seq,
                           const int* cu_seqlens, const int* state_slots, int num_tokens, int width, int y_dtype, int h_dtype,
                           cudaStream_t stream) {
@@ -248,11 +330,12 @@ TI_API int ti_stream_step(const float* x_in, float* x_out, const void* y, const 
     TI_REQUIRE(!shift || (!rows && num_rows == num_tokens && prev && token_seq && cu_seqlens && state_slots && x_out != x_in),
                "stream_step: a token shift works on all of a step's tokens, from one buffer into another");
     TI_REQUIRE(!rows || !x_out, "stream_step: chosen rows are not stored back");
+    TI_REQUIRE(!moe_rows || (moe_slots && moe_top > 0), "stream_step: experts' rows come with their slots");
     if (num_rows == 0) return 0;
-    StreamStepArgs a = {x_in, x_out, y, y_scale, y_factor, add_rows, add_vec, norm_w, eps, h, rows, shift, prev, prev_stride,
+    StreamStepArgs a = {x_in, x_out, y, y_scale, y_factor, y2, moe_rows, moe_slots, moe_top, moe_weight, add_rows, add_vec, norm_w, eps, h, rows, shift, prev, prev_stride,
                         token_seq, cu_seqlens, state_slots, num_tokens, width};
-    const uintptr_t all = (uintptr_t)x_in | (uintptr_t)x_out | (uintptr_t)y | (uintptr_t)y_scale | (uintptr_t)add_rows |
-                          (uintptr_t)add_vec | (uintptr_t)norm_w | (uintptr_t)h | (uintptr_t)shift | (uintptr_t)prev;
+    const uintptr_t all = (uintptr_t)x_in | (uintptr_t)x_out | (uintptr_t)y | (uintptr_t)y_scale | (uintptr_t)y2 | (uintptr_t)moe_rows |
+                          (uintptr_t)add_rows | (uintptr_t)add_vec | (uintptr_t)norm_w | (uintptr_t)h | (uintptr_t)shift | (uintptr_t)prev;
     const bool wide = width % 4 == 0 && all % 16 == 0 && (!shift || prev_stride % 4 == 0);
     int threads = 64;
     while (threads < SS_MAX_THREADS && threads * 4 < width) threads <<= 1;

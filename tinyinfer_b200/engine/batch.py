@@ -68,6 +68,8 @@ class StepContext:
     feed_dst: Optional[torch.Tensor] = None
     feed_src: Optional[torch.Tensor] = None
     num_feeds: int = 0
+    # filled by the model at the start of a step: the routing of feed-forwards that depends on the token ids alone
+    routings: Dict = field(default_factory=dict)
     # filled by the runner: entry of the run order -> CacheView
     views: Dict[int, CacheView] = field(default_factory=dict)
 

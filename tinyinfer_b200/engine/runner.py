@@ -187,7 +187,7 @@ class ModelRunner:
             for part in (block, block.mixer, block.feed_forward, block.mixer_norm, block.feed_forward_norm):
                 if part is not None:
                     let_go(part)
-        self.model.embedding = self.model.head = None
+        self.model.embedding = self.model.head = self.model.entry_weight = self.model.table_routes = None
         ops.release_scratch(self.device)
         if self.device.type == "cuda":
             import gc

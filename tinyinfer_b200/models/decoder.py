@@ -15,6 +15,7 @@ import torch
 
 from .. import ops
 from ..config.specs import ModelSpec
+from ..parts.experts import TableRoutes
 from ..parts import CacheNeed, StateNeed, TensorSpec, build_block, build_norm
 
 
@@ -29,6 +30,8 @@ class DecoderModel:
         self.final_norm = build_norm(spec.final_norm, dtype, self.device)
         self.embedding: Optional[torch.Tensor] = None
         self.head: Optional[torch.Tensor] = None
+        self.entry_weight: Optional[torch.Tensor] = None      # of the entries that project [x; embedding]
+        self.table_routes: Optional[TableRoutes] = None       # feed-forwards whose routing depends on the token ids alone
         self.step_vectors: Optional[torch.Tensor] = None      # float32 [rows, hidden]: what entries of the run order add
 
     # ------------------------------------------------------------------ tensors
@@ -52,6 +55,8 @@ class DecoderModel:
             for prefix, part in self._part_prefixes(i):
                 for local, ts in part.tensors().items():
                     out[prefix + local] = ts
+        if spec.entry_projection:
+            out[spec.entry_projection] = TensorSpec((spec.hidden_size, 2 * spec.hidden_size))
         if spec.step_vectors:
             out[spec.step_vectors[0]] = TensorSpec((spec.step_vectors[1], spec.hidden_size), role="vector32")
         for local, ts in self.final_norm.tensors().items():
@@ -76,6 +81,10 @@ class DecoderModel:
         for i in range(len(self.blocks)):
             for prefix, part in self._part_prefixes(i):
                 part.load({local: tensors[prefix + local] for local in part.tensors()})
+        table_parts = [b.feed_forward for b in self.blocks if getattr(b.feed_forward, "table", None) is not None]
+        self.table_routes = TableRoutes(table_parts) if table_parts else None
+        if spec.entry_projection:
+            self.load_entry_projection(tensors[spec.entry_projection])
         if spec.step_vectors:
             self.step_vectors = tensors[spec.step_vectors[0]].contiguous()
         self.final_norm.load({local: tensors[spec.names.final_norm + local]
@@ -109,6 +118,8 @@ class DecoderModel:
     def forward(self, step) -> torch.Tensor:
         """Runs the tokens of ``step`` (a StepContext) and returns float32 logits [N, V] at
         ``step.logit_rows``."""
+        if self.table_routes is not None:
+            self.table_routes.route(step)
         x = self.run_blocks(self.embed(step), step)
         if step.num_logit_rows == 0:
             return torch.empty((0, self.spec.vocab_size), dtype=torch.float32, device=self.device)
@@ -123,14 +134,18 @@ class DecoderModel:
         link = None        # what a block's last product leaves for the next block's first norm (see parts.base)
         order = self.spec.execution
         for i, entry in enumerate(order):
-            if entry.adds_embedding or entry.adds_vector is not None:
-                x, link = self.enter(x, entry), None
+            if entry.adds_embedding or entry.projects_embedding or entry.adds_vector is not None:
+                x, link = self.enter(x, entry, step), None
             after = self.blocks[order[i + 1].layer].mixer_norm if i + 1 < len(order) else None
             x, link = self.blocks[entry.layer].forward_linked(x, link, after, step, step.cache_view(entry))
         return x
 
-    def enter(self, x, entry):
-        """What an entry of the run order adds to the residual right before its layer."""
+    def load_entry_projection(self, weight: torch.Tensor) -> None:
+        """``weight`` [hidden, 2 hidden] of the entries that project [x; embedding]."""
+        self.entry_weight = weight.contiguous()
+
+    def enter(self, x, entry, step=None):
+        """What an entry of the run order does to the residual right before its layer."""
         raise NotImplementedError(f"{type(self).__name__} has no residual that an entry of the run order could add to")
 
     def logits(self, x: torch.Tensor, step) -> torch.Tensor:
@@ -171,13 +186,30 @@ class ScaledResidualDecoderModel(DecoderModel):
     """The frame of the decoders whose blocks are 'scaled_residual' blocks: the embedding times a constant starts one
     float32 stream [T, width]; what travels between the blocks is the pair (stream, update still to be applied). Entries of
     the run order may add the embedding's output and a row of the step vectors before their layer; both ride in the update.
-    At the end the last update, the final norm and the choice of the wanted rows are one kernel, then the head."""
+    Entries may also replace the stream by W [x; x0], x0 being the embedding's output: one kernel applies the update and lays
+    the operand rows out, a product makes the new stream. In a bfloat16 model x travels there as two halves, x = hi + lo, so
+    that the residual never passes through 16 bits.
+    At the end the last update, the final norm and the choice of the wanted rows are one kernel, then the head; a constant
+    factor on the logits rides in the final norm's weight."""
 
-    def __init__(self, spec: ModelSpec, dtype, device, *, embedding_scale: float = 1.0):
+    def __init__(self, spec: ModelSpec, dtype, device, *, embedding_scale: float = 1.0, logit_scale: float = 1.0):
         super().__init__(spec, dtype, device)
         self.embedding_scale = float(embedding_scale)
+        self.logit_scale = float(logit_scale)
+        self._logit_norm = None
         self._needs_start = any(e.adds_embedding for e in spec.execution)
         self._start = None
+
+    def load_tensors(self, tensors) -> None:
+        super().load_tensors(tensors)
+        weight = self.final_norm.as_rms()[0]
+        self._logit_norm = weight if self.logit_scale == 1.0 else (weight * self.logit_scale).contiguous()
+
+    def load_entry_projection(self, weight):
+        if self.dtype == torch.bfloat16:                  # the columns of x twice: for its upper and its lower half
+            w = self.spec.hidden_size
+            weight = torch.cat([weight[:, :w], weight], dim=1)
+        super().load_entry_projection(weight)
 
     def embed(self, step):
         # the stream is updated in place: where later entries add what it started from, the kernel makes a second copy
@@ -191,8 +223,13 @@ class ScaledResidualDecoderModel(DecoderModel):
         finally:
             self._start = None
 
-    def enter(self, x, entry):
+    def enter(self, x, entry, step=None):
         stream, pending = x
+        if entry.projects_embedding:
+            if entry.adds_embedding or entry.adds_vector is not None:
+                raise ValueError("an entry projects the embedding or adds it, not both")
+            rows = ops.residual_enter(stream, pending, self.embedding, step.token_ids, self.embedding_scale)
+            return ops.linear(rows, self.entry_weight, out_float32=True), None
         pending = pending if pending is not None else ops.ResidualUpdate()
         pending.add_rows = self._start if entry.adds_embedding else None
         pending.add_vec = self.step_vectors[entry.adds_vector] if entry.adds_vector is not None else None
@@ -200,6 +237,5 @@ class ScaledResidualDecoderModel(DecoderModel):
 
     def logits(self, x, step):
         stream, pending = x
-        rms = self.final_norm.as_rms()
-        _, h = ops.residual_step(stream, pending, rms[0], rms[1], self.dtype, rows=step.logit_rows)
+        _, h = ops.residual_step(stream, pending, self._logit_norm, self.final_norm.as_rms()[1], self.dtype, rows=step.logit_rows)
         return ops.linear(h, self.head, out_float32=True)

@@ -76,6 +76,8 @@ _SIGNATURES = {
         "ti_moe_route": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                          c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
                          c_int, c_float, c_int, c_int, c_void_p],
+        "ti_moe_route_table": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                               c_int, c_int, c_int, c_void_p],
         "ti_moe_tile_rows": [],
         "ti_moe_gemm": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                         c_void_p],
@@ -95,13 +97,16 @@ _SIGNATURES = {
         "ti_soft_cap": [c_void_p, c_ll, c_float, c_void_p],
         "ti_head_rotation": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p,
                              c_void_p, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int,
-                             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
+                             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int,
+                             c_void_p],
         "ti_delta_scan": [c_void_p, c_void_p, c_ll, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int,
                           c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_float, c_float, c_void_p,
                           c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_ll, c_int, c_void_p],
         "ti_streams_step": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int,
                             c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p],
-        "ti_stream_step": [c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_float, c_void_p,
+        "ti_stream_enter": [c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_float, c_void_p,
+                            c_void_p, c_void_p, c_void_p, c_int, c_float, c_int, c_int, c_int, c_int, c_void_p],
+        "ti_stream_step": [c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_float, c_void_p, c_void_p, c_void_p, c_float, c_void_p,
                            c_void_p, c_int, c_void_p, c_void_p, c_ll, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                            c_void_p],
         "ti_qkv_prepare": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_ll, c_int, c_int, c_int,
@@ -122,8 +127,8 @@ _SIGNATURES = {
                                c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                                c_int, c_int, c_void_p, c_int, c_void_p],
         "ti_attention_rows": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                              c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_float, c_void_p, c_void_p, c_int, c_int,
-                              c_float, c_float, c_void_p, c_int, c_void_p],
+                              c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_int, c_int,
+                              c_int, c_float, c_float, c_int, c_float, c_float, c_void_p, c_int, c_void_p],
         "ti_linear_scan": [c_void_p, c_void_p, c_ll, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int,
                            c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p, c_float, c_void_p,
                            c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_ll, c_void_p, c_int, c_void_p],
@@ -159,15 +164,16 @@ _SIGNATURES["sm100"]["ti_attention_decode_bf16"] = [
     c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p]
 _SIGNATURES["sm100"]["ti_attention_decode_sink_bf16"] = [
     c_void_p, c_void_p, c_void_p, c_void_p, c_ll, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
-    c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p, c_int, c_int,
-    c_float, c_void_p, c_void_p]
+    c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p, c_int, c_int,
+    c_int, c_float, c_int, c_float, c_float, c_void_p, c_void_p]
 _SIGNATURES["sm100"]["ti_attention_prefill_pair_sink_bf16"] = [
     c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-    c_float, c_int, c_int, c_float, c_float, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p]
+    c_float, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_int, c_float,
+    c_float, c_void_p, c_void_p]
 _SIGNATURES["sm100"]["ti_attention_prefill_tc_sink_bf16"] = [
     c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-    c_float, c_int, c_int, c_int, c_int, c_void_p, c_ll, c_int, c_float, c_float, c_void_p, c_void_p, c_int, c_int,
-    c_float, c_void_p, c_void_p]
+    c_float, c_int, c_int, c_int, c_int, c_int, c_void_p, c_ll, c_int, c_float, c_float, c_void_p, c_void_p, c_int, c_int,
+    c_int, c_float, c_void_p, c_void_p]
 _SIGNATURES["sm100"]["ti_attention_decode_scratch_floats"] = [c_int, c_int, c_int, c_int, c_int, c_int]
 _SIGNATURES["sm100"]["ti_attention_prefill_pair_bf16"] = [
     c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
@@ -453,8 +459,8 @@ GATED_ACTIVATIONS = {"silu": 1, "gelu_tanh": 2}
 
 
 def gated_linear(x: torch.Tensor, w_gate_up: torch.Tensor, *, link: Optional[NormLink] = None,
-                 link_eps: float = 0.0, activation: str = "silu") -> torch.Tensor:
-    """act(x.Wg^T) * (x.Wu^T) with ``w_gate_up`` = [Wg; Wu] of shape [2I, K] -> [M, I]; the
+                 link_eps: float = 0.0, activation: str = "silu", bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """act(x.Wg^T + bg) * (x.Wu^T + bu) (``bias`` float32 [2I] = [bg | bu], or None) with ``w_gate_up`` = [Wg; Wu] of shape [2I, K] -> [M, I]; the
     activation ('silu' or 'gelu_tanh') and the product act on the float32 accumulators, one rounding. ``link``: as in
     ``linear`` (both halves are scaled before the activation)."""
     if activation not in GATED_ACTIVATIONS:
@@ -466,23 +472,25 @@ def gated_linear(x: torch.Tensor, w_gate_up: torch.Tensor, *, link: Optional[Nor
     if w_gate_up.shape[1] != k or w_gate_up.shape[0] % 2:
         raise KernelError("gated_linear: weight must be [2I, K]")
     inter = w_gate_up.shape[0] // 2
+    if bias is not None and _check(bias, "bias", torch.float32, 1).shape[0] != 2 * inter:
+        raise KernelError("gated_linear: a bias for every row of the weight")
     out = torch.empty((m, inter), dtype=x.dtype, device=x.device)
     if link is not None:
-        if not (_tensor_core_ok(x, w_gate_up) and norm_link_ok(x)):
+        if bias is not None or not (_tensor_core_ok(x, w_gate_up) and norm_link_ok(x)):
             raise KernelError("gated_linear: a norm link needs the tensor-core product of at most 64 rows")
         _gemm_linked(out, x, w_gate_up, None, None, m, inter, k, act, (link, link_eps), None)
         return out
     if _tensor_core_ok(x, w_gate_up) and m >= PAIR_MIN_TOKENS and inter >= 128:
-        _run("sm100", "ti_gemm_pair_bf16", out.data_ptr(), x.data_ptr(), w_gate_up.data_ptr(), None, None,
+        _run("sm100", "ti_gemm_pair_bf16", out.data_ptr(), x.data_ptr(), w_gate_up.data_ptr(), _ptr(bias), None,
              m, inter, k, act, 0, kernel_status(x.device).data_ptr(), _stream())
         return out
     if _tensor_core_ok(x, w_gate_up):
         ws, counters = _gemm_scratch(x.device)
-        _run("sm100", "ti_gemm_bf16", out.data_ptr(), x.data_ptr(), w_gate_up.data_ptr(), None, None,
+        _run("sm100", "ti_gemm_bf16", out.data_ptr(), x.data_ptr(), w_gate_up.data_ptr(), _ptr(bias), None,
              m, inter, k, act, 0, ws.data_ptr(), ws.numel(), counters.data_ptr(), counters.numel(),
              kernel_status(x.device).data_ptr(), _stream())
         return out
-    _run("core", "ti_gemm_simt", out.data_ptr(), x.data_ptr(), w_gate_up.data_ptr(), None, None,
+    _run("core", "ti_gemm_simt", out.data_ptr(), x.data_ptr(), w_gate_up.data_ptr(), _ptr(bias), None,
          m, inter, k, act, 0, _dtype_code(x), _stream())
     return out
 
@@ -588,12 +596,12 @@ def plan_attention(q_lens, starts):
     return decode_rows, [x for t in pairs + singles for x in t], len(pairs)
 
 
-def attention_tensor_cores_ok(q: torch.Tensor, kv_cache: torch.Tensor) -> bool:
-    """The tensor-core attention kernels take bfloat16, head sizes 64 and 128, up to 16 query heads
-    per kv head, and pages of 16, 32 or a multiple of 64 tokens."""
+def attention_tensor_cores_ok(q: torch.Tensor, kv_cache: torch.Tensor, maps: int = 1) -> bool:
+    """The tensor-core attention kernels take bfloat16, head sizes 64 and 128, up to 16 query heads (or, with two maps a
+    head, 8) per kv head, and pages of 16, 32 or a multiple of 64 tokens."""
     _, hq, d = q.shape
     hkv, page = kv_cache.shape[2], kv_cache.shape[3]
-    return (q.dtype == torch.bfloat16 and d in (64, 128) and hq % hkv == 0 and hq // hkv <= 16
+    return (q.dtype == torch.bfloat16 and d in (64, 128) and hq % hkv == 0 and hq // hkv * maps <= 16
             and (page in (16, 32) or page % 64 == 0))
 
 
@@ -664,12 +672,19 @@ def _mask_code(window: Optional[int], chunk: Optional[int]) -> int:
     return int(window or 0) or -int(chunk or 0)
 
 
+def _keep_first(keep_first: int, window: Optional[int]) -> int:
+    if keep_first < 0 or (keep_first and not window):
+        raise KernelError("attention: first positions are kept beside a window")
+    return int(keep_first)
+
+
 def paged_attention(q: torch.Tensor, kv_cache: torch.Tensor, *, positions: torch.Tensor,
                     token_seq: torch.Tensor, block_table: torch.Tensor, scale: float,
                     window: Optional[int] = None, chunk: Optional[int] = None, step=None,
                     status: Optional[torch.Tensor] = None, sink: Optional[float] = None,
                     out_scale: float = 1.0, head_sinks: Optional[torch.Tensor] = None,
-                    gate: Optional[torch.Tensor] = None, gate_offset: int = 0, softcap: float = 0.0) -> torch.Tensor:
+                    gate: Optional[torch.Tensor] = None, gate_offset: int = 0, softcap: float = 0.0,
+                    keep_first: int = 0, feature_gate: bool = False, difference: Optional[tuple] = None) -> torch.Tensor:
     """Causal attention of q [T, Hq, D] over the pages of each token's own request.
     Token t sees keys max(0, pos - window + 1) .. pos of request ``token_seq[t]``, or, with ``chunk``, those from
     floor(pos / chunk) * chunk on.
@@ -677,6 +692,11 @@ def paged_attention(q: torch.Tensor, kv_cache: torch.Tensor, *, positions: torch
     of exp(score)); ``head_sinks`` float32 [Hq]: such a logit per query head instead; ``gate`` [T, cols] of q's dtype:
     the output of (token, head) is multiplied by sigmoid(gate[token, gate_offset + head]); ``out_scale``: a factor on
     the output before its rounding; ``softcap`` > 0: a score s becomes softcap * tanh(s / softcap) before the softmax.
+    ``keep_first``: a window keeps the request's first so many positions; ``feature_gate``: the gate has a column per output
+    feature, feature f of the heads side by side is multiplied by sigmoid(gate[token, gate_offset + f]).
+    ``difference`` (share, eps), differential attention: the D features of a query head and of a key are two maps of D / 2
+    features, each with a softmax of its own over the same values; with the maps' outputs a1 and a2, o = a1 - share * a2 is
+    divided by its root mean square over the head's features and multiplied by ``out_scale``.
     Returns [T, Hq * D]. ``step`` (the StepContext of the batch) carries the split of the batch
     into decoded tokens and prompt portions; without it the split is derived here (a device read)."""
     _check(q, "q", None, 3)
@@ -693,15 +713,23 @@ def paged_attention(q: torch.Tensor, kv_cache: torch.Tensor, *, positions: torch
         return out
     mask = _mask_code(window, chunk)
     has_sink, sink_v = int(sink is not None), float(sink or 0.0)
-    _check_head_extras(q, head_sinks, gate, gate_offset)
-    extras = (_ptr(head_sinks), _ptr(gate), gate.shape[1] if gate is not None else 0, int(gate_offset), float(softcap or 0.0))
-    if not attention_tensor_cores_ok(q, kv_cache):
+    _check_head_extras(q, head_sinks, gate, gate_offset, d if feature_gate else 1)
+    maps, share, diff_eps = (1, 0.0, 0.0) if difference is None else (2, float(difference[0]), float(difference[1]))
+    if maps == 2 and (d % 2 or has_sink or head_sinks is not None):
+        raise KernelError("paged_attention: two maps have equal halves of the features and no sinks")
+    keep = _keep_first(keep_first, window)
+    extras = (_ptr(head_sinks), _ptr(gate), gate.shape[1] if gate is not None else 0, int(gate_offset), int(feature_gate),
+              float(softcap or 0.0))
+    two_maps = (maps, share, diff_eps)
+    aligned = not feature_gate or (gate.shape[1] % 8 == 0 and gate_offset % 8 == 0 and gate.data_ptr() % 16 == 0)
+    if not attention_tensor_cores_ok(q, kv_cache, maps) or not aligned:
         if q.dtype == torch.bfloat16:
             _warn_generic_attention(hq, hkv, d, page_size)
-        if softcap or has_sink or out_scale != 1.0 or head_sinks is not None or gate is not None:
+        if softcap or has_sink or out_scale != 1.0 or head_sinks is not None or gate is not None or keep or maps == 2:
             return attention_rows(q, kv_cache, v_dim=d, positions=positions, token_seq=token_seq, block_table=block_table,
                                   scale=scale, sink=sink, window=window, chunk=chunk, out_scale=out_scale, status=status,
-                                  head_sinks=head_sinks, gate=gate, gate_offset=gate_offset, softcap=softcap)
+                                  head_sinks=head_sinks, gate=gate, gate_offset=gate_offset, softcap=softcap,
+                                  keep_first=keep_first, feature_gate=feature_gate, difference=difference)
         _run("core", "ti_attention_generic", out.data_ptr(), q.data_ptr(), kv_cache.data_ptr(),
              positions.data_ptr(), token_seq.data_ptr(), block_table.data_ptr(), block_table.shape[1],
              t, hq, hkv, d, page_size, num_pages, float(scale), mask, _ptr(status),
@@ -733,11 +761,11 @@ def paged_attention(q: torch.Tensor, kv_cache: torch.Tensor, *, positions: torch
         num_decode, num_tiles, max_context = len(rows_l), len(tiles_l) // 4, max(pos_h) + 1
     kstatus = kernel_status(q.device).data_ptr()
     if num_decode:
-        scratch = _decode_scratch(q.device, decode_scratch_floats(num_decode, hq, hkv, d, max_context, mask))
+        scratch = _decode_scratch(q.device, decode_scratch_floats(num_decode, hq * maps, hkv, d, max_context, mask))
         _run("sm100", "ti_attention_decode_sink_bf16", out.data_ptr(), q.data_ptr(), kv_cache.data_ptr(),
              scratch.data_ptr(), scratch.numel(), decode_rows.data_ptr(), num_decode, positions.data_ptr(),
              token_seq.data_ptr(), block_table.data_ptr(), block_table.shape[1], hq, hkv, d, page_size,
-             num_pages, float(scale), mask, int(max_context), has_sink, sink_v, float(out_scale), *extras,
+             num_pages, float(scale), mask, keep, int(max_context), has_sink, sink_v, float(out_scale), *extras, *two_maps,
              kstatus, _stream())
     def one_tile_kernel(first: int, count: int, halves: int) -> None:
         # Few query tiles behind a long prefix: the keys are shared out over CTAs too (at least 1,024 to a CTA),
@@ -753,13 +781,23 @@ def paged_attention(q: torch.Tensor, kv_cache: torch.Tensor, *, positions: torch
             scratch_ptr, scratch_floats = scratch.data_ptr(), scratch.numel()
         _run("sm100", "ti_attention_prefill_tc_sink_bf16", out.data_ptr(), q.data_ptr(), kv_cache.data_ptr(),
              tiles.data_ptr() + 16 * first, count, t, block_table.data_ptr(), block_table.shape[1], hq, hkv, d, page_size,
-             num_pages, float(scale), mask, halves, splits, split_keys, scratch_ptr, scratch_floats, has_sink,
+             num_pages, float(scale), mask, keep, halves, splits, split_keys, scratch_ptr, scratch_floats, has_sink,
              sink_v, float(out_scale), *extras, kstatus, _stream())
 
-    if num_pairs * hq >= PAIR_MIN_CTAS:             # two query tiles a CTA
+    def two_tile_kernel(first: int, count: int, halves: int) -> None:
         _run("sm100", "ti_attention_prefill_pair_sink_bf16", out.data_ptr(), q.data_ptr(), kv_cache.data_ptr(),
-             tiles.data_ptr(), num_pairs, t, block_table.data_ptr(), block_table.shape[1], hq, hkv, d, page_size,
-             num_pages, float(scale), mask, has_sink, sink_v, float(out_scale), *extras, kstatus, _stream())
+             tiles.data_ptr() + 16 * first, count, t, block_table.data_ptr(), block_table.shape[1], hq, hkv, d, page_size,
+             num_pages, float(scale), mask, keep, has_sink, sink_v, float(out_scale), *extras, maps, halves, share, diff_eps,
+             kstatus, _stream())
+
+    if maps == 2:                                   # a CTA's two tiles are the two maps of the same 128 rows
+        if num_pairs:
+            two_tile_kernel(0, num_pairs, 1)
+        if num_tiles > num_pairs:
+            two_tile_kernel(num_pairs, num_tiles - num_pairs, 0)
+        return out
+    if num_pairs * hq >= PAIR_MIN_CTAS:             # two query tiles a CTA
+        two_tile_kernel(0, num_pairs, 0)
     elif num_pairs:                                 # too few of them to fill the machine: one query tile a CTA
         one_tile_kernel(0, num_pairs, 1)
     if num_tiles > num_pairs:                       # ends of portions of at most 128 rows
@@ -1098,6 +1136,34 @@ def route_experts(x32: torch.Tensor, w_router: torch.Tensor, top: int, weight_ep
                          num_tiles, max_tiles, counts, tile_rows, slot_weight)
 
 
+class ExpertRows:
+    """A mixture's output not summed yet: weight * sum_c rows[slots[t, c]] (``rows`` float32 [T * top, H] in expert order,
+    ``slots`` int32 [T, top], one weight for all)."""
+
+    def __init__(self, rows: torch.Tensor, slots: torch.Tensor, weight: float):
+        self.rows, self.slots, self.weight = rows, slots, float(weight)
+
+
+def route_by_tables(token_ids: torch.Tensor, tables: torch.Tensor, num_experts: int, tile_rows: int) -> list:
+    """The routing of several mixtures without routers from a step's token ids alone, in one launch: ``tables`` int32
+    [layers, V, top], row i of a layer's table naming the experts of token id i, each of weight 1 / top. Returns an
+    ``ExpertRouting`` per layer."""
+    _check(token_ids, "token_ids", torch.int32, 1)
+    _check(tables, "tables", torch.int32, 3)
+    t, (layers, vocab, top) = token_ids.shape[0], tables.shape
+    n, max_tiles = t * top, (t * top + tile_rows - 1) // tile_rows + num_experts
+    ints = torch.empty(layers * (3 * n + 3 * max_tiles + 1), dtype=torch.int32, device=tables.device)
+    chosen, slot_of, token_of = (ints[i * layers * n:(i + 1) * layers * n].view(layers, n) for i in range(3))
+    at = 3 * layers * n
+    tiles = ints[at:at + layers * 3 * max_tiles].view(layers, max_tiles, 3)
+    num_tiles = ints[at + layers * 3 * max_tiles:].view(layers, 1)
+    _run("experts", "ti_moe_route_table", chosen.data_ptr(), slot_of.data_ptr(), token_of.data_ptr(), tiles.data_ptr(),
+         num_tiles.data_ptr(), token_ids.data_ptr(), tables.data_ptr(), layers, t, vocab, top, num_experts, int(tile_rows), max_tiles,
+         _stream())
+    return [ExpertRouting(chosen[i].view(t, top), None, slot_of[i].view(t, top), token_of[i], tiles[i], num_tiles[i], max_tiles, None,
+                          tile_rows) for i in range(layers)]
+
+
 def expert_tiles_may_be_wide(x: torch.Tensor, *inner_sizes: int) -> bool:
     """True if the grouped products of ``x`` [T, K] (and of rows of the given other sizes) run on the tensor cores,
     which alone take row tiles of 64."""
@@ -1110,12 +1176,17 @@ EXPERT_TCGEN05_MIN_ROWS = 96     # rows an expert gets on average from which the
 def expert_tile_rows(x: torch.Tensor, num_experts: int, top: int, *inner_sizes: int) -> int:
     """The height of the row tiles that the grouped products of a step should be planned with: 128 (tcgen05: many
     rows an expert, bfloat16, whole k blocks of 64), 64 or 32 (the warp-level tensor-core tiles; 32 also float32)."""
-    t = x.shape[0]
-    if x.dtype == torch.bfloat16 and t * top >= EXPERT_TCGEN05_MIN_ROWS * num_experts:
+    return expert_tile_rows_of(x.shape[0], x.shape[1], x.dtype, num_experts, top, *inner_sizes)
+
+
+def expert_tile_rows_of(t: int, hidden: int, dtype: torch.dtype, num_experts: int, top: int, *inner_sizes: int) -> int:
+    """``expert_tile_rows`` for a step of ``t`` tokens whose rows are not there yet."""
+    bf16 = dtype == torch.bfloat16
+    if bf16 and t * top >= EXPERT_TCGEN05_MIN_ROWS * num_experts:
         ok = _fn("sm100", "ti_moe_gemm_tcgen05_ok")
-        if all(int(ok(t * top, num_experts, n, k)) for n, k in ((inner_sizes[0], x.shape[1]), (x.shape[1], inner_sizes[0]))):
+        if all(int(ok(t * top, num_experts, n, k)) for n, k in ((inner_sizes[0], hidden), (hidden, inner_sizes[0]))):
             return int(_fn("sm100", "ti_moe_tcgen05_tile_rows")())
-    if t * top >= 48 * num_experts and expert_tiles_may_be_wide(x, *inner_sizes):
+    if t * top >= 48 * num_experts and all(int(_fn("experts", "ti_moe_wide_tiles_ok")(k, int(bf16))) for k in (hidden,) + inner_sizes):
         return 64
     return int(_fn("experts", "ti_moe_tile_rows")())
 
@@ -1218,6 +1289,8 @@ def experts_combine(down: torch.Tensor, x: torch.Tensor, routing: ExpertRouting,
             raise KernelError("experts_combine: the gate belongs to a shared expert and has a number per feature")
     _check(x, "x", None, 2)
     t, size = x.shape
+    if weighted and routing.weight is None:          # equal weights of a table's experts
+        routing.weight = torch.full(routing.chosen.shape, 1.0 / routing.chosen.shape[1], dtype=torch.float32, device=x.device)
     if down.shape[1] != size or routing.chosen.shape[0] != t:
         raise KernelError("experts_combine: the rows do not fit the routing")
     out = torch.empty_like(x)
@@ -1286,12 +1359,58 @@ def streams_step(x: torch.Tensor, pending: Optional[StreamUpdate], read_in: Opti
 
 class ResidualUpdate:
     """What lies between two sublayers of a decoder with one float32 residual stream x [T, W], applied by the next
-    ``residual_step``: x <- x + factor * (scale * y), ``scale`` float32 [W] or None; then x <- x + add_rows + add_vec
+    ``residual_step``: x <- x + factor * (scale * y), ``scale`` float32 [W] or None; x <- x + factor * second, the output of a
+    sublayer beside the first (rows of y's dtype, or ``ExpertRows``); then x <- x + add_rows + add_vec
     (float32 [T, W] and [W], or None)."""
 
     def __init__(self, y: Optional[torch.Tensor] = None, scale: Optional[torch.Tensor] = None, factor: float = 1.0,
-                 add_rows: Optional[torch.Tensor] = None, add_vec: Optional[torch.Tensor] = None):
+                 add_rows: Optional[torch.Tensor] = None, add_vec: Optional[torch.Tensor] = None, second=None):
         self.y, self.scale, self.factor, self.add_rows, self.add_vec = y, scale, float(factor), add_rows, add_vec
+        self.second = second
+
+    def launch_args(self, t: int, width: int):
+        """The kernels' arguments for the update, checked: y, scale, factor, y2, experts' rows, slots, top and weight,
+        add_rows, add_vec."""
+        rows = self.second if isinstance(self.second, ExpertRows) else None
+        y2 = None if rows is not None else self.second
+        for name, ten, shape, dtype in (("y", self.y, (t, width), None), ("scale", self.scale, (width,), torch.float32),
+                                        ("second", y2, (t, width), self.y.dtype if self.y is not None else None),
+                                        ("add_rows", self.add_rows, (t, width), torch.float32),
+                                        ("add_vec", self.add_vec, (width,), torch.float32)):
+            if ten is not None and tuple(_check(ten, name, dtype).shape) != shape:
+                raise KernelError(f"residual update: {name} has shape {tuple(ten.shape)}, not {shape}")
+        if y2 is not None and self.y is None:
+            raise KernelError("residual update: a second sublayer's rows come beside a first one's")
+        top = 0
+        if rows is not None:
+            top = _check(rows.slots, "slots", torch.int32, 2).shape[1]
+            if rows.slots.shape[0] != t or tuple(_check(rows.rows, "rows", torch.float32, 2).shape) != (t * top, width):
+                raise KernelError("residual update: the experts' rows do not fit the stream")
+        return (_ptr(self.y), _ptr(self.scale), self.factor, _ptr(y2), _ptr(rows.rows) if rows is not None else None,
+                _ptr(rows.slots) if rows is not None else None, top, rows.weight if rows is not None else 0.0,
+                _ptr(self.add_rows), _ptr(self.add_vec))
+
+    @property
+    def changes(self) -> bool:
+        return any(v is not None for v in (self.y, self.second, self.add_rows, self.add_vec))
+
+
+def residual_enter(x: torch.Tensor, pending: Optional[ResidualUpdate], table: torch.Tensor, token_ids: torch.Tensor,
+                   scale: float = 1.0) -> torch.Tensor:
+    """The operand rows of the product W [x; x0] that replaces the stream x float32 [T, W]: with the pending update applied (x
+    itself stays as it was) and x0 = scale * table[token_ids], rows [hi | lo | x0] of ``table``'s bfloat16 with x = hi + lo, or
+    [x | x0] of float32."""
+    _check(x, "x", torch.float32, 2)
+    _check(token_ids, "token_ids", torch.int32, 1)
+    t, width = x.shape
+    if _check(table, "table", None, 2).shape[1] != width or token_ids.shape[0] != t:
+        raise KernelError("residual_enter: the embedding does not fit the stream")
+    p = pending if pending is not None else ResidualUpdate()
+    out = torch.empty((t, (2 if table.dtype == torch.float32 else 3) * width), dtype=table.dtype, device=x.device)
+    _run("hybrid", "ti_stream_enter", out.data_ptr(), x.data_ptr(), *p.launch_args(t, width), table.data_ptr(), token_ids.data_ptr(),
+         table.shape[0], float(scale), t, width, _dtype_code(p.y) if p.y is not None else _dtype_code(table), _dtype_code(table),
+         _stream())
+    return out
 
 
 def residual_step(x: torch.Tensor, pending: Optional[ResidualUpdate], norm_weight: torch.Tensor, eps: float,
@@ -1307,15 +1426,13 @@ def residual_step(x: torch.Tensor, pending: Optional[ResidualUpdate], norm_weigh
     t, width = x.shape
     _check(norm_weight, "norm_weight", torch.float32, 1)
     p = pending if pending is not None else ResidualUpdate()
-    for name, ten, shape, dtype in (("y", p.y, (t, width), None), ("scale", p.scale, (width,), torch.float32),
-                                    ("add_rows", p.add_rows, (t, width), torch.float32),
-                                    ("add_vec", p.add_vec, (width,), torch.float32), ("shift", shift, (width,), torch.float32),
-                                    ("norm_weight", norm_weight, (width,), torch.float32)):
-        if ten is not None and tuple(_check(ten, name, dtype).shape) != shape:
-            raise KernelError(f"residual_step: {name} has shape {tuple(ten.shape)}, not {shape}")
+    update = p.launch_args(t, width)
+    for name, ten in (("shift", shift), ("norm_weight", norm_weight)):
+        if ten is not None and tuple(_check(ten, name, torch.float32).shape) != (width,):
+            raise KernelError(f"residual_step: {name} has shape {tuple(ten.shape)}, not {(width,)}")
     n = t if rows is None else _check(rows, "rows", torch.int32, 1).shape[0]
     h = torch.empty((n, width), dtype=out_dtype, device=x.device)
-    changes = p.y is not None or p.add_rows is not None or p.add_vec is not None
+    changes = p.changes
     fresh, stride = x, 0
     if shift is not None:
         if rows is not None or previous is None or step is None:
@@ -1323,8 +1440,7 @@ def residual_step(x: torch.Tensor, pending: Optional[ResidualUpdate], norm_weigh
         stride = _slot_stride(previous, width, "previous")
         fresh = torch.empty_like(x) if changes and keep else x
     stored = fresh.data_ptr() if changes and keep and rows is None else None
-    _run("hybrid", "ti_stream_step", x.data_ptr(), stored, _ptr(p.y), _ptr(p.scale), p.factor, _ptr(p.add_rows), _ptr(p.add_vec),
-         norm_weight.data_ptr(), float(eps), h.data_ptr(), _ptr(rows), n, _ptr(shift),
+    _run("hybrid", "ti_stream_step", x.data_ptr(), stored, *update, norm_weight.data_ptr(), float(eps), h.data_ptr(), _ptr(rows), n, _ptr(shift),
          previous.data_ptr() if shift is not None else None, stride, _ptr(step.token_seq) if shift is not None else None,
          _ptr(step.cu_seqlens) if shift is not None else None, _ptr(step.state_slots) if shift is not None else None, t, width,
          _dtype_code(p.y) if p.y is not None else _dtype_code(h), _dtype_code(h), _stream())
@@ -1466,7 +1582,7 @@ def conv_qkv_append(qkv: torch.Tensor, *, num_heads: int, num_kv_heads: int, hea
     return q
 
 
-def _check_head_extras(q, head_sinks, gate, gate_offset) -> None:
+def _check_head_extras(q, head_sinks, gate, gate_offset, gates_a_head: int = 1) -> None:
     t, hq, _ = q.shape
     if head_sinks is not None:
         _check(head_sinks, "head_sinks", torch.float32, 1)
@@ -1474,21 +1590,25 @@ def _check_head_extras(q, head_sinks, gate, gate_offset) -> None:
             raise KernelError("attention: one sink per query head")
     if gate is not None:
         _check(gate, "gate", q.dtype, 2)
-        if gate.shape[0] != t or gate_offset < 0 or gate_offset + hq > gate.shape[1]:
-            raise KernelError("attention: the gate holds one column per query head for every token")
+        if gate.shape[0] != t or gate_offset < 0 or gate_offset + hq * gates_a_head > gate.shape[1]:
+            raise KernelError("attention: the gate holds one column per query head, or per output feature, for every token")
+    elif gates_a_head > 1:
+        raise KernelError("attention: a gate per feature needs its logits")
 
 
 def attention_rows(q: torch.Tensor, cache: torch.Tensor, *, v_dim: int, positions: torch.Tensor, token_seq: torch.Tensor,
                    block_table: torch.Tensor, scale: float, sink: Optional[float] = None, window: Optional[int] = None,
                    chunk: Optional[int] = None, out_scale: float = 1.0, step=None, status: Optional[torch.Tensor] = None,
                    head_sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-                   gate_offset: int = 0, softcap: float = 0.0) -> torch.Tensor:
+                   gate_offset: int = 0, softcap: float = 0.0, keep_first: int = 0, feature_gate: bool = False,
+                   difference: Optional[tuple] = None) -> torch.Tensor:
     """Causal attention of q [T, Hq, d] over pages whose rows are [k (d) | v (dv)] (``cache``
     [1, pages, Hkv, page, d + dv]; or planes [2, pages, Hkv, page, d] where d == dv), float32 arithmetic, any sizes. ``sink``: a logit whose exponential joins every softmax denominator without a
     value (0.0: one is added to the sum of exp(score)); ``head_sinks`` float32 [Hq]: such a logit per query head
     instead. ``gate`` [T, cols] of q's dtype: the output of (token, head) is also multiplied by
     sigmoid(gate[token, gate_offset + head]). ``softcap`` > 0: a score s becomes softcap * tanh(s / softcap) before the
-    softmax. ``window``, ``chunk``: as in ``paged_attention``. Returns [T, Hq * dv], multiplied by ``out_scale`` before its rounding."""
+    softmax. ``window``, ``chunk``, ``keep_first``, ``feature_gate``, ``difference``: as in ``paged_attention`` (two maps of
+    d / 2 features). Returns [T, Hq * dv], multiplied by ``out_scale`` before its rounding."""
     _check(q, "q", None, 3)
     _check(cache, "cache", q.dtype, 5)
     _check(positions, "positions", torch.int32, 1)
@@ -1500,11 +1620,15 @@ def attention_rows(q: torch.Tensor, cache: torch.Tensor, *, v_dim: int, position
     out = torch.empty((t, hq * v_dim), dtype=q.dtype, device=q.device)
     if t == 0:
         return out
-    _check_head_extras(q, head_sinks, gate, gate_offset)
+    _check_head_extras(q, head_sinks, gate, gate_offset, v_dim if feature_gate else 1)
+    maps, share, diff_eps = (1, 0.0, 0.0) if difference is None else (2, float(difference[0]), float(difference[1]))
+    if maps == 2 and d % 2:
+        raise KernelError("attention_rows: two maps have equal halves of the features")
     _run("hybrid", "ti_attention_rows", out.data_ptr(), q.data_ptr(), cache.data_ptr(), positions.data_ptr(),
-         token_seq.data_ptr(), block_table.data_ptr(), block_table.shape[1], t, hq, hkv, d, v_dim, page_size, num_pages,
-         planes, float(scale), _mask_code(window, chunk), int(sink is not None), float(sink or 0.0), _ptr(head_sinks), _ptr(gate),
-         gate.shape[1] if gate is not None else 0, int(gate_offset), float(out_scale), float(softcap or 0.0), _ptr(status),
+         token_seq.data_ptr(), block_table.data_ptr(), block_table.shape[1], t, hq, hkv, d // maps, v_dim, page_size, num_pages,
+         planes, float(scale), _mask_code(window, chunk), _keep_first(keep_first, window), int(sink is not None), float(sink or 0.0),
+         _ptr(head_sinks), _ptr(gate), gate.shape[1] if gate is not None else 0, int(gate_offset), int(feature_gate),
+         float(out_scale), float(softcap or 0.0), maps, share, diff_eps, _ptr(status),
          _dtype_code(q), _stream())
     return out
 
@@ -1596,19 +1720,24 @@ def head_rotation(rows: torch.Tensor, *, num_heads: int, num_kv_heads: int, head
                   eps: float = 0.0, rotation: Optional[Rotation] = None, q_scale: float = 1.0, k_scale: float = 1.0,
                   cache: Optional[torch.Tensor] = None, block_table: Optional[torch.Tensor] = None,
                   out_float32: bool = False, status: Optional[torch.Tensor] = None,
-                  norm_after: bool = False) -> torch.Tensor:
+                  norm_after: bool = False, maps: int = 1, values_are_keys: bool = False) -> torch.Tensor:
     """Per-head RMS norm (plain weights, optional), rotation and constant factors on the query heads, and with
     ``has_kv`` the key heads, that lie in columns [offset, ...) of ``rows`` [T, cols] as [q (Hq d) | k (Hkv d) |
     v (Hkv dv)]; values pass unchanged. With ``cache`` (planes [2, pages, Hkv, page, d] where d == dv, or rows
     [1, pages, Hkv, page, d + dv]) keys and values go to their token's place in the pages and q [T, Hq, d] is
     returned; without one, and with ``has_kv``, the result is the row [q | k | v] (for a recurrent mixer), float32
     if ``out_float32``. ``norm_after``: the norm of q and k comes after the rotation, with the weights or, without
-    them, as a plain division by the root mean square. Float32 arithmetic, one rounding."""
+    them, as a plain division by the root mean square. ``maps``: a query and a key head are that many maps of ``head_dim``
+    features side by side, each normed and rotated by itself (the cached key then has maps * head_dim features, and q is
+    [T, Hq, maps * d]). ``values_are_keys``: the rows have no value columns, the values are the key columns as they come.
+    Float32 arithmetic, one rounding."""
     _check(rows, "rows", None, 2)
     _check(positions, "positions", torch.int32, 1)
     _check(token_seq, "token_seq", torch.int32, 1)
     t = rows.shape[0]
-    nq, nk, nv = num_heads * head_dim, num_kv_heads * head_dim, num_kv_heads * v_dim
+    nq, nk, nv = num_heads * maps * head_dim, num_kv_heads * maps * head_dim, 0 if values_are_keys else num_kv_heads * v_dim
+    if values_are_keys and (maps != 1 or v_dim != head_dim or cache is None):
+        raise KernelError("head_rotation: values that are the keys have one map, their size and a cache to go to")
     if offset < 0 or offset + nq + ((nk + nv) if has_kv else 0) > rows.shape[1]:
         raise KernelError("head_rotation: the rows do not hold these heads")
     for name, w in (("q_norm_weight", q_norm_weight), ("k_norm_weight", k_norm_weight)):
@@ -1625,7 +1754,7 @@ def head_rotation(rows: torch.Tensor, *, num_heads: int, num_kv_heads: int, head
             raise KernelError("head_rotation: a cache is written with keys and values")
         _check(cache, "cache", rows.dtype, 5)
         _check(block_table, "block_table", torch.int32, 2)
-        planes = _kv_planes(cache, num_kv_heads, head_dim, v_dim)
+        planes = _kv_planes(cache, num_kv_heads, maps * head_dim, v_dim)
         num_pages, page_size, max_blocks = cache.shape[1], cache.shape[3], block_table.shape[1]
     to_row = has_kv and cache is None
     width = nq + nk + nv if to_row else nq
@@ -1635,9 +1764,10 @@ def head_rotation(rows: torch.Tensor, *, num_heads: int, num_kv_heads: int, head
         _run("hybrid", "ti_head_rotation", out.data_ptr(), width, _ptr(cache), planes, rows.data_ptr(), rows.shape[1],
              int(offset), _ptr(q_norm_weight), _ptr(k_norm_weight), float(eps), *_rotation_args(rotation), float(q_scale),
              float(k_scale), positions.data_ptr(), token_seq.data_ptr(), _ptr(block_table), max_blocks, t, num_heads,
-             num_kv_heads, head_dim, v_dim, int(has_kv), page_size, num_pages, _ptr(status), int(out_float32),
+             num_kv_heads, head_dim, v_dim, int(has_kv), page_size, num_pages, int(maps), int(values_are_keys), _ptr(status),
+             int(out_float32),
              int(norm_after), _dtype_code(rows), _stream())
-    return out if to_row else out.view(t, num_heads, head_dim)
+    return out if to_row else out.view(t, num_heads, maps * head_dim)
 
 
 def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay_logits: torch.Tensor, beta_logits: torch.Tensor,

@@ -11,7 +11,10 @@ output gate sigmoid(W_g x)_h per (token, head) (``head_gate``: W_g's rows ride i
 layer without key/value tensors that reads what another layer cached (``shares_cache``), biases on q, k and v alone
 (``qkv_bias``), scores capped smoothly by a tanh (``softcap``) and q and k divided by their root mean square after the
 rotation (``qk_unit_norm``); these may be combined with a window, or with chunks (``chunk``: a query sees the keys of its
-own chunk of positions). Such a layer runs
+own chunk of positions). A window may keep a request's first positions (``keep_first``), the values may be the keys
+before norm and rotation (``values_are_keys``), the gate may be one per output feature (``feature_gate``), and a head
+may be the difference of two attention maps over the same values (``difference``: the maps of a head lie side by side in q
+and in the cached key, so a token's row in the cache is one key of twice the size and one value). Such a layer runs
 ``_attend_general``: packed product [q | k | v | g], per-head norm + rotation + append (``ops.head_rotation``),
 attention with the sinks and the gate in its epilogue. A short causal convolution over q, k and v (``conv_taps``) and a
 norm over all rows of q, and of k, at once (``qk_row_norm``) take the kernel that does everything between product and
@@ -37,9 +40,11 @@ class Attention(Mixer):
         self._rotation = self.position.rotation()      # opaque here: the kernel reads it
         self.w_qkv = self.b_qkv = self.w_o = self.b_o = None
         self.q_norm = self.k_norm = self.sinks = self.conv_w = None
+        self.share = 0.0            # of two maps: what of the second one's output is subtracted
         self._by_token = spec.conv_taps > 0 or spec.qk_row_norm is not None      # prepared a token at a time, not a head
         self._general = bool(spec.value_dim != spec.head_dim or spec.head_sinks or spec.head_gate or spec.shares_cache
                              or spec.qkv_bias or spec.softcap or spec.qk_unit_norm is not None or spec.chunk or self._by_token
+                             or spec.keep_first or spec.values_are_keys or spec.feature_gate or spec.difference is not None
                              or getattr(spec.position, "interleaved", False) or getattr(spec.position, "blend", None))
         if self._general and spec.bias:
             raise ValueError("biases on all four projections are not combined with value sizes, sinks, gates or shared caches")
@@ -47,6 +52,18 @@ class Attention(Mixer):
             raise ValueError("q and k are normed once: per head before the rotation or after it, or all rows at once")
         if spec.window and spec.chunk:
             raise ValueError("an attention layer has a window or chunks, not both")
+        if spec.keep_first and not spec.window:
+            raise ValueError("first positions are kept beside a window")
+        if spec.keep_first < 0 or (spec.head_gate and spec.feature_gate):
+            raise ValueError("a gate per head or one per feature, and a number of kept positions that is not negative")
+        if spec.values_are_keys and (spec.value_dim != spec.head_dim or spec.difference is not None or spec.qkv_bias):
+            raise ValueError("values that are the keys have their size, one map and no bias of their own")
+        if (spec.values_are_keys or spec.feature_gate or spec.difference is not None) and (self._by_token or spec.shares_cache
+                                                                                          or not spec.short_names):
+            raise ValueError("values that are keys, gates per feature and two maps come with short tensor names, key tensors of "
+                             "the layer's own and no convolution or row norm")
+        if spec.difference is not None and (spec.head_sinks or spec.chunk):
+            raise ValueError("two maps are not combined with sinks or chunks")
         if spec.conv_taps < 0 or (self._by_token and (spec.shares_cache or not spec.short_names)):
             raise ValueError("convolutions and row norms come with short tensor names and key/value tensors of the layer's own")
         if spec.qkv_bias and (spec.bias or spec.shares_cache or not spec.short_names):
@@ -59,13 +76,18 @@ class Attention(Mixer):
 
     def cache_need(self):
         s = self.spec
-        if s.value_dim != s.head_dim:       # keys and values of different sizes lie side by side in one row a token
-            return CacheNeed(s.num_kv_heads, s.head_dim + s.value_dim, s.window, planes=1, chunk=s.chunk)
-        return CacheNeed(s.num_kv_heads, s.head_dim, s.window, chunk=s.chunk)
+        key_dim = s.maps * s.head_dim
+        if s.value_dim != key_dim:          # keys and values of different sizes lie side by side in one row a token
+            return CacheNeed(s.num_kv_heads, key_dim + s.value_dim, s.window, planes=1, chunk=s.chunk, keep_first=s.keep_first)
+        return CacheNeed(s.num_kv_heads, key_dim, s.window, chunk=s.chunk, keep_first=s.keep_first)
+
+    def _value_rows(self):
+        """Rows of the packed product that are the values' own."""
+        return 0 if self.spec.values_are_keys else self.spec.num_kv_heads * self.spec.value_dim
 
     def _packed_width(self):
         s = self.spec
-        return s.q_size + s.kv_size + s.num_kv_heads * s.value_dim
+        return s.q_size + s.kv_size + self._value_rows()
 
     def state_need(self):
         taps = self.spec.conv_taps
@@ -76,7 +98,8 @@ class Attention(Mixer):
         t = {n["q"]: TensorSpec((s.q_size, s.hidden_size))}
         if not s.shares_cache:
             t[n["k"]] = TensorSpec((s.kv_size, s.hidden_size))
-            t[n["v"]] = TensorSpec((s.num_kv_heads * s.value_dim, s.hidden_size))
+            if not s.values_are_keys:
+                t[n["v"]] = TensorSpec((s.num_kv_heads * s.value_dim, s.hidden_size))
         t[n["o"]] = TensorSpec((s.hidden_size, s.num_heads * s.value_dim))
         if s.qk_norm is not None:
             t[n["q_norm"]] = TensorSpec((s.head_dim,), role="vector32", init="ones_noise")
@@ -92,6 +115,11 @@ class Attention(Mixer):
             t[n["sink"]] = TensorSpec((s.num_heads,), role="vector32")
         if s.head_gate:
             t[n["g"]] = TensorSpec((s.num_heads, s.hidden_size))
+        if s.feature_gate:
+            t[n["g"]] = TensorSpec((s.num_heads * s.value_dim, s.hidden_size))
+        if s.difference is not None:
+            for name in ("lq1", "lk1", "lq2", "lk2"):
+                t[name] = TensorSpec((s.head_dim,), role="vector32")
         if s.qkv_bias:
             t[n["q"] + ".b"] = TensorSpec((s.q_size,), role="vector32")
             t[n["k"] + ".b"] = TensorSpec((s.kv_size,), role="vector32")
@@ -105,8 +133,13 @@ class Attention(Mixer):
 
     def load(self, tensors):
         s, n = self.spec, self._n
-        rows = [tensors[n["q"]]] + ([] if s.shares_cache else [tensors[n["k"]], tensors[n["v"]]])
-        if s.head_gate:
+        rows = [tensors[n["q"]]] + ([] if s.shares_cache else [tensors[n["k"]]])
+        if not (s.shares_cache or s.values_are_keys):
+            rows.append(tensors[n["v"]])
+        if s.difference is not None:                     # lambda, made once
+            lq1, lk1, lq2, lk2 = (tensors[name].double().cpu() for name in ("lq1", "lk1", "lq2", "lk2"))
+            self.share = float(torch.exp((lq1 * lk1).sum()) - torch.exp((lq2 * lk2).sum()) + s.difference)
+        if s.head_gate or s.feature_gate:
             rows.append(tensors[n["g"]])                 # the gate's rows follow q, k and v
         if self._general:
             # zero rows fill the packed matrix up to a multiple of eight rows, which the tensor-core product wants
@@ -140,16 +173,19 @@ class Attention(Mixer):
         if own != bool(cache.writes):
             raise ValueError("a layer with key/value tensors writes its cache entry; one without them only reads")
         packed = ops.linear(x, self.w_qkv, bias=self.b_qkv)  # [T, q | (k | v) | (g) | fill]
-        gate_at = s.q_size + ((s.kv_size + s.num_kv_heads * s.value_dim) if own else 0)
+        gate_at = s.q_size + ((s.kv_size + self._value_rows()) if own else 0)
         q = self._prepare_by_token(packed, step, cache) if self._by_token else ops.head_rotation(
                               packed, num_heads=s.num_heads, num_kv_heads=s.num_kv_heads, head_dim=s.head_dim,
-                              v_dim=s.value_dim, has_kv=own, positions=step.positions, token_seq=step.token_seq,
+                              v_dim=s.value_dim, has_kv=own, maps=s.maps, values_are_keys=s.values_are_keys, positions=step.positions, token_seq=step.token_seq,
                               q_norm_weight=self.q_norm, k_norm_weight=self.k_norm,
                               eps=(s.qk_norm.eps if s.qk_norm is not None else s.qk_unit_norm or 0.0),
                               rotation=self._rotation, norm_after=s.qk_unit_norm is not None,
                               cache=cache.kv if own else None, block_table=cache.block_table, status=step.status)
-        extras = dict(head_sinks=self.sinks, gate=packed if s.head_gate else None, gate_offset=gate_at,
-                      window=s.window, chunk=s.chunk, softcap=s.softcap or 0.0)
+        extras = dict(head_sinks=self.sinks, gate=packed if s.head_gate or s.feature_gate else None, gate_offset=gate_at,
+                      feature_gate=s.feature_gate, window=s.window, chunk=s.chunk, keep_first=s.keep_first,
+                      softcap=s.softcap or 0.0)
+        if s.difference is not None:
+            extras.update(difference=(self.share, s.difference_eps), out_scale=1.0 - s.difference)
         if cache.kv.shape[0] == 2:          # keys and values of one size: the paged attention, tensor cores where the sizes allow
             return ops.paged_attention(q, cache.kv, positions=step.positions, token_seq=step.token_seq,
                                        block_table=cache.block_table, scale=s.scale, step=step, status=step.status,

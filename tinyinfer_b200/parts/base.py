@@ -21,12 +21,13 @@ class TensorSpec:
     """A tensor a part wants from the checkpoint.
     role 'matrix': kept in the compute dtype (bfloat16 or float32);
     role 'vector32': kept in float32 whatever the compute dtype (norm weights, biases of
-    32-bit parts); role 'int': kept as int32. A size of -1 is one that only the checkpoint gives (the
+    32-bit parts); role 'int': kept as int32 (random-weights mode: every row ``shape[-1]`` different numbers below ``below``). A size of -1 is one that only the checkpoint gives (the
     loader accepts any; the random-weights mode cannot draw such a tensor)."""
     shape: Tuple[int, ...]
     role: str = "matrix"
     init: str = "normal"          # random-weights mode: 'normal' N(0, std), 'ones_noise' 1 + N(0, 0.1) or
                                   # 'eye_noise' (a square matrix) identity + N(0, 0.1)
+    below: int = 1
 
 
 @dataclass(frozen=True)
@@ -34,12 +35,14 @@ class CacheNeed:
     """Paged keys and values a mixer wants per token: ``num_kv_heads * head_dim`` for K and V
     each. ``window`` None: every key stays; n: only the last n positions are ever read, older
     pages may be given back. ``chunk`` n: a position reads its own chunk of n positions only (chunks
-    counted from position 0 of the request), so the pages of earlier chunks may be given back."""
+    counted from position 0 of the request), so the pages of earlier chunks may be given back. ``keep_first`` n: beside the
+    window the first n positions are read to the end of the request, so their pages stay."""
     num_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     planes: int = 2          # 2: keys and values; 1: one row per token (a latent that both are made from)
     chunk: Optional[int] = None
+    keep_first: int = 0
 
     @property
     def keeps_all(self) -> bool:
@@ -47,7 +50,7 @@ class CacheNeed:
         return self.window is None and self.chunk is None
 
     def first_read(self, position: int) -> int:
-        """The lowest position that a query at ``position`` or later reads."""
+        """The lowest position that a query at ``position`` or later reads (beside the ``keep_first`` first ones)."""
         if self.chunk is not None:
             return position // self.chunk * self.chunk
         return 0 if self.window is None else max(0, position - self.window + 1)

@@ -184,7 +184,31 @@ class ScaledResidualBlock(Block):
         return (stream, pending), None
 
 
+class ParallelResidualBlock(Block):
+    """x <- x + m * (mixer(h) + feed_forward(h)), h = norm(x): one norm, which both sublayers read, around one float32 stream.
+    What travels between blocks is the pair (stream [T, width], update still to be applied); the update holds both sublayers'
+    outputs, which are summed in float32 as they are applied. Experts of equal weight leave their rows unsummed for that."""
+
+    def forward(self, x, step, cache):
+        return self.forward_linked(x, None, None, step, cache)[0]
+
+    def forward_linked(self, x, link, next_norm, step, cache):
+        from .. import ops
+        stream, pending = x
+        rms = self.mixer_norm.as_rms()
+        if rms is None:
+            raise ValueError("the parallel arrangement needs RMSNorms")
+        stream, h = ops.residual_step(stream, pending, rms[0], rms[1], self.mixer.dtype)
+        second = None
+        if self.feed_forward is not None:
+            run = self.feed_forward.forward_rows if getattr(self.feed_forward, "sums_rows", False) else self.feed_forward.forward
+            second = run(h, step)
+        mixed = self.mixer.forward(h, step, cache)
+        return (stream, ops.ResidualUpdate(mixed, factor=self.spec.residual_mult, second=second)), None
+
+
 register_block("pre_norm", PreNormBlock)
 register_block("multi_stream", MultiStreamBlock)
 register_block("output_norm", OutputNormBlock)
 register_block("scaled_residual", ScaledResidualBlock)
+register_block("parallel_residual", ParallelResidualBlock)

@@ -13,7 +13,10 @@ the token's row, expert(w h), and the outputs are summed as they are: the up pro
 the weight multiplies both halves of the stored product inside the activation kernel and costs no pass of its own),
 ``groups`` (equal runs of neighbouring experts, of which the ``keep_groups`` with the best expert take part in the choice),
 ``weight_scale`` (a factor on the weights) and ``shared_gate`` (the shared expert's output times one sigmoid a token; a
-shared expert of a silu-gated mixture is silu-gated too).
+shared expert of a silu-gated mixture is silu-gated too), ``table_rows`` (no router: row i of a table of integers names the
+experts of token id i, each of weight 1 / top). The routing of table layers is known from the step's token ids alone:
+``TableRoutes`` makes it for all of a model's layers in one launch before the first layer runs, and a layer that runs
+several times in a pass uses it every time.
 
 A step's (token, choice) pairs are put in expert order on the device and the experts run as two grouped
 products over row tiles; nothing is read back to the host and no token is ever dropped, so a token's result
@@ -52,6 +55,10 @@ class Experts(FeedForward):
             raise ValueError("the groups of experts are equal, and one to all of them are kept")
         if spec.keep_groups * ((spec.num_experts + spec.identity_experts) // spec.groups) < spec.top:
             raise ValueError("the kept groups hold fewer experts than are chosen")
+        if spec.table_rows < 0 or (spec.table_rows and (spec.identity_experts or spec.score_correction or spec.weight_input
+                                                        or spec.groups != 1 or spec.weight_scale != 1.0)):
+            raise ValueError("experts named by a table are plain experts of equal weight")
+        self.table = None
         self.glu = spec.activation in ("clamped_glu", "silu_glu")
         self.w_router = self.w_up = self.w_down = self.w_shared_up = self.w_shared_down = self.correction = None
         self.w_shared_gate = None
@@ -64,7 +71,10 @@ class Experts(FeedForward):
                 t[f"e{e}.gate"] = TensorSpec((s.expert_size, s.hidden_size))
             t[f"e{e}.up"] = TensorSpec((s.expert_size, s.hidden_size))
             t[f"e{e}.down"] = TensorSpec((s.hidden_size, s.expert_size))
-        t["router"] = TensorSpec((s.num_experts + s.identity_experts, s.hidden_size))
+        if s.table_rows:
+            t["table"] = TensorSpec((s.table_rows, s.top), role="int", below=s.num_experts)
+        else:
+            t["router"] = TensorSpec((s.num_experts + s.identity_experts, s.hidden_size))
         if s.score_correction:
             t["correction"] = TensorSpec((s.num_experts + s.identity_experts,), role="vector32")
         if s.shared_size:
@@ -86,7 +96,12 @@ class Experts(FeedForward):
         if s.score_correction:
             self.correction = tensors["correction"].contiguous()
         self.w_down = torch.stack([tensors[f"e{e}.down"] for e in range(s.num_experts)]).contiguous()
-        self.w_router = tensors["router"].contiguous()
+        if s.table_rows:
+            self.table = tensors["table"].contiguous()
+            if int(self.table.min()) < 0 or int(self.table.max()) >= s.num_experts:
+                raise ValueError(f"the table names experts outside 0..{s.num_experts - 1}")
+        else:
+            self.w_router = tensors["router"].contiguous()
         if s.shared_size:
             self.w_shared_up = (torch.cat([tensors["shared.gate"], tensors["shared.up"]], dim=0) if self.glu
                                 else tensors["shared.up"]).contiguous()
@@ -94,12 +109,32 @@ class Experts(FeedForward):
         if s.shared_gate:
             self.w_shared_gate = tensors["shared.sg"].reshape(-1).contiguous()
 
-    def _experts(self, x32, x):
+    @property
+    def sums_rows(self):
+        """The output is a plain sum of expert rows with equal weights, which the residual's own kernel can make
+        (``forward_rows``)."""
+        return bool(self.spec.table_rows) and not self.spec.shared_size
+
+    def forward_rows(self, x, step):
+        """The output as the experts' rows and where a token's lie (``ops.ExpertRows``), not summed yet."""
+        routing, down, _ = self._experts(x, x, step)
+        return ops.ExpertRows(down, routing.slot_of, 1.0 / self.spec.top)
+
+    def _table_routing(self, x, step):
+        made = getattr(step, "routings", {}).get(self)
+        return made if made is not None else ops.route_by_tables(step.token_ids, self.table[None], self.spec.num_experts,
+                                                                 self.tile_rows(x.shape[0]))[0]
+
+    def tile_rows(self, num_tokens):
+        """The more rows an expert gets, the taller the row tiles its grouped products are planned with."""
+        s = self.spec
+        return ops.expert_tile_rows_of(num_tokens, s.hidden_size, self.dtype, s.num_experts, s.top, s.expert_size)
+
+    def _experts(self, x32, x, step):
         """(routing, float32 sorted rows of the experts' outputs, the shared expert's output or None)."""
         s = self.spec
-        # the more rows an expert gets, the taller the row tiles its grouped products are planned with
-        routing = ops.route_experts(x32, self.w_router, s.top, s.weight_eps,
-                                    tile_rows=ops.expert_tile_rows(x, s.num_experts, s.top, s.expert_size),
+        routing = self._table_routing(x, step) if s.table_rows else ops.route_experts(x32, self.w_router, s.top, s.weight_eps,
+                                    tile_rows=self.tile_rows(x.shape[0]),
                                     correction=self.correction, renormalize=s.renormalize, real_experts=s.num_experts,
                                     scoring=s.scoring, groups=s.groups, keep_groups=s.keep_groups,
                                     weight_scale=s.weight_scale)
@@ -125,7 +160,7 @@ class Experts(FeedForward):
         if self.spec.identity_experts or self.spec.weight_input or self.spec.shared_gate:
             raise ValueError("identity experts, experts weighted at their input and gated shared experts are not built into "
                              "the fused output of this arrangement")
-        routing, down, shared = self._experts(x if self.spec.router_input == "input" else x32, x)
+        routing, down, shared = self._experts(x if self.spec.router_input == "input" else x32, x, step)
         return ops.experts_combine_norm_add(x32, down, shared, routing, rms[0], rms[1], self.dtype)
 
     def forward(self, x, step=None):
@@ -134,9 +169,32 @@ class Experts(FeedForward):
         s = self.spec
         if s.identity_experts and s.router_input != "input":
             raise ValueError("identity experts pass the sublayer's input on, which is also what the router must read")
-        routing, down, shared = self._experts(x if s.router_input == "input" or x.dtype == torch.float32 else x.float(), x)
+        routing, down, shared = self._experts(x if s.router_input == "input" or s.table_rows or x.dtype == torch.float32 else x.float(), x, step)
         return ops.experts_combine(down, x, routing, s.num_experts, weighted=not s.weight_input, shared=shared,
                                    shared_gate=self.w_shared_gate)
+
+
+class TableRoutes:
+    """The routing of all table-routed mixtures of a model, made at the start of a step: parts of equal sizes share one launch
+    and one tensor of tables (each part then holds a view of it)."""
+
+    def __init__(self, parts):
+        groups = {}
+        for part in parts:
+            s = part.spec
+            groups.setdefault((s.table_rows, s.num_experts, s.top, s.hidden_size, s.expert_size), []).append(part)
+        self.groups = []
+        for members in groups.values():
+            tables = torch.stack([p.table for p in members]).contiguous()
+            for p, view in zip(members, tables):
+                p.table = view
+            self.groups.append((members, tables))
+
+    def route(self, step):
+        step.routings = {}
+        for members, tables in self.groups:
+            made = ops.route_by_tables(step.token_ids, tables, members[0].spec.num_experts, members[0].tile_rows(step.num_tokens))
+            step.routings.update(zip(members, made))
 
 
 register_feed_forward("experts", Experts)

@@ -1,4 +1,4 @@
-"""Dense gated feed-forward: down(act(gate(x)) * up(x)), act silu (SwiGLU) or the tanh form of gelu, no bias
+"""Dense gated feed-forward: down(act(gate(x)) * up(x)), act silu (SwiGLU) or the tanh form of gelu, with or without biases
 (tinyinfer/models/qwen3.py:148-150,170-175 of the reference). Gate and up are packed as one
 [2I, H] matrix so that one matrix product feeds the activation, which acts on the float32
 accumulators as the reference's kernel does (tinyinfer/csrc/mlp.cu:116-141)."""
@@ -16,12 +16,15 @@ class GatedMLP(FeedForward):
         super().__init__(spec, dtype, device)
         if spec.activation not in ops.GATED_ACTIVATIONS:
             raise ValueError(f"activation {spec.activation!r} is not supported ({', '.join(ops.GATED_ACTIVATIONS)})")
-        self.w_gate_up = self.w_down = None
+        self.w_gate_up = self.w_down = self.b_gate_up = self.b_down = None
 
     def tensors(self):
         s = self.spec
         gate, up, down = s.names
+        biases = {name + ".b": TensorSpec((rows,), role="vector32") for name, rows in
+                  ((gate, s.intermediate_size), (up, s.intermediate_size), (down, s.hidden_size))} if s.bias else {}
         return {
+            **biases,
             gate: TensorSpec((s.intermediate_size, s.hidden_size)),
             up: TensorSpec((s.intermediate_size, s.hidden_size)),
             down: TensorSpec((s.hidden_size, s.intermediate_size)),
@@ -31,19 +34,22 @@ class GatedMLP(FeedForward):
         gate, up, down = self.spec.names
         self.w_gate_up = torch.cat([tensors[gate], tensors[up]], dim=0).contiguous()
         self.w_down = tensors[down].contiguous()
+        if self.spec.bias:
+            self.b_gate_up = torch.cat([tensors[gate + ".b"], tensors[up + ".b"]]).contiguous()
+            self.b_down = tensors[down + ".b"].contiguous()
 
     def _hidden(self, x, **link):
-        return ops.gated_linear(x, self.w_gate_up, activation=self.spec.activation, **link)
+        return ops.gated_linear(x, self.w_gate_up, bias=self.b_gate_up, activation=self.spec.activation, **link)
 
     def forward(self, x, step=None):
-        return ops.linear(self._hidden(x), self.w_down)
+        return ops.linear(self._hidden(x), self.w_down, bias=self.b_down)
 
     def forward_residual(self, x, residual, step=None):
-        return ops.linear(self._hidden(x), self.w_down, residual=residual)
+        return ops.linear(self._hidden(x), self.w_down, bias=self.b_down, residual=residual)
 
     def forward_prenorm(self, x, norm, link, next_norm, step=None):
         rms = norm.as_rms()
-        if rms is None or not ops.norm_link_ok(x):
+        if rms is None or self.spec.bias or not ops.norm_link_ok(x):
             return super().forward_prenorm(x, norm, link, next_norm, step)
         if link is not None and link.weight is rms[0]:
             hidden = self._hidden(link.scaled, link=link, link_eps=rms[1])

@@ -8,6 +8,7 @@ import math
 
 import torch
 
+from ..config.specs import WavelengthBlend
 from .base import PositionEncoding, register_position
 
 
@@ -21,7 +22,9 @@ class RotaryEncoding(PositionEncoding):
         if getattr(spec, "exact_frequencies", False) or blend is not None:
             exponent = torch.arange(0, spec.rotary_dim, 2, dtype=torch.float64) / spec.rotary_dim
             freq = float(spec.theta) ** -exponent
-            if blend is not None:
+            if isinstance(blend, WavelengthBlend):
+                freq = blended_by_wavelength(freq, blend)
+            elif blend is not None:
                 freq, self.factor = blended(freq, spec.rotary_dim, float(spec.theta), blend)
             self.inv_freq = freq.to(torch.float32).to(device)
         else:
@@ -50,6 +53,17 @@ def blended(freq: torch.Tensor, rotary_dim: int, theta: float, blend):
     j = torch.arange(rotary_dim // 2, dtype=torch.float64)
     ramp = torch.clamp((j - lo) / max(hi - lo, 0.001), 0.0, 1.0)
     return freq / blend.factor * ramp + freq * (1.0 - ramp), 0.1 * math.log(blend.factor) + 1.0
+
+
+def blended_by_wavelength(freq: torch.Tensor, blend: WavelengthBlend) -> torch.Tensor:
+    """Frequencies of a ``WavelengthBlend``. Float64 in, float64 out."""
+    if not blend.factor > 0 or not blend.original > 0 or not 0 < blend.low <= blend.high:
+        raise ValueError("a blend by wavelength needs a positive factor and original length, and 0 < low <= high")
+    length = 2.0 * math.pi / freq
+    share = (blend.original / length - blend.low) / max(blend.high - blend.low, 1e-300)
+    mixed = (1.0 - share) * freq / blend.factor + share * freq
+    return torch.where(length < blend.original / blend.high, freq,
+                       torch.where(length > blend.original / blend.low, freq / blend.factor, mixed))
 
 
 class NoPosition(PositionEncoding):

@@ -24,7 +24,10 @@ def _draw(ts, generator, std: float, device="cpu") -> torch.Tensor:
         raise ValueError(f"a tensor of shape {ts.shape} has a size that only a checkpoint gives: name it in the "
                          "configuration to draw random weights")
     if ts.role == "int":
-        return torch.zeros(ts.shape, dtype=torch.int32, device=device)
+        if ts.below <= 1:
+            return torch.zeros(ts.shape, dtype=torch.int32, device=device)
+        order = torch.rand((*ts.shape[:-1], ts.below), generator=generator, device=device).argsort(dim=-1)
+        return order[..., :ts.shape[-1]].to(torch.int32)
     t = torch.randn(ts.shape, generator=generator, dtype=torch.float32, device=device)
     if ts.init == "ones_noise":
         return 1.0 + 0.1 * t
