@@ -153,7 +153,7 @@ def test_pages_behind_a_window_go_back_and_those_of_kept_positions_stay(window, 
     assert manager.stats()["groups"][0]["free_pages"] == most
 
 
-@pytest.mark.parametrize("blend", [None, (4.0, 1.0, 4.0, 512), (8.0, 2.0, 2.0, 100), (2.0, 1.0, 32.0, 64)])
+@pytest.mark.parametrize("blend", [None, (4.0, 1.0, 4.0, 512), (8.0, 2.0, 2.0, 100), (2.0, 1.0, 8.0, 64)])
 def test_frequencies_scaled_by_wavelength(blend):
     """Against the plain statement, pair by pair; the middle range is reached where there is one."""
     rot = dict(base=5000.0, dims=32)

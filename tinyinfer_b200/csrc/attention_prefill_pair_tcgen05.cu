@@ -196,13 +196,15 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap q_map, const _
     }
     const bool has_b = t1x[1] > t0x[1];
     const int tmin = has_b ? min(t0x[0], t0x[1]) : t0x[0], tmax = has_b ? max(t1x[0], t1x[1]) : t1x[0];
-    // The CTA's tiles are numbered without a gap: 0 .. kept - 1 are those of kept first positions, number v >= kept is tile
-    // tmin + v - kept. Query tile X visits the kept ones and a run of the others that starts gap[X] tiles later (A's first key
-    // is never above B's, so gap[0] is 0): its i-th tile has number number_of(x, i), and it visits count[x] tiles.
+    // The CTA's tiles are numbered without a gap: 0 .. kept - 1 are those of kept first positions before the first tile of A's
+    // window, number v >= kept is tile tmin + v - kept. Query tile X visits own_kept[X] tiles from number 0 on (B's window may
+    // begin behind tiles of kept positions that lie in A's), then a run that begins gap[X] numbers later: its i-th tile has
+    // number number_of(x, i), and it visits count[x] tiles. A's first key is never above B's, so A leaves none out.
     const int kept = FORM == 0 ? 0 : ti_kept_tiles(p.keep, tmin, KT);
-    const int gap[2] = {t0x[0] - tmin, has_b ? t0x[1] - tmin : 0};
-    const int count[2] = {t1x[0] > t0x[0] ? kept + t1x[0] - t0x[0] : 0, has_b ? kept + t1x[1] - t0x[1] : 0};
-    auto number_of = [&](int x, int i) { return FORM != 0 && i < kept ? i : i + gap[x]; };
+    const int own_kept[2] = {kept, FORM == 0 ? 0 : ti_kept_tiles(p.keep, t0x[1], KT)};
+    const int gap[2] = {0, has_b ? kept + t0x[1] - tmin - own_kept[1] : 0};
+    const int count[2] = {t1x[0] > t0x[0] ? kept + t1x[0] - t0x[0] : 0, has_b ? own_kept[1] + t1x[1] - t0x[1] : 0};
+    auto number_of = [&](int x, int i) { return FORM != 0 && i < own_kept[x] ? i : i + gap[x]; };
     auto tile_of = [&](int v) { return FORM == 0 ? tmin + v : ti_nth_tile(v, kept, tmin); };
     const int lo = ti_first_key(pos0, p.window);                     // first key any query of the CTA sees
     const int hi = pos0 + nrows;                                     // one past the last
@@ -255,8 +257,8 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap q_map, const _
             unsigned long long idle_since = 0;
             // which of X's tiles number v is, or -1 if X does not visit it
             auto place_of = [&](int x, int v) {
-                const int i = FORM != 0 && v < kept ? v : v - gap[x];
-                return (FORM != 0 && v < kept ? count[x] > 0 : i >= kept && i < count[x]) ? i : -1;
+                const int i = FORM != 0 && v < own_kept[x] ? v : v - gap[x];
+                return i < count[x] && (FORM != 0 ? i == v || i >= own_kept[x] : i >= 0) ? i : -1;
             };
             auto all_issued = [&](const int* next, int v) {                // every query tile that visits number v has issued it
                 const int a = place_of(0, v), b = place_of(1, v);
@@ -301,7 +303,7 @@ prefill_attention_pair_kernel(const __grid_constant__ CUtensorMap q_map, const _
                     // whose keys may begin any number of tiles after A's (its rows lie in the next chunk), starts its
                     // first two tiles (behind the kept ones, and of those) only once A has issued P V of the number two before.
                     if (js[x] < count[x] && js[x] == jp[x] &&
-                        (x == 0 || js[1] >= (FORM != 0 && js[1] < kept ? 2 : kept + 2) || jp[0] + 1 >= number_of(1, js[1]))) {
+                        (x == 0 || js[1] >= (FORM != 0 && js[1] < own_kept[1] ? 2 : own_kept[1] + 2) || jp[0] + 1 >= number_of(1, js[1]))) {
                         const int v = number_of(x, js[x]), li = 2 * v, b = li % NBUF;
                         if (mbar_test_wait(kv_full(b), (li / NBUF) & 1u)) {
                             tmem_fence_after();
