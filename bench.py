@@ -31,6 +31,9 @@ width, the nearest design with latent attention and routed experts around a floa
 ``--design tarupel`` does it for the Tarupel design (chunked attention with short convolutions, windowed attention with
 whole-projection norms, the generalized delta rule, experts chosen by groups with a gated shared expert), beside Qwen3 and
 the Sinulix preset of the same width, the nearest design with a delta rule and gated experts.
+``--design zetonex`` does it for the Zetonex design (sublayers side by side, windows that keep first positions, differential
+attention, experts named by a table, a stretch of layers that runs twice), beside Qwen3 and the Fezozen preset of the same
+width, the nearest design with capped and windowed attention and experts around a float32 stream.
 
 ``--impl reference`` runs the unmodified reference project from ``baseline/_ref`` through its own
 public API (``tinyinfer.LLM(Config(...))``, ``add_request``, ``step``) on a model folder of the same
@@ -698,6 +701,42 @@ def tarupel_numbers(cfg, batch, context):
     return dict(macs=macs, attn_per_key=0.0, attn_window_keys=per_layer, head=head, step_bytes=step_bytes, scan_flops=scan_flops)
 
 
+def zetonex_numbers(cfg, batch, context):
+    """As ``fezozen_numbers`` for the Zetonex design: matrix elements a token multiplies (active experts, the projection a pass
+    of the loop starts with), attention flops per key (two maps and both products with the values in a differential layer)
+    with the keys a layer's window holds, and the bytes a decode step must move: dense weights of every layer run (a layer that
+    runs twice is read twice), the experts a batch of this size is expected to touch, the head, and of every run's cache the
+    rows its window and its kept positions hold."""
+    w, macs, dense, expert_bytes, cache_bytes, per_layer = cfg.width, 0, 0, 0.0, 0.0, []
+    for entry in cfg.execution():
+        layer = cfg.layers[entry.layer]
+        m, f = layer["mixer"], layer.get("mlp")
+        h, g, d, v = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        mask = m.get("mask") or {}
+        window = mask.get("size") or 0
+        seen = min(context, window + mask.get("keep_first", 0)) if window else context
+        if layer["type"] == "attention":
+            part = w * (h * d + g * d + h * v) + w * h * v
+            per_layer.append((2.0 * h * (d + v), window))
+        else:
+            part = w * (2 * h * d + g * (2 * d + v)) + w * h * v
+            per_layer.append((2.0 * h * 2 * (d + v), window))
+        cache_bytes += seen * g * ((1 if layer["type"] == "attention" else 2) * d + v) * 2
+        if f is not None and f["kind"] == "dense":
+            part += 3 * f["ff"] * w
+        elif f is not None:
+            e, top, ff = f["router"]["experts"], f["router"]["top"], f["expert"]["ff"]
+            macs += top * 3 * ff * w
+            expert_bytes += e * (1.0 - (1.0 - top / e) ** batch) * 3 * ff * w * 2
+        if entry.projects_embedding:
+            part += 2 * w * w
+        macs += part
+        dense += part
+    head = cfg.vocab * w
+    step_bytes = dense * 2 + expert_bytes + head * 2 + batch * cache_bytes
+    return dict(macs=macs, attn_per_key=0.0, attn_window_keys=per_layer, head=head, step_bytes=step_bytes)
+
+
 def windowed_attention_flops(per_layer, t):
     """Attention flops of a prompt of ``t`` tokens: position p sees min(p + 1, window) keys of a layer, or, where the
     size is negative, the p % size + 1 keys of its chunk."""
@@ -719,10 +758,12 @@ DESIGNS = {      # design -> (what its numbers are made with, [(its preset, the 
     "ravutar": (ravutar_numbers, (("ravutar-1b", "0.6b"), ("ravutar-2b", "1.7b"))),
     "sinulix": (sinulix_numbers, (("sinulix-1b", "0.6b"), ("sinulix-2b", "1.7b"))),
     "tarupel": (tarupel_numbers, (("tarupel-1b", "0.6b"), ("tarupel-2b", "1.7b"))),
+    "zetonex": (zetonex_numbers, (("zetonex-1b", "0.6b"), ("zetonex-2b", "1.7b"))),
 }
 SIBLINGS = {"sinulix-1b": ("ravutar", "ravutar-1b"), "sinulix-2b": ("ravutar", "ravutar-2b"),   # also measured beside it
             "fezozen-1b": ("gulisun", "gulisun-1b"), "fezozen-2b": ("gulisun", "gulisun-2b"),
-            "tarupel-1b": ("sinulix", "sinulix-1b"), "tarupel-2b": ("sinulix", "sinulix-2b")}
+            "tarupel-1b": ("sinulix", "sinulix-1b"), "tarupel-2b": ("sinulix", "sinulix-2b"),
+            "zetonex-1b": ("fezozen", "fezozen-1b"), "zetonex-2b": ("fezozen", "fezozen-2b")}
 
 
 
@@ -808,7 +849,7 @@ def design_comparison(args) -> int:
             sib = preset_config(preset)
             sn = DESIGNS[kind][0](sib, batch, context)
             sflops = (2.0 * sn["macs"] * t + sn["attn_per_key"] * t * (t + 1) / 2.0 + 2.0 * sn["head"]
-                      + sn.get("scan_flops", 0.0) * t)
+                      + sn.get("scan_flops", 0.0) * t + windowed_attention_flops(sn.get("attn_window_keys", ()), t))
             row[kind] = measure_design(sib, peaks, sflops, sn["step_bytes"], batch, context, steps, warmup, prefill_tokens)
             row[kind]["preset"] = preset
             row[kind]["layers"] = len(sib.run_order()) if hasattr(sib, "run_order") else len(sib.layers)
@@ -836,7 +877,7 @@ def main() -> int:
     ap.add_argument("--skip-points", action="store_true", help="only the headline batch")
     ap.add_argument("--skip-extras", action="store_true", help="leave out the 'configs' of the line")
     ap.add_argument("--extras", default="32b,mix,cpu", help="which of the other configurations to run")
-    ap.add_argument("--design", default="", choices=["", "gulisun", "ravutar", "sinulix", "fezozen", "tarupel"],
+    ap.add_argument("--design", default="", choices=["", "gulisun", "ravutar", "sinulix", "fezozen", "tarupel", "zetonex"],
                     help="instead of the headline: prefill and decode of this design beside Qwen3 at equal size")
     ap.add_argument("--ref-block-size", type=int, default=256, help="reference arm: its kvcache_block_size (its default)")
     ap.add_argument("--ref-step-tokens", type=int, default=32,

@@ -15,7 +15,13 @@ void ti_set_error(const char* fmt, ...) {
 }
 void ti_count_launch(int n) { g_launches.fetch_add(n, std::memory_order_relaxed); }
 
+// The next launch of this thread waits for everything it depends on to have ended (set where its stream has just been told to
+// wait for another one's work).
+static thread_local int g_plain_next = 0;
+TI_API void ti_plain_next_launch() { g_plain_next = 1; }
+
 bool ti_pdl_enabled() {
+    if (g_plain_next) { g_plain_next = 0; return false; }
     static int on = -1;
     if (on < 0) {
         const char* v = getenv("TINYINFER_B200_PDL");

@@ -45,15 +45,15 @@ PRESETS = {
                             rot=dict(base=10000.0, dims=8, scaling=_scaling(64))),
                        dict(kind="dense", ff=96), _moe(6, 2, 32))),
     "zetonex-1b": dict(
-        vocab=102400, width=1024, norm=dict(eps=1e-6), logit_scale=1.0,
-        layers=_layers("kD" * 4, dict(heads=8, kv_heads=4, dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=1024, keep_first=4),
+        vocab=102400, width=1024, norm=dict(eps=1e-6), logit_scale=1.0, loop=dict(start=2, stop=4, times=2),
+        layers=_layers("kD" * 3, dict(heads=8, kv_heads=4, dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=1024, keep_first=4),
                                       rot=dict(base=10000.0, dims=64)),
                        dict(heads=8, kv_heads=4, dim=64, vdim=128, scale=0.125, softcap=50.0, diff=0.3, mask=dict(size=2048),
                             rot=dict(base=500000.0, dims=64, scaling=_scaling(8192))),
                        dict(kind="dense", ff=3072), _moe(32, 4, 704))),
     "zetonex-2b": dict(
-        vocab=102400, width=2048, norm=dict(eps=1e-6), logit_scale=1.0,
-        layers=_layers("kD" * 4, dict(heads=16, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=1024, keep_first=4),
+        vocab=102400, width=2048, norm=dict(eps=1e-6), logit_scale=1.0, loop=dict(start=2, stop=4, times=2),
+        layers=_layers("kD" * 3, dict(heads=16, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, mask=dict(size=1024, keep_first=4),
                                       rot=dict(base=10000.0, dims=64)),
                        dict(heads=16, kv_heads=8, dim=64, vdim=128, scale=0.125, softcap=50.0, diff=0.3, mask=dict(size=2048),
                             rot=dict(base=500000.0, dims=64, scaling=_scaling(8192))),

@@ -243,13 +243,13 @@ _workspace = {}
 
 
 def _gemm_scratch(device):
-    """(partials, counters) shared by all tensor-core matrix products on this device; safe because
-    they are ordered on one stream and every launch leaves the counters at zero."""
-    key = torch.device(device)
+    """(partials, counters) shared by all tensor-core matrix products of a chain of kernels on this device; safe because
+    they are ordered on its stream and every launch leaves the counters at zero."""
+    key = (torch.device(device), _branch)
     pair = _workspace.get(key)
     if pair is None:
-        pair = _workspace[key] = (torch.empty(_WORKSPACE_FLOATS, dtype=torch.float32, device=key),
-                                  torch.zeros(_NUM_COUNTERS, dtype=torch.int32, device=key))
+        pair = _workspace[key] = (torch.empty(_WORKSPACE_FLOATS, dtype=torch.float32, device=key[0]),
+                                  torch.zeros(_NUM_COUNTERS, dtype=torch.int32, device=key[0]))
     return pair
 
 
@@ -273,6 +273,10 @@ def _fn(lib_name: str, name: str):
 
 
 def _run(lib_name: str, name: str, *args) -> None:
+    global _plain_next
+    if _plain_next:
+        library.load(lib_name).ti_plain_next_launch()
+        _plain_next = False
     rc = _fn(lib_name, name)(*args)
     if rc != 0:
         msg = library.load(lib_name).ti_last_error().decode(errors="replace")
@@ -288,6 +292,48 @@ def _stream() -> int:
     if _raw_stream is not None:
         return _raw_stream(torch.cuda.current_device())
     return torch.cuda.current_stream().cuda_stream
+
+
+_plain_next = False       # the next launch follows another stream's work and must not start before that has ended
+_branch = 0               # 1 while a ``Beside`` is open: products then use scratch of their own
+_side_streams = {}
+
+
+class Beside:
+    """Two independent chains of kernels side by side: what is launched inside ``with Beside(device) as b:`` runs on a second
+    stream behind everything launched so far; what is launched between its end and ``b.join()`` runs on the current stream
+    beside it, and what follows ``join`` waits for both. Eagerly and inside a graph capture alike. The second stream has the higher
+    priority: its chain should be the one of short kernels that wait for each other. Tensors made in one chain may be used
+    after the join; scratch that kernels of both chains would share (matrix products' partial sums) is kept apart. Kernels whose
+    CTAs wait for one another may run in one of the chains only: the other one's must come to an end by themselves."""
+
+    def __init__(self, device):
+        key = torch.device(device)
+        side = _side_streams.get(key)
+        if side is None:
+            side = _side_streams[key] = torch.cuda.Stream(key, priority=-1)
+        self.side, self.main = side, torch.cuda.current_stream(key)
+
+    def __enter__(self):
+        global _branch, _plain_next
+        if _branch:
+            raise KernelError("one chain beside another, not more")
+        self.side.wait_stream(self.main)
+        self._guard = torch.cuda.stream(self.side)
+        self._guard.__enter__()
+        _branch, _plain_next = 1, True
+        return self
+
+    def __exit__(self, *exc):
+        global _branch, _plain_next
+        _branch, _plain_next = 0, False
+        self._guard.__exit__(*exc)
+        return False
+
+    def join(self) -> None:
+        global _plain_next
+        self.main.wait_stream(self.side)
+        _plain_next = True
 
 
 def _dtype_code(t: torch.Tensor) -> int:
@@ -657,7 +703,8 @@ def release_scratch(device) -> None:
     key = torch.device(device)
     _attn_scratch.pop(key, None)
     _attn_scratch_outgrown.clear()
-    _workspace.pop(key, None)
+    for branch in (0, 1):
+        _workspace.pop((key, branch), None)
     _argmax_scratch.pop(key, None)
     _sample_scratch.pop(key, None)
 

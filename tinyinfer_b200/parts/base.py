@@ -180,6 +180,11 @@ class Mixer(Part):
 
 
 class FeedForward(Part):
+    def runs_beside(self, num_tokens: int) -> bool:
+        """Whether a step of so many tokens gains from running this part beside a mixer that reads the same input (few tokens:
+        chains of short kernels), and none of its kernels' CTAs wait for one another then (see ``ops.Beside``)."""
+        return False
+
     graph_safe = False      # as for a mixer: a feed-forward that picks its experts' rows on the host is not
 
     def forward(self, x: torch.Tensor, step) -> torch.Tensor:

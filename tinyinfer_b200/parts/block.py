@@ -187,7 +187,9 @@ class ScaledResidualBlock(Block):
 class ParallelResidualBlock(Block):
     """x <- x + m * (mixer(h) + feed_forward(h)), h = norm(x): one norm, which both sublayers read, around one float32 stream.
     What travels between blocks is the pair (stream [T, width], update still to be applied); the update holds both sublayers'
-    outputs, which are summed in float32 as they are applied. Experts of equal weight leave their rows unsummed for that."""
+    outputs, which are summed in float32 as they are applied. Experts of equal weight leave their rows unsummed for that.
+    In steps of few tokens, where a layer is two chains of kernels too short to fill the machine, the mixer's chain runs on a
+    stream of its own beside the feed-forward's."""
 
     def forward(self, x, step, cache):
         return self.forward_linked(x, None, None, step, cache)[0]
@@ -199,11 +201,16 @@ class ParallelResidualBlock(Block):
         if rms is None:
             raise ValueError("the parallel arrangement needs RMSNorms")
         stream, h = ops.residual_step(stream, pending, rms[0], rms[1], self.mixer.dtype)
-        second = None
-        if self.feed_forward is not None:
-            run = self.feed_forward.forward_rows if getattr(self.feed_forward, "sums_rows", False) else self.feed_forward.forward
+        if self.feed_forward is None:
+            return (stream, ops.ResidualUpdate(self.mixer.forward(h, step, cache), factor=self.spec.residual_mult)), None
+        run = self.feed_forward.forward_rows if getattr(self.feed_forward, "sums_rows", False) else self.feed_forward.forward
+        if self.feed_forward.runs_beside(step.num_tokens):
+            with ops.Beside(h.device) as chains:
+                mixed = self.mixer.forward(h, step, cache)
             second = run(h, step)
-        mixed = self.mixer.forward(h, step, cache)
+            chains.join()
+        else:
+            mixed, second = self.mixer.forward(h, step, cache), run(h, step)
         return (stream, ops.ResidualUpdate(mixed, factor=self.spec.residual_mult, second=second)), None
 
 

@@ -109,6 +109,9 @@ class Experts(FeedForward):
         if s.shared_gate:
             self.w_shared_gate = tensors["shared.sg"].reshape(-1).contiguous()
 
+    def runs_beside(self, num_tokens):
+        return num_tokens <= 64 and not self.spec.shared_size       # grouped products: no CTA waits for another
+
     @property
     def sums_rows(self):
         """The output is a plain sum of expert rows with equal weights, which the residual's own kernel can make

@@ -38,6 +38,9 @@ class GatedMLP(FeedForward):
             self.b_gate_up = torch.cat([tensors[gate + ".b"], tensors[up + ".b"]]).contiguous()
             self.b_down = tensors[down + ".b"].contiguous()
 
+    def runs_beside(self, num_tokens):
+        return num_tokens < 16            # from 16 tokens on the units of a product's tile wait for each other's partial sums
+
     def _hidden(self, x, **link):
         return ops.gated_linear(x, self.w_gate_up, bias=self.b_gate_up, activation=self.spec.activation, **link)
 
