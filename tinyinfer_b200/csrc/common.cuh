@@ -193,11 +193,11 @@ template <int N, typename P> __device__ __forceinline__ void ti_gate_features(co
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
             const float2 z = __bfloat1622float2(z2[i]);
-            v[2 * i] *= 1.f / (1.f + expf(-z.x));
-            v[2 * i + 1] *= 1.f / (1.f + expf(-z.y));
+            v[2 * i] = __fdividef(v[2 * i], 1.f + __expf(-z.x));          // v is rounded to 8 bits next
+            v[2 * i + 1] = __fdividef(v[2 * i + 1], 1.f + __expf(-z.y));
         }
     } else {
 #pragma unroll
-        for (int i = 0; i < N; ++i) v[i] *= 1.f / (1.f + expf(-__bfloat162float(g[i])));
+        for (int i = 0; i < N; ++i) v[i] = __fdividef(v[i], 1.f + __expf(-__bfloat162float(g[i])));
     }
 }

@@ -592,7 +592,8 @@ __global__ void moe_clamped_glu_vec_kernel(__nv_bfloat16* __restrict__ out, cons
             const float2 g = __bfloat1622float2(g2[k]), u = __bfloat1622float2(u2[k]);
             const float ga = fminf(g.x, limit), gb = fminf(g.y, limit);
             const float ua = fminf(fmaxf(u.x, -limit), limit), ub = fminf(fmaxf(u.y, -limit), limit);
-            o2[k] = __floats2bfloat162_rn(ga / (1.f + expf(-alpha * ga)) * (ua + 1.f), gb / (1.f + expf(-alpha * gb)) * (ub + 1.f));
+            o2[k] = __floats2bfloat162_rn(__fdividef(ga, 1.f + __expf(-alpha * ga)) * (ua + 1.f),      // rounded to 8 bits
+                                          __fdividef(gb, 1.f + __expf(-alpha * gb)) * (ub + 1.f));
         }
         reinterpret_cast<uint4*>(out + r * ff)[c] = o4;
     }
