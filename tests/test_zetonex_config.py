@@ -153,7 +153,7 @@ def test_pages_behind_a_window_go_back_and_those_of_kept_positions_stay(window, 
     assert manager.stats()["groups"][0]["free_pages"] == most
 
 
-@pytest.mark.parametrize("blend", [None, (4.0, 1.0, 4.0, 512), (8.0, 2.0, 2.0, 100), (2.0, 1.0, 8.0, 64)])
+@pytest.mark.parametrize("blend", [None, (5.0, 1.0, 4.0, 400), (8.0, 2.0, 2.0, 100), (2.0, 1.0, 8.0, 64)])
 def test_frequencies_scaled_by_wavelength(blend):
     """Against the plain statement, pair by pair; the middle range is reached where there is one."""
     rot = dict(base=5000.0, dims=32)
@@ -253,7 +253,7 @@ def test_plain_difference_of_equal_maps():
 
 def test_plain_scaled_frequency_meets_at_both_ends():
     """At the two wavelengths where the ranges meet, the blend equals what the range beyond it gives."""
-    s = zh.scaling(4.0, 1.0, 4.0, 512)
-    for length, want in ((512 / 4.0, 1.0), (512 / 1.0, 0.25)):
+    s = zh.scaling(5.0, 1.5, 6.0, 400)
+    for length, want in ((400 / 6.0, 1.0), (400 / 1.5, 0.2)):
         share = (s["original"] / length - s["low"]) / (s["high"] - s["low"])
         assert math.isclose((1 - share) / s["factor"] + share, want)
